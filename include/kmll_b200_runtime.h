@@ -28,7 +28,7 @@ extern "C" {
 
 typedef void* kmll_decoder_t;
 
-enum { KMLL_FORMAT_RS_I8 = 0, KMLL_FORMAT_W4G128 = 1 };
+enum { KMLL_FORMAT_RS_I8 = 0, KMLL_FORMAT_W4G128 = 1, KMLL_FORMAT_BF16 = 2 /* layered decoders: bf16 rows as a checkpoint stores them */ };
 
 /* Tensor ids for kmll_decoder_*_tensor.  Linear weights are [out_features, in_features]
  * (crates/inference/src/model.rs:8711-8760); names follow kmll's layer fields. */
@@ -46,7 +46,17 @@ enum {
     KMLL_T_EMBEDDING = 10,     /* bf16 [vocab, dim]     (layer = -1) */
     KMLL_T_OUTPUT = 11,        /* lm_head [vocab, dim]  (layer = -1) */
     KMLL_T_Q_NORM = 12,        /* optional, bf16 [head_dim]: per-head RMSNorm of the query rows before RoPE (model.rs:10165-10194); */
-    KMLL_T_K_NORM = 13         /* same for the key rows.  Set them before the first decode step; a model without them sets neither. */
+    KMLL_T_K_NORM = 13,        /* same for the key rows.  Set them before the first decode step; a model without them sets neither. */
+    /* layered decoders (kmll_layered_create).  ATTENTION_NORM / FFN_NORM are the norms ahead of the mixer and of the feed-forward,
+     * WQ / WK / WV / WO the mixer's projections, W3 / W2 the feed-forward's up and down projections. */
+    KMLL_T_POSITION = 14,      /* learned position vectors [position_rows, dim]   (layer = -1) */
+    KMLL_T_GATE = 15,          /* linear attention: output gate [heads*vdim, dim] */
+    KMLL_T_MIX_NORM = 16,      /* linear attention: weight [heads*vdim] of the norm over all heads */
+    KMLL_T_DKV = 17,           /* latent attention: [kv_rank + rot_dim, dim] */
+    KMLL_T_DKV_NORM = 18,      /* latent attention: [kv_rank] */
+    KMLL_T_UK = 19,            /* latent attention: latent -> keys [heads*dim, kv_rank] */
+    KMLL_T_UV = 20,            /* latent attention: latent -> values [heads*vdim, kv_rank] */
+    KMLL_T_ACT = 21            /* PolyNorm coefficients a, b, c, e [4] */
 };
 
 /* TextConfig of kmll (crates/inference/src/model.rs:271-366) reduced to what the decoder path uses. */
@@ -154,6 +164,69 @@ int kmll_decoder_launches_per_step(kmll_decoder_t dec);
 size_t kmll_decoder_weight_bytes(kmll_decoder_t dec);
 size_t kmll_decoder_kv_bytes(kmll_decoder_t dec);
 size_t kmll_decoder_resident_bytes(kmll_decoder_t dec);
+
+/* ---- layered decoders ----------------------------------------------------------------------------------------------
+ * A decoder over a list of layer descriptions with bf16 weights: pre-norm layers (x += mixer(norm(x)), x += feed_forward(
+ * norm(x))) whose mixers are latent attention or linear attention with a fixed decay per head, in any order and with sizes of
+ * their own.  The handle is an ordinary kmll_decoder_t: prefill, generate_greedy, enqueue_steps, history, step_host, next_top,
+ * set_pending, rewind, position, last_hidden, next_logits, set_tensor / get_tensor / init_random, the byte counts and destroy
+ * work on it (rewind replays tokens from the nearest remembered state, since a recurrent state cannot be cut back).  No
+ * counterpart in kmll.  Not for layered decoders: tensor parallelism, the lockstep batch, archives, prefill_token_loop. */
+enum { KMLL_MIXER_LATENT_ATTENTION = 1, KMLL_MIXER_LINEAR_ATTENTION = 2 };
+enum { KMLL_ACT_NONE = 0, KMLL_ACT_SILU = 1, KMLL_ACT_SIGMOID = 2 };
+enum { KMLL_MLP_NONE = 0, KMLL_MLP_POLYNORM = 1 };
+/* norm of a linear-attention output ahead of its gate */
+enum { KMLL_OUT_NORM_PER_HEAD = 0 /* each head over its own root mean square, no weight */, KMLL_OUT_NORM_JOINT = 1 /* all heads together, weighted */ };
+
+typedef struct {
+    int mixer;       /* KMLL_MIXER_* */
+    int heads;
+    int dim;         /* per head: query / key size (latent attention: the part that is not rotated) */
+    int vdim;        /* per head: value size */
+    /* latent attention: one latent of kv_rank values (RMS-normed) and one rotated key part of rot_dim values per position;
+     * scores (q . W_uk c + q_rot . k_rot) * score_scale, values W_uv c */
+    int kv_rank;
+    int rot_dim;     /* even; 0 = no rotated part */
+    int window;      /* > 0: a position sees itself and the window - 1 positions before it; 0: every earlier position */
+    float score_scale;
+    /* linear attention: S <- decay S + k v^T, o = S^T q; q, k, v through qkv_act, the first rot_dim entries of q and k rotated,
+     * k times key_scale; o normed (out_norm), times gate_act(W_g h) */
+    int qkv_act;     /* KMLL_ACT_NONE / KMLL_ACT_SILU */
+    int gate_act;    /* KMLL_ACT_SILU / KMLL_ACT_SIGMOID */
+    int out_norm;    /* KMLL_OUT_NORM_* */
+    float key_scale;
+    int mlp;         /* KMLL_MLP_* */
+    int ff;          /* feed-forward width */
+} kmll_layer_spec;
+
+typedef struct {
+    int n_layers;
+    int dim;
+    int vocab_size;
+    int max_seq_len;
+    int position_rows; /* > 0: a learned position vector is added to the embedding (max_seq_len <= position_rows); 0: none */
+    float norm_eps;
+    float norm_offset; /* layer and final norms multiply by (norm_offset + w): 1 for weights stored around zero, else 0 */
+    int compute_f32;   /* 0: bf16 activations into the tensor-core projections of a prompt, bf16 latent cache; 1: f32 throughout */
+} kmll_layered_config;
+
+size_t kmll_layer_spec_bytes(void);
+size_t kmll_layered_config_bytes(void);
+int kmll_layered_create(const kmll_layered_config* config, const kmll_layer_spec* layers, kmll_decoder_t* out);
+/* Rotation of a layer with rot_dim > 0: rot_dim / 2 frequencies and the factor on cos and sin.  Entry i is paired with entry
+ * i + rot_dim / 2; the table is built on the device in f64 and rounded once. */
+int kmll_layered_set_rotation(kmll_decoder_t dec, int layer, const double* freqs_host, int count, double magnitude);
+/* Decay of every head of a linear-attention layer. */
+int kmll_layered_set_decay(kmll_decoder_t dec, int layer, const double* decay_host, int count);
+/* The next n tokens of the sequence, continuing at kmll_decoder_position (a portion of a prompt, or one decoded token).
+ * want[n_want]: ascending offsets into `tokens` whose logits go to the device buffer logits_device [n_want, vocab_size].
+ * Leaves the arg-max of the last token pending.  Enqueues, then synchronises. */
+int kmll_decoder_extend(kmll_decoder_t dec, kmll_stream_t stream, const uint32_t* tokens_host, int n, const int* want, int n_want, float* logits_device);
+/* Forget the sequence: the next kmll_decoder_extend starts at position 0. */
+int kmll_decoder_reset(kmll_decoder_t dec, kmll_stream_t stream);
+/* The residual stream behind every layer for the last extend call is kept when a buffer [n_layers, n, dim] is attached (null
+ * detaches); parity checks. */
+int kmll_layered_tap(kmll_decoder_t dec, float* residual_device);
 
 /* ---- on-disk archive of the quantized linear weights ---------------------------------------------------------
  * The directory layout of kmll's quantization export, so an archive written by either side loads on the other:

@@ -260,6 +260,7 @@ int kmll_archive_validate(const char* dir, const kmll_decoder_config* config, co
 }
 
 int kmll_decoder_export_archive(kmll_decoder_t dec, const kmll_decoder_config* config, const char* dir, const char* weights_path) {
+    if (config != nullptr && config->format == KMLL_FORMAT_BF16) return fail(KMLL_ERR_UNSUPPORTED, "archives hold quantized tensors; bf16 weights stay in their checkpoint");
     KMLL_REQUIRE_PTR(dec); KMLL_REQUIRE_PTR(config); KMLL_REQUIRE_PTR(dir);
     if (config->tp_size != 1) return fail(KMLL_ERR_UNSUPPORTED, "export needs the full tensors: use a decoder with tp_size 1");
     for (const TensorSpec& t : tensor_specs(*config)) {
@@ -277,6 +278,7 @@ int kmll_decoder_export_archive(kmll_decoder_t dec, const kmll_decoder_config* c
 // MinistralAllLinearInt8Runtime::new_from_export (crates/inference/src/model.rs:6327-6384): validate, then read and upload
 // every linear tensor (every tensor-parallel rank reads the full tensor and keeps its shard)
 int kmll_decoder_load_archive(kmll_decoder_t dec, const kmll_decoder_config* config, const char* dir, const char* expected_weights_path) {
+    if (config != nullptr && config->format == KMLL_FORMAT_BF16) return fail(KMLL_ERR_UNSUPPORTED, "archives hold quantized tensors; bf16 weights stay in their checkpoint");
     KMLL_REQUIRE_PTR(dec); KMLL_REQUIRE_PTR(config); KMLL_REQUIRE_PTR(dir);
     int rc = kmll_archive_validate(dir, config, expected_weights_path);
     if (rc != KMLL_OK) return rc;

@@ -11,6 +11,7 @@
 #include <mutex>
 
 #include "internal.cuh"
+#include "mma_bf16.cuh"
 
 namespace kmll {
 
@@ -533,48 +534,6 @@ __global__ void __launch_bounds__(kAttnThreads, 2) decode_attention_kernel(const
 // remainder like the other operand; three of the four partial products are accumulated, so both operands count with 16
 // mantissa bits (a relative 2^-17 per product, far inside the tolerance of the parity tests, but not the f32 products
 // of the kernel above).  One block per multiprocessor (137 KB of stages).
-// the same copies with the destination given as a shared-space address; the second form writes zeros when src_bytes is 0
-__device__ inline void cp_async16_to(uint32_t smem_addr, const void* gmem_src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr), "l"(gmem_src) : "memory");
-}
-__device__ inline void cp_async16_zfill_to(uint32_t smem_addr, const void* gmem_src, uint32_t src_bytes) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr), "l"(gmem_src), "r"(src_bytes) : "memory");
-}
-__device__ inline float ex2_approx(float x) {  // 2^x, about 2 ulp; ex2(-inf) = 0
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ inline void ldmatrix_x4(uint32_t (&r)[4], const void* smem_row) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"((uint32_t)__cvta_generic_to_shared(smem_row))
-                 : "memory");
-}
-__device__ inline void ldmatrix_x4_trans(uint32_t (&r)[4], const void* smem_row) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"((uint32_t)__cvta_generic_to_shared(smem_row))
-                 : "memory");
-}
-// 8x8 transpose of 16-bit elements across the warp: lane T holds row T/4, columns 2(T%4), 2(T%4)+1 before and after
-__device__ inline uint32_t movmatrix_trans(uint32_t a) {
-    uint32_t d;
-    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(d) : "r"(a));
-    return d;
-}
-// D += A * B, m16n8k16, bf16 operands, f32 accumulate
-__device__ inline void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// (x0, x1) -> bf16 pair of the values rounded to nearest-even (x0 in the low half) and bf16 pair of the remainders
-__device__ inline void split_bf16x2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
-    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(hi) : "f"(x1), "f"(x0));
-    const float r0 = x0 - __uint_as_float(hi << 16), r1 = x1 - __uint_as_float(hi & 0xffff0000u);
-    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(lo) : "f"(r1), "f"(r0));
-}
 
 template <int HD, int GQM, bool F32KV>
 __global__ void __launch_bounds__(kAttnThreads, F32KV ? 1 : 2) decode_attention_mma_kernel(const DecodeAttnParams p_in) {

@@ -187,4 +187,16 @@ inline cudaError_t launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_
     return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
 
+// Opt a kernel in to all the dynamic shared memory a block can have (227 KB less the kernel's static part).  Set to the same
+// value at every launch, on whatever device is current: a CUDA graph replays its kernel nodes against the attribute the
+// function has at that time, so a value that followed the needs of the last captured launch would be too small for an
+// earlier node that needs more.
+template <typename K>
+inline cudaError_t allow_all_dynamic_smem(K kernel) {
+    cudaFuncAttributes fa;
+    cudaError_t e = cudaFuncGetAttributes(&fa, kernel);
+    if (e != cudaSuccess) return e;
+    return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - (int)fa.sharedSizeBytes);
+}
+
 }  // namespace kmll

@@ -3,6 +3,7 @@
 // CUDA graph stays valid while the sequence grows.
 #pragma once
 
+#include "../../include/kmll_b200_runtime.h"
 #include "common.cuh"
 
 namespace kmll {
@@ -164,10 +165,11 @@ int prepare_prefill_offset(cudaStream_t stream, const float* q, const float* k, 
 int write_kv_row(cudaStream_t stream, const float* x, int position, int token_len, int head_dim, float* cache, int kv_bf16);
 int prefill_attention_launch(cudaStream_t stream, const float* q_batch, const float* k_cache, const float* v_cache, int prompt_len,
                              int n_heads, int n_kv_heads, int head_dim, float* out, int kv_bf16, int window, int tensor_cores);
-// hidden = embedding[state->next_top.token]; also records next_top into history[state->step] and
+// hidden = embedding[state->next_top.token] (+ pos_table[position]); token_log[position] = token; also records next_top into history[state->step] and
 // sets seq_len = position + 1.
 int decode_begin(cudaStream_t stream, const uint16_t* table, int vocab, int dim, DecodeState* state, uint64_t* history,
-                 int history_cap, float* hidden, unsigned int* exchange_epoch = nullptr);
+                 int history_cap, float* hidden, unsigned int* exchange_epoch = nullptr, const uint16_t* pos_table = nullptr,
+                 uint32_t* token_log = nullptr);
 // state->next_top = *packed; position += 1; step += 1.
 int decode_end(cudaStream_t stream, const uint64_t* packed, DecodeState* state);
 
@@ -199,6 +201,110 @@ int linear_batched_form(int form, cudaStream_t stream, int fmt, const float* x, 
                         const void* const* w, const void* const* scales, const int* rows, int cols, float* const* outs,
                         const float* residual, void* workspace = nullptr, float* gate_tmp = nullptr, float* up_tmp = nullptr);
 size_t linear_batched_workspace_bytes(int batch, int in_dim);
+// ---- bf16 weights (linear_bf16.cuh) ------------------------------------------------------------------------------------
+// What happens to the vector x ahead of a projection:
+//   PRO_RMSNORM   x / rms(x) * (norm_offset + norm_w)
+//   PRO_POLYNORM  a N(x) + b N(x^2) + c N(x^3) + e with coef = (a, b, c, e), N = division by the root mean square
+//   PRO_GATED     x / rms (over all of x times norm_w, or per head_len entries when norm_w is null) * gate_act(gate)
+enum { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_POLYNORM = 2, PRO_GATED = 3 };
+constexpr int kMatvecMaxBlocks = 4096;  // partial arg-max entries a caller provides
+struct Bf16Matvec {
+    const uint16_t* w;   // [rows, ldw] bf16
+    int rows, K, ldw;
+    const float* x;      // [K]
+    int pro;
+    float eps, norm_offset;
+    const uint16_t* norm_w;
+    const uint16_t* coef;
+    const float* gate;
+    int gate_act, head_len;
+    float* y;            // [rows]
+    const float* residual;
+    int silu_rows;       // rows below this index go through SiLU
+    // arg-max over the rows (packed != null): partials of kMatvecMaxBlocks entries, a zeroed counter; state != null: the decode
+    // step ends here (next_top, position, step)
+    uint32_t* part_tok;
+    float* part_logit;
+    unsigned int* counter;
+    uint64_t* packed;
+    DecodeState* state;
+};
+int bf16_matvec(cudaStream_t stream, const Bf16Matvec& a);
+struct Bf16Gemm {
+    const void* x;       // [T, ldx] bf16, or f32 with x_f32
+    int x_f32, ldx, T, K;
+    const uint16_t* w;   // [rows, ldw] bf16
+    int rows, ldw;
+    void* out;           // [T, ldo] f32, or bf16 with out_bf16
+    int out_bf16, ldo;
+    const float* residual;  // [T, ldo] f32 or null; may be `out`
+    int silu_rows;
+};
+int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g);
+
+// ---- row operators of the layered decoders (layered_rows.cu) -----------------------------------------------------------
+int embed_rows(cudaStream_t stream, const uint16_t* table, const uint16_t* pos_table, int vocab, int dim, const uint32_t* tokens, int pos0, int T, float* x);
+// out[t] = x[row[t]] normed (row null: t); out_f32 selects the type of out
+int norm_rows(cudaStream_t stream, const float* x, int dim, const int* row, int T, const uint16_t* w, float offset, float eps, int out_f32, void* out, int ldo);
+int polynorm_rows(cudaStream_t stream, const void* z, int f32, int ldz, int n, int T, const uint16_t* coef, float eps, void* out, int ldo);
+int gated_rows(cudaStream_t stream, const float* o, int ldi, int n, int T, const uint16_t* norm_w, int head_len, float eps, const void* gate, int f32,
+               int ldg, int gate_act, void* out, int ldo);
+// rows of f32 -> bf16 or f32 at another pitch
+int convert_rows(cudaStream_t stream, const float* x, int ldi, int n, int T, int out_f32, void* out, int ldo);
+// table[p][i] = magnitude * (cos, sin)(p * freq[i]), evaluated in f64
+int rotation_table(cudaStream_t stream, const double* freqs, int half, int positions, double magnitude, float2* table);
+
+// ---- linear attention with a fixed decay per head (linear_attention.cu) ------------------------------------------------
+constexpr int kLinChunk = 64;  // tokens per chunk of the prompt form
+struct LinearAttnArgs {
+    const void* in;      // [T, ld]: q at q_off, k at k_off, v at v_off, head by head
+    int in_f32, ld, q_off, k_off, v_off;
+    int T, heads, dk, dv;
+    int rot;             // rotated entries of q and k (0 = none)
+    const float2* table; // [position][rot / 2]
+    const DecodeState* at;  // position of the first token: at->position, or pos0 when null
+    int pos0;
+    float key_scale;
+    const float* powers; // [heads][kLinChunk + 1]: decay^0 .. decay^kLinChunk
+    float* state;        // [heads, dk, dv] f32
+    float* out;          // [T, heads * dv] f32
+    float* scratch;      // linear_attention_scratch_floats()
+};
+size_t linear_attention_scratch_floats(int T, int heads, int dk, int dv);
+int linear_attention_recurrent(cudaStream_t stream, const LinearAttnArgs& a);  // token after token, f32 (decode; prompts in f32)
+int linear_attention_chunked(cudaStream_t stream, const LinearAttnArgs& a);    // bf16 q, k, v: chunks on the tensor cores
+bool linear_attention_chunked_ok(const LinearAttnArgs& a);
+
+// ---- latent attention (latent_attention.cu) ----------------------------------------------------------------------------
+struct LatentArgs {
+    const void* in;      // [T, ld]: q at q_off (per head: dim, then rot), the latent and the shared key part at dkv_off
+    int in_f32, ld, q_off, dkv_off;
+    int T, heads, dim, rot, vdim, rank, window;
+    float scale, eps;
+    const uint16_t* norm_w;  // [rank]
+    const uint16_t* uk;      // [heads * dim, ldu], W_uv follows: [heads * vdim, ldu]
+    const uint16_t* uv;
+    int ldu;
+    const float2* table;     // [position][rot / 2]
+    const DecodeState* at;
+    int pos0;
+    void* cache;             // [max_seq, pitch]: normed latent at 0, rotated key part at kr_off; f32 or bf16
+    int cache_f32, pitch, kr_off, max_seq;
+    float* out;              // [T, heads * vdim] f32
+    float* work;             // decode: latent_decode_work_floats()
+    unsigned int* counters;  // decode: [heads] zeros
+    void* expanded;          // prompt in bf16: keys and values of every visible position [rows, ldx]
+    int lde;
+    int first;               // first position held by `expanded`
+};
+int latent_write_cache(cudaStream_t stream, const LatentArgs& a);
+int latent_attention_plain(cudaStream_t stream, const LatentArgs& a);   // any size, f32 arithmetic, after latent_write_cache
+size_t latent_decode_work_floats(int heads, int rank, int rot, int span);
+bool latent_decode_ok(const LatentArgs& a);
+int latent_attention_decode(cudaStream_t stream, const LatentArgs& a);  // T = 1, bf16 cache; writes the cache row itself
+bool latent_prefill_ok(const LatentArgs& a);
+int latent_attention_prefill(cudaStream_t stream, const LatentArgs& a); // after latent_write_cache and the expansion
+
 // Deterministic merge of per-rank packed results: higher logit wins, ties -> lower token.
 int merge_packed_top1(cudaStream_t stream, const uint64_t* packed_all, int n, uint64_t* packed_out);
 

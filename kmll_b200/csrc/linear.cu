@@ -818,18 +818,6 @@ int w4_prepare(cudaStream_t stream, const uint8_t* pa, const uint16_t* sa, const
     return check_launch("w4g128_prepare");
 }
 
-// Opt a kernel in to all the dynamic shared memory a block can have (227 KB less the kernel's static part).  Set to the same
-// value at every launch, on whatever device is current: a CUDA graph replays its kernel nodes against the attribute the
-// function has at that time, so a value that followed the needs of the last captured launch would be too small for an
-// earlier node that needs more.
-template <typename K>
-static cudaError_t allow_all_dynamic_smem(K kernel) {
-    cudaFuncAttributes fa;
-    cudaError_t e = cudaFuncGetAttributes(&fa, kernel);
-    if (e != cudaSuccess) return e;
-    return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - (int)fa.sharedSizeBytes);
-}
-
 int launch_chain(cudaStream_t stream, ChainParams& cp) {
     if (cp.n_phases < 1 || cp.n_phases > kCMaxPhases) return fail(KMLL_ERR_SHAPE, "chain: %d phases", cp.n_phases);
     int kmax = 0, units_max = 0;
@@ -990,6 +978,12 @@ static int make_map_2d(CUtensorMap* map, CUtensorMapDataType type, int elem, con
     if (r != CUDA_SUCCESS) return fail(KMLL_ERR_CUDA, "cuTensorMapEncodeTiled failed (%d)", (int)r);
     return KMLL_OK;
 }
+
+}  // namespace kmll
+
+#include "linear_bf16.cuh"
+
+namespace kmll {
 
 static bool gemm_enabled() {
     static const bool on = [] {

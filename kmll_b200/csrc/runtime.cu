@@ -4,28 +4,13 @@
 // (crates/inference/src/model.rs:5151-5166, :6327-6384) built on this library's own C ABI operators:
 // every launch below goes through the same entry points an external host would bind.
 #include <dlfcn.h>
-#include <nccl.h>
-
 #include <cmath>
 #include <cstring>
 #include <vector>
 
-#include "../../include/kmll_b200_runtime.h"
-#include "internal.cuh"
+#include "decoder.cuh"
 
 namespace kmll {
-
-#define KMLL_TRY(expr)                 \
-    do {                               \
-        int rc__ = (expr);             \
-        if (rc__ != KMLL_OK) return rc__; \
-    } while (0)
-
-#define KMLL_CUDA(expr)                                                                        \
-    do {                                                                                       \
-        cudaError_t e__ = (expr);                                                              \
-        if (e__ != cudaSuccess) return fail(KMLL_ERR_CUDA, "%s: %s", #expr, cudaGetErrorString(e__)); \
-    } while (0)
 
 // ---- NCCL, loaded on first use (single-GPU users need no NCCL at all) ------------------------------
 struct NcclApi {
@@ -57,85 +42,6 @@ static NcclApi* nccl_api() {
         api.AllGather == nullptr)
         return nullptr;
     return &api;
-}
-
-struct QWeight {
-    void* w = nullptr;       // int8 values or packed nibbles
-    void* scales = nullptr;  // float[rows] or half[rows, cols/128]
-    int rows = 0, cols = 0;  // local (sharded) shape
-    uint8_t* prep = nullptr;  // W4-G128: the same values in the prepared layout the batch-1 kernels stream
-};
-
-struct Layer {
-    uint16_t* attention_norm = nullptr;
-    uint16_t* q_norm = nullptr;  // optional per-head RMSNorm weights [head_dim] of the query / key rows (null: the model has none)
-    uint16_t* k_norm = nullptr;
-    uint16_t* ffn_norm = nullptr;
-    QWeight wq, wk, wv, wo, w1, w3, w2;
-    uint8_t* w13_prep = nullptr;  // W4-G128: gate (w1) and up (w3) interleaved in the prepared layout
-    float* key_cache = nullptr;
-    float* value_cache = nullptr;
-};
-
-enum ShardKind { SHARD_NONE, SHARD_ROWS, SHARD_COLS };
-
-struct Decoder {
-    kmll_decoder_config cfg;
-    int device = 0;
-    int n_heads_l = 0, n_kv_l = 0, hidden_l = 0, vocab_l = 0;  // per-rank sizes
-    std::vector<Layer> layers;
-    uint16_t* final_norm = nullptr;
-    uint16_t* embedding = nullptr;
-    QWeight output;
-    float* freqs = nullptr;
-    // per-token scratch (crates/inference/src/model.rs:9339-9498 allocates the same set once)
-    float *hidden_a = nullptr, *hidden_b = nullptr, *hidden_mid = nullptr;
-    float *normed = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *q_rot = nullptr, *k_rot = nullptr;
-    float *attn = nullptr, *delta = nullptr, *gate = nullptr, *up = nullptr, *act = nullptr;
-    float* attn_ws = nullptr;
-    uint32_t* part_tok = nullptr;
-    float* part_logit = nullptr;
-    uint64_t* packed = nullptr;      // this rank's arg-max
-    uint64_t* packed_all = nullptr;  // [tp_size]
-    uint64_t* packed_final = nullptr;
-    DecodeState* state = nullptr;
-    uint64_t* history = nullptr;
-    int history_cap = 0;
-    uint64_t* pinned = nullptr;  // host, pinned
-    int host_position = 0;
-    bool have_next = false;
-    bool warmed = false;
-    cudaGraphExec_t graph = nullptr;
-    unsigned long long graph_trace_generation = 0;  // trace_generation() when `graph` was captured
-    cudaStream_t capture_stream = nullptr;  // the caller's stream may be the legacy default stream, which cannot capture
-    ncclComm_t comm = nullptr;
-    // peer-memory exchange (tensor parallel decode step); null = NCCL collectives
-    TpExchange* xc = nullptr;          // device copy of the tables
-    TpExchange xc_host;                // the same tables on the host (the chained kernel takes them by value)
-    void* xc_local = nullptr;          // this rank's exchange buffer (shared with the peers through CUDA IPC)
-    unsigned int* xc_epoch = nullptr;  // inside xc_local
-    void* xc_peer_base[kMaxTp] = {};   // peers' buffers as mapped here (null for the own rank)
-    std::vector<void*> allocs;
-    size_t weight_bytes = 0, kv_bytes = 0, resident_bytes = 0;  // resident = every device allocation of this decoder
-    int launches_per_step = 0;
-    bool weights_set = false;
-    // chained decode step (W4-G128, fused): prepared weights, exchange words also on a single GPU
-    bool chain = false;            // the decode step runs linear_chain_kernel
-    bool chain_split = true;       // ... one launch per projection (default) instead of one launch per layer (KMLL_CHAIN=layer)
-    bool chain_words = false;      // one GPU, one launch per projection: still hand the vectors over as exchange words (KMLL_CHAIN=words)
-    bool prepared_valid = false;   // the prepared buffers match the canonical tensors
-    unsigned int* top1_counter = nullptr;
-};
-
-template <typename T>
-static int dalloc(Decoder* d, T** out, size_t count) {
-    void* p = nullptr;
-    cudaError_t e = cudaMalloc(&p, count * sizeof(T) + 16);
-    if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "cudaMalloc(%zu bytes): %s", count * sizeof(T), cudaGetErrorString(e));
-    d->allocs.push_back(p);
-    d->resident_bytes += count * sizeof(T);
-    *out = static_cast<T*>(p);
-    return KMLL_OK;
 }
 
 static size_t qweight_bytes(int fmt, int rows, int cols, size_t* scale_bytes) {
@@ -565,6 +471,7 @@ static int enqueue_step_chain(Decoder* d, cudaStream_t s, int* launches) {
 }
 
 static int enqueue_step(Decoder* d, cudaStream_t s, int* launches) {
+    if (d->lay != nullptr) return layered_enqueue_step(d, s, launches);
     return d->chain ? enqueue_step_chain(d, s, launches) : enqueue_step_fused(d, s, launches);
 }
 
@@ -630,6 +537,16 @@ static int write_state(Decoder* d, cudaStream_t s, int position, int step, uint6
     return KMLL_OK;
 }
 
+// The arg-max in packed_final becomes the pending token of the sequence at d->host_position.
+static int publish_top(Decoder* d, cudaStream_t s) {
+    KMLL_CUDA(cudaMemcpyAsync(d->pinned, d->packed_final, 8, cudaMemcpyDeviceToHost, s));
+    KMLL_CUDA(cudaStreamSynchronize(s));
+    KMLL_TRY(write_state(d, s, d->host_position, 0, d->pinned[0]));
+    KMLL_CUDA(cudaStreamSynchronize(s));
+    d->have_next = true;
+    return KMLL_OK;
+}
+
 static int ensure_graph(Decoder* d, cudaStream_t s) {
     // a timeline buffer was attached or detached since the capture: the graph holds stale slot pointers
     if (d->graph != nullptr && d->graph_trace_generation != trace_generation()) {
@@ -647,7 +564,9 @@ static int ensure_graph(Decoder* d, cudaStream_t s) {
         KMLL_CUDA(cudaStreamSynchronize(s));
         KMLL_CUDA(cudaMemcpy(&saved, d->state, sizeof(saved), cudaMemcpyDeviceToHost));
         if (d->host_position >= d->cfg.max_seq_len) return fail(KMLL_ERR_CAPACITY, "sequence is full");
+        if (d->lay != nullptr) KMLL_TRY(layered_hold_state(d, s, false));  // (a recurrent state would count the token twice)
         KMLL_TRY(enqueue_step(d, s, &d->launches_per_step));
+        if (d->lay != nullptr) KMLL_TRY(layered_hold_state(d, s, true));
         KMLL_CUDA(cudaStreamSynchronize(s));
         KMLL_CUDA(cudaMemcpy(d->state, &saved, sizeof(saved), cudaMemcpyHostToDevice));
         d->warmed = true;
@@ -1055,6 +974,7 @@ int kmll_decoder_destroy(kmll_decoder_t dec) {
     if (d->xc_local) cudaFree(d->xc_local);
     for (void* p : d->allocs) cudaFree(p);
     if (d->pinned) cudaFreeHost(d->pinned);
+    layered_destroy(d);
     delete d;
     return KMLL_OK;
 }
@@ -1062,6 +982,7 @@ int kmll_decoder_destroy(kmll_decoder_t dec) {
 int kmll_decoder_init_random(kmll_decoder_t dec, uint64_t seed, float std, int tie_embeddings) {
     KMLL_REQUIRE_PTR(dec);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return layered_init_random(d, seed, std, tie_embeddings);
     const kmll_decoder_config& c = d->cfg;
     const int q_full = c.n_heads * c.head_dim;
     size_t max_elems = (size_t)c.vocab_size * c.dim;
@@ -1138,6 +1059,7 @@ int kmll_decoder_set_tensor(kmll_decoder_t dec, int layer, int tensor, const voi
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(values);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return layered_set_tensor(d, layer, tensor, values);
     TensorRef t;
     KMLL_TRY(tensor_ref(d, layer, tensor, &t));
     if (t.bf16 != nullptr) {
@@ -1170,6 +1092,7 @@ int kmll_decoder_set_tensor(kmll_decoder_t dec, int layer, int tensor, const voi
 int kmll_decoder_get_tensor(kmll_decoder_t dec, int layer, int tensor, void* values, void* scales) {
     KMLL_REQUIRE_PTR(dec);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return layered_get_tensor(d, layer, tensor, values);
     TensorRef t;
     KMLL_TRY(tensor_ref(d, layer, tensor, &t));
     KMLL_CUDA(cudaDeviceSynchronize());
@@ -1200,6 +1123,7 @@ int kmll_decoder_tp_init(kmll_decoder_t dec, const unsigned char id[128]) {
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(id);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return fail(KMLL_ERR_UNSUPPORTED, "a layered decoder runs on one GPU");
     if (d->cfg.tp_size == 1) return KMLL_OK;
     NcclApi* api = nccl_api();
     if (api == nullptr) return fail(KMLL_ERR_UNSUPPORTED, "libnccl.so.2 could not be loaded");
@@ -1219,6 +1143,7 @@ int kmll_decoder_prefill_token_loop(kmll_decoder_t dec, kmll_stream_t stream, co
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(tokens);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return fail(KMLL_ERR_UNSUPPORTED, "a layered decoder has no operator-by-operator step");
     cudaStream_t s = as_stream(stream);
     KMLL_REQUIRE(n_tokens > 0 && n_tokens <= d->cfg.max_seq_len, "prefill: prompt length %d outside 1..max_seq_len %d", n_tokens, d->cfg.max_seq_len);
     if (!d->weights_set) return fail(KMLL_ERR_STATE, "decoder has no weights");
@@ -1247,6 +1172,12 @@ int kmll_decoder_prefill(kmll_decoder_t dec, kmll_stream_t stream, const uint32_
     KMLL_REQUIRE(n > 0 && n <= c.max_seq_len, "prefill: prompt length %d outside 1..max_seq_len %d", n, c.max_seq_len);
     if (!d->weights_set) return fail(KMLL_ERR_STATE, "decoder has no weights");
     for (int i = 0; i < n; ++i) KMLL_REQUIRE(tokens[i] < (uint32_t)c.vocab_size, "prefill: token %u out of range", tokens[i]);
+    if (d->lay != nullptr) {
+        d->have_next = false;
+        KMLL_TRY(layered_reset(d, s));
+        KMLL_TRY(layered_forward(d, s, tokens, nullptr, n, nullptr, 0, nullptr, true));
+        return publish_top(d, s);
+    }
     const int q_len = d->n_heads_l * c.head_dim, kv_len = d->n_kv_l * c.head_dim;
     d->host_position = 0;
     d->have_next = false;
@@ -1360,6 +1291,7 @@ int kmll_decoder_generate_greedy(kmll_decoder_t dec, kmll_stream_t stream, int n
     KMLL_REQUIRE(n_steps >= 0 && n_steps <= d->history_cap, "generate: step count %d outside 0..%d", n_steps, d->history_cap);
     if (n_steps == 0) return KMLL_OK;
     std::vector<uint64_t> hist(n_steps);
+    if (d->lay != nullptr) KMLL_TRY(layered_save_state(d, s));  // a caller that generated too far rewinds to here cheaply
     if (d->cfg.fused) {
         // restart the history index, keep position and pending token
         KMLL_CUDA(cudaStreamSynchronize(s));
@@ -1432,6 +1364,50 @@ int kmll_decoder_step_host(kmll_decoder_t dec, kmll_stream_t stream, uint32_t to
     return KMLL_OK;
 }
 
+int kmll_decoder_reset(kmll_decoder_t dec, kmll_stream_t stream) {
+    KMLL_REQUIRE_PTR(dec);
+    Decoder* d = static_cast<Decoder*>(dec);
+    cudaStream_t s = as_stream(stream);
+    KMLL_CUDA(cudaStreamSynchronize(s));
+    if (d->lay != nullptr) KMLL_TRY(layered_reset(d, s));
+    d->host_position = 0;
+    d->have_next = false;
+    KMLL_TRY(write_state(d, s, 0, 0, 0));
+    KMLL_CUDA(cudaStreamSynchronize(s));
+    return KMLL_OK;
+}
+
+int kmll_decoder_extend(kmll_decoder_t dec, kmll_stream_t stream, const uint32_t* tokens, int n, const int* want, int n_want, float* logits) {
+    KMLL_REQUIRE_PTR(dec);
+    KMLL_REQUIRE_PTR(tokens);
+    Decoder* d = static_cast<Decoder*>(dec);
+    cudaStream_t s = as_stream(stream);
+    const kmll_decoder_config& c = d->cfg;
+    KMLL_REQUIRE(n > 0 && n_want >= 0, "extend: %d tokens, %d wanted", n, n_want);
+    if (n_want > 0) {
+        KMLL_REQUIRE_PTR(want);
+        KMLL_REQUIRE_PTR(logits);
+    }
+    if (!d->weights_set) return fail(KMLL_ERR_STATE, "decoder has no weights");
+    if (d->host_position + n > c.max_seq_len) return fail(KMLL_ERR_CAPACITY, "position %d exceeds max sequence length %d", d->host_position + n, c.max_seq_len);
+    for (int i = 0; i < n; ++i) KMLL_REQUIRE(tokens[i] < (uint32_t)c.vocab_size, "extend: token %u out of range", tokens[i]);
+    for (int i = 0; i < n_want; ++i)
+        KMLL_REQUIRE(want[i] >= 0 && want[i] < n && (i == 0 || want[i] > want[i - 1]), "extend: wanted places must ascend within the %d tokens", n);
+    if (d->lay != nullptr && (n > 1 || layered_tapped(d))) {
+        KMLL_TRY(layered_forward(d, s, tokens, nullptr, n, want, n_want, logits, true));
+        return publish_top(d, s);
+    }
+    // one token, or a decoder whose prompt path starts at position 0: decode steps
+    int w = 0;
+    for (int i = 0; i < n; ++i) {
+        uint64_t packed = 0;
+        KMLL_TRY(kmll_decoder_step_host(dec, stream, tokens[i], &packed));
+        if (w < n_want && want[w] == i) KMLL_TRY(kmll_decoder_next_logits(dec, stream, logits + (size_t)c.vocab_size * w++));
+    }
+    KMLL_CUDA(cudaStreamSynchronize(s));
+    return KMLL_OK;
+}
+
 int kmll_decoder_next_top(kmll_decoder_t dec, kmll_stream_t stream, uint64_t* packed_out) {
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(packed_out);
@@ -1451,6 +1427,7 @@ int kmll_decoder_rewind(kmll_decoder_t dec, kmll_stream_t stream, int position) 
     KMLL_REQUIRE(position >= 1 && position <= d->host_position, "rewind: position %d outside 1..%d", position, d->host_position);
     uint64_t packed = 0;
     KMLL_TRY(kmll_decoder_next_top(dec, stream, &packed));
+    if (d->lay != nullptr) KMLL_TRY(layered_rewind(d, s, position));
     KMLL_TRY(write_state(d, s, position, 0, packed));
     KMLL_CUDA(cudaStreamSynchronize(s));
     d->host_position = position;
@@ -1488,6 +1465,10 @@ int kmll_decoder_next_logits(kmll_decoder_t dec, kmll_stream_t stream, float* lo
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(logits_device);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) {
+        KMLL_CUDA(cudaMemcpyAsync(logits_device, layered_logits(d), sizeof(float) * d->cfg.vocab_size, cudaMemcpyDeviceToDevice, as_stream(stream)));
+        return KMLL_OK;
+    }
     const kmll_decoder_config& c = d->cfg;
     if (c.tp_size > 1) return fail(KMLL_ERR_UNSUPPORTED, "next_logits: a tensor-parallel decoder holds a slice of the vocabulary per rank");
     cudaStream_t s = as_stream(stream);
@@ -1505,6 +1486,7 @@ int kmll_decoder_set_rope_freqs(kmll_decoder_t dec, const float* freqs_host, int
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(freqs_host);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return fail(KMLL_ERR_UNSUPPORTED, "set_rope_freqs: a layered decoder takes kmll_layered_set_rotation");
     KMLL_REQUIRE(count == d->cfg.rotary_dim / 2, "set_rope_freqs: %d values given, rotary_dim / 2 = %d expected", count, d->cfg.rotary_dim / 2);
     for (int i = 0; i < count; ++i)
         if (!std::isfinite(freqs_host[i])) return fail(KMLL_ERR_SHAPE, "set_rope_freqs: value %d is not finite", i);
@@ -1532,6 +1514,7 @@ int kmll_batch_create(kmll_decoder_t dec, int batch, kmll_batch_t* out) {
     KMLL_REQUIRE_PTR(dec);
     KMLL_REQUIRE_PTR(out);
     Decoder* d = static_cast<Decoder*>(dec);
+    if (d->lay != nullptr) return fail(KMLL_ERR_UNSUPPORTED, "a layered decoder decodes one sequence at a time");
     const kmll_decoder_config& c = d->cfg;
     KMLL_REQUIRE(batch >= 1 && batch <= kMaxBatch, "batch %d outside 1..%d", batch, kMaxBatch);
     if (c.tp_size != 1) return fail(KMLL_ERR_UNSUPPORTED, "batched decode is single-GPU");

@@ -16,8 +16,14 @@ from .lib import KmllError, check, load
 
 FORMAT_RS_I8 = 0
 FORMAT_W4G128 = 1
+FORMAT_BF16 = 2  # layered decoders
 
 T_ATTENTION_NORM, T_WQ, T_WK, T_WV, T_WO, T_FFN_NORM, T_W1, T_W3, T_W2, T_FINAL_NORM, T_EMBEDDING, T_OUTPUT, T_Q_NORM, T_K_NORM = range(14)
+T_POSITION, T_GATE, T_MIX_NORM, T_DKV, T_DKV_NORM, T_UK, T_UV, T_ACT = range(14, 22)  # layered decoders
+MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION = 1, 2
+ACT_NONE, ACT_SILU, ACT_SIGMOID = range(3)
+MLP_NONE, MLP_POLYNORM = range(2)
+OUT_NORM_PER_HEAD, OUT_NORM_JOINT = range(2)
 
 
 class _Config(C.Structure):
@@ -195,6 +201,20 @@ class Decoder:
         check(self._lib.kmll_decoder_last_hidden(self._h, self._stream(), out.ctypes.data))
         return out
 
+    def extend(self, tokens, want=()) -> np.ndarray:
+        """The next tokens of the sequence (a portion of a prompt or decoded tokens); logits [len(want), vocab] of the places
+        in `want` (ascending offsets into `tokens`)."""
+        t = np.ascontiguousarray(tokens, dtype=np.uint32)
+        w = np.ascontiguousarray(want, dtype=np.int32)
+        out = torch.empty((max(1, w.size), self.cfg.vocab_size), dtype=torch.float32, device="cuda")
+        check(self._lib.kmll_decoder_extend(self._h, self._stream(), t.ctypes.data, int(t.size), w.ctypes.data if w.size else None, int(w.size),
+                                            out.data_ptr() if w.size else None))
+        return out[:w.size].cpu().numpy()
+
+    def reset(self) -> None:
+        """Forget the sequence; the next `extend` starts at position 0."""
+        check(self._lib.kmll_decoder_reset(self._h, self._stream()))
+
     @property
     def position(self) -> int:
         return int(self._lib.kmll_decoder_position(self._h))
@@ -215,6 +235,119 @@ class Decoder:
     def resident_bytes(self) -> int:
         """Bytes of every device allocation of the decoder (weights, KV cache, scratch)."""
         return int(self._lib.kmll_decoder_resident_bytes(self._h))
+
+
+class _LayerSpec(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("mixer", "heads", "dim", "vdim", "kv_rank", "rot_dim", "window")] + [("score_scale", C.c_float)] + \
+               [(n, C.c_int) for n in ("qkv_act", "gate_act", "out_norm")] + [("key_scale", C.c_float), ("mlp", C.c_int), ("ff", C.c_int)]
+
+
+class _LayeredConfig(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("n_layers", "dim", "vocab_size", "max_seq_len", "position_rows")] + \
+               [("norm_eps", C.c_float), ("norm_offset", C.c_float), ("compute_f32", C.c_int)]
+
+
+@dataclass
+class Rotation:
+    """Rotary positions: frequencies of the pairs (i, i + len(freqs)) and the factor on cos and sin."""
+    freqs: list
+    magnitude: float = 1.0
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a layered decoder (kmll_layer_spec); unused fields keep their defaults."""
+    mixer: int
+    heads: int
+    dim: int
+    vdim: int
+    kv_rank: int = 0
+    rot_dim: int = 0
+    window: int = 0
+    score_scale: float = 1.0
+    qkv_act: int = ACT_NONE
+    gate_act: int = ACT_SILU
+    out_norm: int = OUT_NORM_PER_HEAD
+    key_scale: float = 1.0
+    mlp: int = MLP_NONE
+    ff: int = 0
+    rotation: Rotation | None = None  # needed when rot_dim > 0
+    decay: list | None = None         # per head, linear attention
+
+    def _c(self) -> _LayerSpec:
+        return _LayerSpec(self.mixer, self.heads, self.dim, self.vdim, self.kv_rank, self.rot_dim, self.window, self.score_scale, self.qkv_act,
+                          self.gate_act, self.out_norm, self.key_scale, self.mlp, self.ff)
+
+
+@dataclass
+class LayeredConfig:
+    dim: int
+    vocab_size: int
+    layers: list
+    max_seq_len: int
+    position_rows: int = 0
+    norm_eps: float = 1.0e-5
+    norm_offset: float = 0.0  # 1.0: norm weights are stored around zero
+    compute_f32: bool = False
+
+    format = FORMAT_BF16
+
+    def _c(self) -> _LayeredConfig:
+        return _LayeredConfig(len(self.layers), self.dim, self.vocab_size, self.max_seq_len, self.position_rows, self.norm_eps, self.norm_offset,
+                              1 if self.compute_f32 else 0)
+
+    def tensor_shape(self, layer: int, tensor: int):
+        d, v = self.dim, self.vocab_size
+        if layer == -1:
+            return {T_EMBEDDING: (v, d), T_POSITION: (self.position_rows, d), T_FINAL_NORM: (d,), T_OUTPUT: (v, d)}[tensor]
+        s = self.layers[layer]
+        latent = s.mixer == MIXER_LATENT_ATTENTION
+        return {T_ATTENTION_NORM: (d,), T_FFN_NORM: (d,), T_WQ: (s.heads * (s.dim + (s.rot_dim if latent else 0)), d), T_WK: (s.heads * s.dim, d),
+                T_WV: (s.heads * s.vdim, d), T_GATE: (s.heads * s.vdim, d), T_MIX_NORM: (s.heads * s.vdim,), T_WO: (d, s.heads * s.vdim),
+                T_DKV: (s.kv_rank + s.rot_dim, d), T_DKV_NORM: (s.kv_rank,), T_UK: (s.heads * s.dim, s.kv_rank), T_UV: (s.heads * s.vdim, s.kv_rank),
+                T_W3: (s.ff, d), T_W2: (d, s.ff), T_ACT: (4,)}[tensor]
+
+
+class LayeredDecoder(Decoder):
+    """A decoder over a list of LayerSpec (kmll_layered_create): same handle, same calls, bf16 weights."""
+
+    def __init__(self, cfg: LayeredConfig):
+        self.cfg = cfg
+        self._lib = load()
+        self._h = C.c_void_p()
+        c = cfg._c()
+        specs = (_LayerSpec * len(cfg.layers))(*[s._c() for s in cfg.layers])
+        check(self._lib.kmll_layered_create(C.byref(c), specs, C.byref(self._h)))
+        for i, s in enumerate(cfg.layers):
+            if s.rot_dim > 0:
+                f = np.ascontiguousarray(s.rotation.freqs, dtype=np.float64)
+                check(self._lib.kmll_layered_set_rotation(self._h, i, f.ctypes.data, int(f.size), float(s.rotation.magnitude)))
+            if s.mixer == MIXER_LINEAR_ATTENTION:
+                d = np.ascontiguousarray(s.decay, dtype=np.float64)
+                check(self._lib.kmll_layered_set_decay(self._h, i, d.ctypes.data, int(d.size)))
+
+    def get_tensor(self, layer: int, tensor: int):
+        out = np.empty(self.cfg.tensor_shape(layer, tensor), dtype=np.uint16)
+        check(self._lib.kmll_decoder_get_tensor(self._h, layer, tensor, out.ctypes.data, None))
+        return out
+
+    def set_tensor(self, layer: int, tensor: int, values: np.ndarray, scales=None) -> None:
+        """bf16 bit patterns (uint16)."""
+        shape = self.cfg.tensor_shape(layer, tensor)
+        if values.dtype != np.uint16 or tuple(values.shape) != tuple(shape):
+            raise KmllError(-2, f"tensor {tensor} of layer {layer}: {values.dtype} {values.shape}, expected uint16 {shape}")
+        super().set_tensor(layer, tensor, values)
+
+    def layer_residuals(self, tokens) -> np.ndarray:
+        """Runs `tokens` as the next portion and returns the residual stream behind every layer [n_layers, n, dim]."""
+        n = len(tokens)
+        buf = torch.empty((len(self.cfg.layers), n, self.cfg.dim), dtype=torch.float32, device="cuda")
+        check(self._lib.kmll_layered_tap(self._h, buf.data_ptr()))
+        try:
+            self.extend(tokens)
+        finally:
+            check(self._lib.kmll_layered_tap(self._h, None))
+        return buf.cpu().numpy()
 
 
 class BatchDecoder:
@@ -268,4 +401,5 @@ def unpack_top1(packed: int):
     return int(token), float(logit)
 
 
-__all__ = ["Decoder", "BatchDecoder", "DecoderConfig", "KmllError", "FORMAT_RS_I8", "FORMAT_W4G128", "unpack_top1"]
+__all__ = ["Decoder", "LayeredDecoder", "BatchDecoder", "DecoderConfig", "LayeredConfig", "LayerSpec", "Rotation", "KmllError", "FORMAT_RS_I8",
+           "FORMAT_W4G128", "FORMAT_BF16", "unpack_top1"]

@@ -14,7 +14,7 @@ import torch
 
 from . import ops
 from .lib import KmllError, check
-from .runtime import FORMAT_W4G128, Decoder, unpack_top1
+from .runtime import FORMAT_BF16, FORMAT_W4G128, Decoder, unpack_top1
 
 DEFAULT_SEED = 0x9E3779B97F4A7C15  # SamplingOptions::default (inference.rs:353-360)
 F32_EPSILON = float(np.finfo(np.float32).eps)
@@ -121,6 +121,8 @@ class Session:
 
     # ---- TokenGenerationRuntime ----------------------------------------------------------------
     def backend(self) -> str:
+        if self.dec.cfg.format == FORMAT_BF16:
+            return "bf16-weights-f32" if self.dec.cfg.compute_f32 else "bf16"
         return "w4-g128" if self.dec.cfg.format == FORMAT_W4G128 else "rowwise-scaled-i8"
 
     def memory_stats(self) -> dict:
@@ -154,6 +156,22 @@ class Session:
         self.dec.prefill(np.asarray(prompt, dtype=np.int64))
         self._tokens = prompt
         self._ready = True
+
+    def extend(self, tokens, want=()) -> np.ndarray:
+        """The next portion of the sequence (from position 0 after `reset_sequence`); logits [len(want), vocab] of the places in
+        `want`, ascending offsets into `tokens`.  Generation continues from the last token."""
+        portion = [int(t) for t in tokens]
+        if not portion:
+            raise KmllError(-2, "a portion must not be empty")
+        if len(self._tokens) + len(portion) > self.max_seq_len:
+            raise KmllError(-2, f"sequence of {len(self._tokens) + len(portion)} tokens exceeds max_seq_len {self.max_seq_len}")
+        if not self._tokens:
+            self.dec.reset()
+        self._ready = False
+        logits = self.dec.extend(np.asarray(portion, dtype=np.int64), want)
+        self._tokens += portion
+        self._ready = True
+        return logits
 
     def _require_ready(self):
         if not self._ready:

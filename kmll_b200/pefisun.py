@@ -35,7 +35,7 @@ def rotation(cfg: dict) -> rt.Rotation:
     if s is None:
         return rt.Rotation(inverse_frequencies(int(cfg["dims"]), float(cfg["base"])))
     magnitude = 0.1 * math.log(float(s["factor"])) + 1.0
-    yarn = YarnRopeConfig(float(s["factor"]), int(s["original"]), float(s["fast"]), float(s["slow"]), magnitude)
+    yarn = YarnRopeConfig(float(s["factor"]), float(s["original"]), float(s["fast"]), float(s["slow"]), magnitude)
     return rt.Rotation(inverse_frequencies(int(cfg["dims"]), float(cfg["base"]), yarn), magnitude)
 
 

@@ -357,6 +357,50 @@ int kmll_argmax_f32_packed(kmll_stream_t stream, const float* logits, size_t n,
 int kmll_top_k_f32(kmll_stream_t stream, const float* logits, size_t n, int k, uint32_t* tokens,
                    float* values);
 
+/* ------------------------------------------------------------------------------------------
+ * Operators of the layered decoders (kmll_layered_create, kmll_b200_runtime.h); no counterpart in kmll.
+ * Weights are bf16 rows at a pitch of `pitch` elements (a multiple of 8, 16-byte aligned rows).
+ * ---------------------------------------------------------------------------------------- */
+/* y = W f(x) (+ residual), one row of x in f32.  What happens to x first:
+ *   kmll_linear_bf16           nothing, or RMSNorm x / rms(x) * (norm_offset + norm_weight) when norm_weight is given; output rows
+ *                              below silu_rows go through SiLU
+ *   kmll_polynorm_linear_bf16  a N(x) + b N(x^2) + c N(x^3) + e, coef = (a, b, c, e) bf16, N = division by the root mean square
+ *   kmll_gated_linear_bf16     x over its root mean square (all of x, times norm_weight; or per head_len entries when norm_weight
+ *                              is null) times silu (gate_sigmoid = 0) or sigmoid (1) of gate */
+int kmll_linear_bf16(kmll_stream_t stream, const float* x, const uint16_t* w, int pitch, int rows, int cols, const uint16_t* norm_weight, float norm_offset,
+                     float eps, const float* residual, int silu_rows, float* y);
+int kmll_polynorm_linear_bf16(kmll_stream_t stream, const float* x, const uint16_t* coef, float eps, const uint16_t* w, int pitch, int rows, int cols,
+                              const float* residual, float* y);
+int kmll_gated_linear_bf16(kmll_stream_t stream, const float* x, const uint16_t* norm_weight, int head_len, float eps, const float* gate, int gate_sigmoid,
+                           const uint16_t* w, int pitch, int rows, int cols, const float* residual, float* y);
+/* out[batch, rows] = x[batch, cols] W^T (+ residual f32 [batch, rows]): x_f32 = 0: x bf16 at pitch ldx (a multiple of 8), tensor
+ * cores, out f32 or (out_bf16) bf16; x_f32 = 1: f32 operands, f32 arithmetic on the CUDA cores. */
+int kmll_linear_batched_bf16(kmll_stream_t stream, const void* x, int x_f32, int ldx, int batch, const uint16_t* w, int pitch, int rows, int cols,
+                             const float* residual, void* out, int out_bf16);
+int kmll_polynorm_rows_bf16(kmll_stream_t stream, const uint16_t* x, int batch, int dim, const uint16_t* coef, float eps, uint16_t* out);
+/* Linear attention S <- decay S + k v^T, o = S^T q over `tokens` rows of `in` (pitch ld; q, k, v at their column offsets, head by
+ * head), from position `position` (or *position_device).  rot > 0: the first rot entries of q and k are rotated with
+ * table[position][rot / 2] = (cos, sin) pairs.  powers [heads][129] = decay^0 .. decay^128; state [heads, dk, dv] f32, updated.
+ * scratch == null: token after token in f32; else (bf16 input) chunks of 128 tokens on the tensor cores,
+ * kmll_linear_attention_scratch_floats() floats. */
+size_t kmll_linear_attention_scratch_floats(int tokens, int heads, int dk, int dv);
+int kmll_linear_attention(kmll_stream_t stream, const void* in, int in_f32, int ld, int q_off, int k_off, int v_off, int tokens, int heads, int dk, int dv,
+                          int rot, const float* table, int position, const int* position_device, float key_scale, const float* powers, float* state,
+                          float* scratch, float* out);
+/* Latent attention of one token over a bf16 cache [max_seq, pitch] (normed latent at column 0, rotated key part at the next
+ * multiple of 8): the row of the token at *position_device is written, then every position of the window is attended.  in =
+ * projected q (per head: dim, rot) and, behind it, the latent and the shared key part.  w_uk [heads*dim], w_uv [heads*vdim]
+ * rows of `rank` values at pitch w_pitch, w_uv directly behind w_uk. */
+size_t kmll_latent_attention_workspace_floats(int heads, int rank, int rot, int window, int max_seq);
+int kmll_latent_attention_decode(kmll_stream_t stream, const float* in, int heads, int dim, int rot, int vdim, int rank, int window, float scale, float eps,
+                                 const uint16_t* latent_norm, const uint16_t* w_uk_uv, int w_pitch, const float* table, const int* position_device,
+                                 uint16_t* cache, int pitch, int max_seq, float* workspace, float* out);
+/* The same for `tokens` prompt rows (bf16, pitch ld) from `position`; their cache rows must be in place, and `expanded` holds
+ * W_uk c | W_uv c (bf16, pitch lde) of every position from `first` on. */
+int kmll_latent_attention_prefill(kmll_stream_t stream, const uint16_t* in, int ld, int tokens, int position, int heads, int dim, int rot, int vdim, int rank,
+                                  int window, float scale, const float* table, const uint16_t* cache, int pitch, int max_seq, const uint16_t* expanded, int lde,
+                                  int first, float* out);
+
 #ifdef __cplusplus
 }
 #endif

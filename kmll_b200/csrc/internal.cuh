@@ -255,7 +255,7 @@ int convert_rows(cudaStream_t stream, const float* x, int ldi, int n, int T, int
 int rotation_table(cudaStream_t stream, const double* freqs, int half, int positions, double magnitude, float2* table);
 
 // ---- linear attention with a fixed decay per head (linear_attention.cu) ------------------------------------------------
-constexpr int kLinChunk = 64;  // tokens per chunk of the prompt form
+constexpr int kLinChunk = 128;  // tokens per chunk of the prompt form
 struct LinearAttnArgs {
     const void* in;      // [T, ld]: q at q_off, k at k_off, v at v_off, head by head
     int in_f32, ld, q_off, k_off, v_off;

@@ -116,9 +116,11 @@ __global__ void __launch_bounds__(kPlainWarps * 32) latent_plain_kernel(const La
 
 // ---- decode form ----------------------------------------------------------------------------------------------------------------
 // Widths: a cache row as staged in shared memory has kp = columns of (c, rotated part) rounded up to 32 for the score MMAs and
-// rp = rank rounded up to 128 for the value MMAs (eight warps of 16-column pairs); the tile is as wide as the larger.
-constexpr int kDT = 64;       // positions per tile
+// rp = rank rounded up to 256 for the value MMAs (16 warps of 16-column pairs); the tile is as wide as the larger.
+constexpr int kDT = 128;      // positions per tile
 constexpr int kDHeads = 16;   // heads per block = MMA rows
+constexpr int kDMaxSplit = 32;
+constexpr int kDWarps = 16;
 struct LatentDecodePlan {
     int kp, rp, width, nsplit, hgroups;
     size_t q_floats, part_floats;
@@ -128,13 +130,13 @@ LatentDecodePlan decode_plan(int heads, int rank, int rot, int span) {
     LatentDecodePlan p;
     const int kr = round_up(rank, 8);
     p.kp = round_up(kr + rot, 32);
-    p.rp = round_up(rank, 128);
+    p.rp = round_up(rank, 256);
     p.width = p.kp > p.rp ? p.kp : p.rp;
     p.hgroups = (heads + kDHeads - 1) / kDHeads;
-    p.nsplit = (span + kDT - 1) / kDT;
+    p.nsplit = (span + 15) / 16;  // a split of fewer than 16 positions would not fill a step of the value MMAs
     const int cap = p.hgroups >= 148 ? 1 : 148 / p.hgroups;
     if (p.nsplit > cap) p.nsplit = cap;
-    if (p.nsplit > 32) p.nsplit = 32;
+    if (p.nsplit > kDMaxSplit) p.nsplit = kDMaxSplit;
     if (p.nsplit < 1) p.nsplit = 1;
     p.q_floats = (size_t)p.hgroups * kDHeads * p.kp;
     p.part_floats = (size_t)p.nsplit * heads * (rank + 2);
@@ -146,13 +148,14 @@ __device__ inline DecodeRange decode_range(int pos, int window, int nsplit) {
     r.pos = pos;
     r.lo = window > 0 ? max(0, pos - window + 1) : 0;
     const int count = pos - r.lo + 1;
-    r.chunk = ((count + nsplit - 1) / nsplit + 15) & ~15;
+    r.chunk = max((count + nsplit - 1) / nsplit, 16);
     r.active = (count + r.chunk - 1) / r.chunk;
     return r;
 }
 
-// q folded through W_uk (times the score factor) and rotated, per head [kp]; the block behind the last head writes the cache row
-__global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentArgs a, float* __restrict__ q, int kp) {
+// q folded through W_uk (times the score factor) and rotated, per head as [kp] bf16 heads and, `lo` elements further on, [kp]
+// remainders; the block behind the last head writes the cache row
+__global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentArgs a, uint16_t* __restrict__ q, size_t lo, int kp) {
     extern __shared__ float asm_[];  // query [dim], then reduction [16][128]
     __shared__ float scratch[40];
     float* const sq = asm_;
@@ -166,8 +169,8 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentArgs a, 
         const int d = grp + i * 16;
         w[i] = (live && d < a.dim) ? ld_stream_u4(a.uk + (size_t)(h * a.dim + d) * a.ldu + r) : make_uint4(0u, 0u, 0u, 0u);
     }
+    const int pos = a.at->position, half = a.rot >> 1;  // (written more than one launch ago)
     pdl_wait();
-    const int pos = a.at->position, half = a.rot >> 1;
     if (h == a.heads) {
         if (blockIdx.y == 0 && pos < a.max_seq) write_row<true, false>(a, (size_t)a.dkv_off, pos, scratch);
         return;
@@ -192,34 +195,39 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentArgs a, 
 #pragma unroll
     for (int e = 0; e < 8; ++e) red[grp * 128 + c * 8 + e] = acc[e];
     __syncthreads();
-    float* const qrow = q + (size_t)h * kp;
+    uint16_t* const qrow = q + (size_t)h * kp;
+    auto put = [&](int col, float v) {
+        const uint16_t hi = f32_to_bf16_bits(v);
+        qrow[col] = hi;
+        qrow[lo + col] = f32_to_bf16_bits(v - bf16_bits_to_f32(hi));
+    };
     if (tid < 128) {
         const int col = blockIdx.y * 128 + tid;
         float s = 0.0f;
 #pragma unroll
         for (int g = 0; g < 16; ++g) s += red[g * 128 + tid];
-        if (col < a.rank) qrow[col] = s * a.scale;
+        if (col < a.rank) put(col, s * a.scale);
     }
     if (blockIdx.y == 0) {
         for (int i = tid; i < kp - a.rank; i += 256) {
             const int col = a.rank + i, j = col - a.kr_off;
             float v = 0.0f;
             if (j >= 0 && j < a.rot) v = rotated<true>(in, (size_t)a.dim, j, half, a.table + (size_t)pos * half) * a.scale;
-            qrow[col] = v;
+            put(col, v);
         }
     }
 }
 
-__global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, const float* __restrict__ q, float* __restrict__ part,
+__global__ void __launch_bounds__(kDWarps * 32) latent_decode_kernel(const LatentArgs a, const uint16_t* __restrict__ q, size_t lo, float* __restrict__ part,
                                                             const LatentDecodePlan pl) {
     extern __shared__ __align__(16) uint16_t dsm[];
     const int W = pl.width + 8;                 // tile row, elements
-    uint16_t* const tile = dsm;                 // [64][W]
+    uint16_t* const tile = dsm;                 // [kDT][W]
     uint16_t* const qh = tile + kDT * W;        // [16][W]
     uint16_t* const ql = qh + kDHeads * W;
-    uint16_t* const ph = ql + kDHeads * W;      // [16][72]
+    uint16_t* const ph = ql + kDHeads * W;      // [16][kDT + 8]
     uint16_t* const plo = ph + kDHeads * (kDT + 8);
-    float* const sc = reinterpret_cast<float*>(plo + kDHeads * (kDT + 8));  // [16][64]
+    float* const sc = reinterpret_cast<float*>(plo + kDHeads * (kDT + 8));  // [16][kDT]
     float* const corr = sc + kDHeads * kDT;     // [16]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
     const int split = blockIdx.x, h0 = blockIdx.y * kDHeads;
@@ -229,82 +237,90 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     const uint16_t* cache = static_cast<const uint16_t*>(a.cache);
     const int runs = a.pitch / 8, wruns = W / 8;
     const bool active = split < R.active;
-    auto load_tile = [&](int t0, int from, int to) {  // rows of positions [from, to) of the tile at t0
-        for (int i = tid; i < kDT * wruns; i += 256) {
-            const int r = i / wruns, c = i - r * wruns, p = t0 + r;
-            if (p >= from && p < to) {
-                const bool live = p < end && c < runs;
-                cp_async16_zfill_to((uint32_t)__cvta_generic_to_shared(tile + (size_t)r * W + c * 8), live ? cache + (size_t)p * a.pitch + c * 8 : cache,
-                                    live ? 16u : 0u);
-            }
+    auto load_tile = [&](int t0, int from, int to) {  // rows of positions [from, to) of the tile at t0; a warp per row
+        const int rows = min(kDT, (end - t0 + 15) & ~15);  // (what the value MMAs read; rows behind the last position are zeros)
+        for (int r = warp; r < rows; r += kDWarps) {
+            const int p = t0 + r;
+            if (p < from || p >= to) continue;
+            const uint16_t* src = cache + (size_t)(p < end ? p : t0) * a.pitch;
+            const uint32_t dst = (uint32_t)__cvta_generic_to_shared(tile + (size_t)r * W);
+            const int live = p < end ? runs : 0;
+            for (int c = lane; c < wruns; c += 32) cp_async16_zfill_to(dst + c * 16, c < live ? src + c * 8 : cache, c < live ? 16u : 0u);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (active) load_tile(begin, begin, R.pos);  // all but the newest row
     pdl_wait();
     if (!active) return;
-    load_tile(begin, max(begin, R.pos), begin + kDT);
-    for (int i = tid; i < kDHeads * W; i += 256) {
-        const int h = i / W, c = i - h * W;
-        const float x = (h0 + h < a.heads && c < pl.kp) ? q[(size_t)(h0 + h) * pl.kp + c] : 0.0f;
-        const uint16_t hi = f32_to_bf16_bits(x);
-        qh[i] = hi;
-        ql[i] = f32_to_bf16_bits(x - bf16_bits_to_f32(hi));
+    for (int r = warp; r < 2 * kDHeads; r += kDWarps) {  // query heads and remainders
+        const int h = r & (kDHeads - 1);
+        const bool live = h0 + h < a.heads;
+        const uint16_t* src = q + (r < kDHeads ? 0 : lo) + (size_t)(live ? h0 + h : 0) * pl.kp;
+        const uint32_t dst = (uint32_t)__cvta_generic_to_shared(qh + (size_t)r * W);
+        for (int c = lane; c < pl.kp / 8; c += 32) cp_async16_zfill_to(dst + c * 16, src + c * 8, live ? 16u : 0u);
     }
-    constexpr int MAXNB = 8;
-    const int nb = pl.rp / 64;  // 8-column blocks per warp (even)
+    load_tile(begin, max(begin, R.pos), begin + kDT);
+    constexpr int MAXNB = 4;
+    const int nb = pl.rp / (kDWarps * 8);  // 8-column blocks per warp (even)
     float o[MAXNB][4];
 #pragma unroll
     for (int i = 0; i < MAXNB; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
-    float m2[2] = {-INFINITY, -INFINITY}, l2[2] = {0.0f, 0.0f};  // heads 2 * warp, 2 * warp + 1
+    float m_run = -INFINITY, l_run = 0.0f;  // of head `warp`
     for (int t0 = begin; t0 < end; t0 += kDT) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        {   // scores: warp w, positions 8 w .. 8 w + 7
-            float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        const int live = min(kDT, end - t0);  // positions of this tile
+        for (int pb = warp * 8; pb < live; pb += kDWarps * 8) {  // scores: eight positions per warp and round
+            float s4[4][4] = {};  // four chains of MMAs
+#pragma unroll 2
             for (int k0 = 0; k0 < pl.kp; k0 += 32) {
                 uint32_t b[4], ah[4], al[4];
-                ldmatrix_x4(b, tile + (size_t)(warp * 8 + (lane & 7)) * W + k0 + (lane >> 3) * 8);
+                ldmatrix_x4(b, tile + (size_t)(pb + (lane & 7)) * W + k0 + (lane >> 3) * 8);
 #pragma unroll
                 for (int kk = 0; kk < 2; ++kk) {
                     const size_t ao = (size_t)(lane & 15) * W + k0 + kk * 16 + (lane >> 4) * 8;
                     ldmatrix_x4(ah, qh + ao);
                     ldmatrix_x4(al, ql + ao);
-                    mma_bf16(s, ah, b[2 * kk], b[2 * kk + 1]);
-                    mma_bf16(s, al, b[2 * kk], b[2 * kk + 1]);
+                    mma_bf16(s4[2 * kk], ah, b[2 * kk], b[2 * kk + 1]);
+                    mma_bf16(s4[2 * kk + 1], al, b[2 * kk], b[2 * kk + 1]);
                 }
             }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int h = g + (e >> 1) * 8, p = warp * 8 + 2 * tq + (e & 1);
-                sc[h * kDT + p] = t0 + p < end ? s[e] : -INFINITY;
-            }
+            for (int e = 0; e < 4; ++e)
+                sc[(g + (e >> 1) * 8) * kDT + pb + 2 * tq + (e & 1)] = (s4[0][e] + s4[1][e]) + (s4[2][e] + s4[3][e]);
         }
         __syncthreads();
+        {   // softmax: warp w, head w
+            float v[kDT / 32], mx = m_run, sum = 0.0f;
 #pragma unroll
-        for (int x = 0; x < 2; ++x) {  // softmax: warp w, heads 2 w and 2 w + 1
-            const int h = warp * 2 + x;
-            const float s0 = sc[h * kDT + lane], s1 = sc[h * kDT + 32 + lane];
-            const float mn = fmaxf(m2[x], warp_max(fmaxf(s0, s1)));  // (position t0 is always live, so mn is finite)
-            const float cf = expf(m2[x] - mn), p0 = expf(s0 - mn), p1 = expf(s1 - mn);
-            m2[x] = mn;
-            l2[x] = l2[x] * cf + warp_sum(p0 + p1);
-            const uint16_t b0 = f32_to_bf16_bits(p0), b1 = f32_to_bf16_bits(p1);
-            ph[h * (kDT + 8) + lane] = b0;
-            ph[h * (kDT + 8) + 32 + lane] = b1;
-            plo[h * (kDT + 8) + lane] = f32_to_bf16_bits(p0 - bf16_bits_to_f32(b0));
-            plo[h * (kDT + 8) + 32 + lane] = f32_to_bf16_bits(p1 - bf16_bits_to_f32(b1));
-            if (lane == 0) corr[h] = cf;
+            for (int i = 0; i < kDT / 32; ++i) {
+                v[i] = lane + 32 * i < live ? sc[warp * kDT + lane + 32 * i] : -INFINITY;
+                mx = fmaxf(mx, v[i]);
+            }
+            mx = warp_max(mx);  // (position t0 is always live, so it is finite)
+            const float cf = expf(m_run - mx);
+#pragma unroll
+            for (int i = 0; i < kDT / 32; ++i) {
+                const float w = expf(v[i] - mx);
+                sum += w;
+                const uint16_t hi = f32_to_bf16_bits(w);
+                ph[warp * (kDT + 8) + lane + 32 * i] = hi;
+                plo[warp * (kDT + 8) + lane + 32 * i] = f32_to_bf16_bits(w - bf16_bits_to_f32(hi));
+            }
+            m_run = mx;
+            l_run = l_run * cf + warp_sum(sum);
+            if (lane == 0) corr[warp] = cf;
         }
         __syncthreads();
-        {   // weighted latents: warp w, columns w * rp / 8 ..
+        {   // weighted latents: warp w, columns w * rp / 16 ..
             const float ca = corr[g], cb = corr[g + 8];
 #pragma unroll
             for (int i = 0; i < MAXNB; ++i) { o[i][0] *= ca; o[i][1] *= ca; o[i][2] *= cb; o[i][3] *= cb; }
 #pragma unroll
             for (int j = 0; j < kDT / 16; ++j) {
+                if (j * 16 >= live) break;
                 uint32_t ah[4], al[4], b[4];
                 const int ao = (lane & 15) * (kDT + 8) + j * 16 + (lane >> 4) * 8;
                 ldmatrix_x4(ah, ph + ao);
@@ -329,69 +345,113 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     for (int i = 0; i < MAXNB; ++i) {
         if (i >= nb) break;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int h = h0 + g + (e >> 1) * 8, c = warp * nb * 8 + i * 8 + 2 * tq + (e & 1);
-            if (h < a.heads && c < a.rank) base[(size_t)h * (a.rank + 2) + c] = o[i][e];
-        }
-    }
-    if (lane == 0)
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-            const int h = h0 + warp * 2 + x;
-            if (h < a.heads) {
-                base[(size_t)h * (a.rank + 2) + a.rank] = m2[x];
-                base[(size_t)h * (a.rank + 2) + a.rank + 1] = l2[x];
+        for (int e = 0; e < 4; e += 2) {
+            const int h = h0 + g + (e >> 1) * 8, c = warp * nb * 8 + i * 8 + 2 * tq;
+            if (h < a.heads && c < a.rank) {
+                float* p = base + (size_t)h * (a.rank + 2) + c;
+                if ((a.rank & 1) == 0) {
+                    *reinterpret_cast<float2*>(p) = make_float2(o[i][e], o[i][e + 1]);
+                } else {
+                    p[0] = o[i][e];
+                    if (c + 1 < a.rank) p[1] = o[i][e + 1];
+                }
             }
         }
+    }
+    if (lane == 0 && h0 + warp < a.heads) {
+        base[(size_t)(h0 + warp) * (a.rank + 2) + a.rank] = m_run;
+        base[(size_t)(h0 + warp) * (a.rank + 2) + a.rank + 1] = l_run;
+    }
 }
 
-// splits of a head merged, then W_uv: block (head, 32 values)
+// splits of a head merged, then W_uv: block (head, 64 values)
 __global__ void __launch_bounds__(256) latent_merge_kernel(const LatentArgs a, const float* __restrict__ part, int nsplit) {
-    extern __shared__ float msm[];  // weighted latent [rank rounded up to 8] | split factors [nsplit]
+    extern __shared__ float msm[];  // weighted latent [rank rounded up to 8] | split factors [kDMaxSplit]
     const int rp = round_up(a.rank, 8);
     float* const lat = msm;
     float* const f = msm + rp;
     const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    uint4 u[8][2];  // W_uv rows of this warp's eight values (rank <= 512), ahead of the dependency wait
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int v = blockIdx.y * 64 + warp + i * 8, r = lane * 8 + j * 256;
+            u[i][j] = (v < a.vdim && r < rp) ? ld_stream_u4(a.uv + (size_t)(h * a.vdim + v) * a.ldu + r) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    const DecodeRange R = decode_range(a.at->position, a.window, nsplit);  // (the position was written more than one launch ago)
     pdl_wait();
-    const DecodeRange R = decode_range(a.at->position, a.window, nsplit);
     const size_t hs = a.rank + 2, ss = (size_t)a.heads * hs;
     const float* p = part + (size_t)h * hs;
-    if (warp == 0) {
-        float mx = -INFINITY;
-        for (int s = lane; s < R.active; s += 32) mx = fmaxf(mx, p[s * ss + a.rank]);
-        mx = warp_max(mx);
-        float total = 0.0f;
-        for (int s = lane; s < R.active; s += 32) {
-            const float w = expf(p[s * ss + a.rank] - mx);
-            f[s] = w;
-            total += w * p[s * ss + a.rank + 1];
-        }
-        total = warp_sum(total);
-        for (int s = lane; s < R.active; s += 32) f[s] /= total;
-    }
-    __syncthreads();
-    for (int r = tid; r < rp; r += 256) {
-        float v = 0.0f;
-        if (r < a.rank)
-            for (int s = 0; s < R.active; ++s) v = fmaf(f[s], p[s * ss + r], v);
-        lat[r] = v;
-    }
-    __syncthreads();
-    for (int v = blockIdx.y * 32 + warp; v < min(a.vdim, ((int)blockIdx.y + 1) * 32); v += 8) {
-        const uint16_t* u = a.uv + (size_t)(h * a.vdim + v) * a.ldu;
-        float s = 0.0f;
-        for (int r = lane * 8; r < rp; r += 256) {
-            const uint4 t = *reinterpret_cast<const uint4*>(u + r);
-            const uint32_t w[4] = {t.x, t.y, t.z, t.w};
+    // the splits' weighted latents of columns 2 tid, 2 tid + 1 (or tid, tid + 256 for an odd rank)
+    float x[2][kDMaxSplit];
+    const bool even = (a.rank & 1) == 0;
+    const int c0 = even ? 2 * tid : tid, c1 = even ? 2 * tid + 1 : tid + 256;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                s = fmaf(__uint_as_float(w[e] << 16), lat[r + 2 * e], s);
-                s = fmaf(__uint_as_float(w[e] & 0xffff0000u), lat[r + 2 * e + 1], s);
+    for (int s = 0; s < kDMaxSplit; ++s) {
+        x[0][s] = x[1][s] = 0.0f;
+        if (s < R.active) {
+            if (even) {
+                if (c0 < a.rank) {
+                    const float2 t = *reinterpret_cast<const float2*>(p + s * ss + c0);
+                    x[0][s] = t.x;
+                    x[1][s] = t.y;
+                }
+            } else {
+                if (c0 < a.rank) x[0][s] = p[s * ss + c0];
+                if (c1 < a.rank) x[1][s] = p[s * ss + c1];
             }
         }
-        s = warp_sum(s);
-        if (lane == 0) a.out[(size_t)h * a.vdim + v] = s;
     }
+    if (warp == 0) {
+        const bool live = lane < R.active;
+        const float m = live ? p[lane * ss + a.rank] : -INFINITY, l = live ? p[lane * ss + a.rank + 1] : 0.0f;
+        const float mx = warp_max(m), w = live ? expf(m - mx) : 0.0f, total = warp_sum(w * l);
+        f[lane] = w / total;
+    }
+    __syncthreads();
+    {
+        float v0 = 0.0f, v1 = 0.0f;
+#pragma unroll
+        for (int s = 0; s < kDMaxSplit; ++s) {
+            v0 = fmaf(f[s], x[0][s], v0);
+            v1 = fmaf(f[s], x[1][s], v1);
+        }
+        if (c0 < rp) lat[c0] = v0;
+        if (c1 < rp) lat[c1] = v1;
+    }
+    __syncthreads();
+    float acc[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        acc[i] = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int r = lane * 8 + j * 256;
+            if (r < rp) {
+                const uint32_t w[4] = {u[i][j].x, u[i][j].y, u[i][j].z, u[i][j].w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    acc[i] = fmaf(__uint_as_float(w[e] << 16), lat[r + 2 * e], acc[i]);
+                    acc[i] = fmaf(__uint_as_float(w[e] & 0xffff0000u), lat[r + 2 * e + 1], acc[i]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int n = 4, off = 16; n >= 1; n >>= 1, off >>= 1) {  // eight sums over 32 lanes: lanes keep one half of them in each step
+        const bool up = (lane & off) != 0;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (i < n) {
+                const float keep = up ? acc[i + n] : acc[i], give = up ? acc[i] : acc[i + n];
+                acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+            }
+    }
+    acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 2);
+    acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
+    const int v = blockIdx.y * 64 + warp + (lane >> 2) * 8;
+    if ((lane & 3) == 0 && v < a.vdim) a.out[(size_t)h * a.vdim + v] = acc[0];
 }
 
 // ---- prompt form ------------------------------------------------------------------------------------------------------------------
@@ -419,12 +479,27 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a)
     // columns that no load writes stay zero
     for (int i = tid; i < (64 * PQ + 2 * BK * PQ + 2 * BK * PV) / 8; i += 128) reinterpret_cast<uint4*>(fsm)[i] = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();
-    for (int i = tid; i < 64 * (a.dim + a.rot); i += 128) {
-        const int r = i / (a.dim + a.rot), c = i - r * (a.dim + a.rot), row = r0 + r;
-        if (row < a.T) {
-            const size_t at = (size_t)row * a.ld + a.q_off + (size_t)h * (a.dim + a.rot);
-            if (c < a.dim) qs[r * PQ + c] = in[at + c];
-            else qs[r * PQ + ro + c - a.dim] = f32_to_bf16_bits(rotated<false>(in, at + a.dim, c - a.dim, half, a.table + (size_t)(pos0 + row) * half));
+    const int qw = a.dim + a.rot;
+    if (fast && ((a.ld | a.q_off) & 7) == 0) {  // one run of eight entries at a time
+        const int ru = a.dim >> 3;
+        for (int r = warp; r < 64 && r0 + r < a.T; r += 4) {
+            const uint16_t* row = in + (size_t)(r0 + r) * a.ld + a.q_off + (size_t)h * qw;
+            for (int c = lane; c < ru; c += 32) *reinterpret_cast<uint4*>(qs + r * PQ + c * 8) = *reinterpret_cast<const uint4*>(row + c * 8);
+        }
+    } else {
+        for (int i = tid; i < 64 * a.dim; i += 128) {
+            const int r = i / a.dim, c = i - r * a.dim;
+            if (r0 + r < a.T) qs[r * PQ + c] = in[(size_t)(r0 + r) * a.ld + a.q_off + (size_t)h * qw + c];
+        }
+    }
+    for (int r = warp; r < 64 && r0 + r < a.T; r += 4) {
+        const uint16_t* row = in + (size_t)(r0 + r) * a.ld + a.q_off + (size_t)h * qw + a.dim;
+        const float2* cs = a.table + (size_t)(pos0 + r0 + r) * half;
+        for (int j = lane; j < half; j += 32) {
+            const float u = bf16_bits_to_f32(row[j]), v = bf16_bits_to_f32(row[j + half]);
+            const float2 f = cs[j];
+            qs[r * PQ + ro + j] = f32_to_bf16_bits(u * f.x - v * f.y);
+            qs[r * PQ + ro + j + half] = f32_to_bf16_bits(v * f.x + u * f.y);
         }
     }
     auto load_tile = [&](int t0, int buf) {
@@ -432,8 +507,13 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a)
         uint16_t* const vt = vs + buf * BK * PV;
         if (fast) {
             const int ru = a.dim >> 3, rr = ru + (a.rot >> 3), rv = rr + (a.vdim >> 3);
-            for (int i = tid; i < BK * rv; i += 128) {
-                const int r = i / rv, c = i - r * rv, p = t0 + r;
+            const int dr = 128 / rv, dc = 128 - dr * rv;
+            for (int r = tid / rv, c = tid - r * rv; r < BK; r += dr, c += dc) {
+                if (c >= rv) {
+                    c -= rv;
+                    if (++r >= BK) break;
+                }
+                const int p = t0 + r;
                 const bool live = p <= last && p >= a.first;
                 const uint16_t* src;
                 uint16_t* dst;
@@ -605,13 +685,14 @@ bool latent_decode_ok(const LatentArgs& a) {
 int latent_attention_decode(cudaStream_t stream, const LatentArgs& a) {
     const int span = a.window > 0 && a.window < a.max_seq ? a.window : a.max_seq;
     const LatentDecodePlan p = decode_plan(a.heads, a.rank, a.rot, span);
-    float* const q = a.work;
+    uint16_t* const q = reinterpret_cast<uint16_t*>(a.work);
+    const size_t lo = p.q_floats;  // elements: the remainders fill the second half of the area
     float* const part = a.work + p.q_floats;
-    const size_t s1 = (size_t)(round_up(a.dim, 4) + 16 * 128) * 4, s3 = (size_t)(round_up(a.rank, 8) + p.nsplit) * 4;
-    cudaError_t e = launch(latent_absorb_kernel, dim3(a.heads + 1, (a.rank + 127) / 128), dim3(256), s1, stream, true, a, q, p.kp);
+    const size_t s1 = (size_t)(round_up(a.dim, 4) + 16 * 128) * 4, s3 = (size_t)(round_up(a.rank, 8) + kDMaxSplit) * 4;
+    cudaError_t e = launch(latent_absorb_kernel, dim3(a.heads + 1, (a.rank + 127) / 128), dim3(256), s1, stream, true, a, q, lo, p.kp);
     if (e == cudaSuccess) e = allow_all_dynamic_smem(latent_decode_kernel);
-    if (e == cudaSuccess) e = launch(latent_decode_kernel, dim3(p.nsplit, p.hgroups), dim3(256), decode_smem(p), stream, true, a, (const float*)q, part, p);
-    if (e == cudaSuccess) e = launch(latent_merge_kernel, dim3(a.heads, (a.vdim + 31) / 32), dim3(256), s3, stream, true, a, (const float*)part, p.nsplit);
+    if (e == cudaSuccess) e = launch(latent_decode_kernel, dim3(p.nsplit, p.hgroups), dim3(kDWarps * 32), decode_smem(p), stream, true, a, (const uint16_t*)q, lo, part, p);
+    if (e == cudaSuccess) e = launch(latent_merge_kernel, dim3(a.heads, (a.vdim + 63) / 64), dim3(256), s3, stream, true, a, (const float*)part, p.nsplit);
     if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "latent attention (decode): %s", cudaGetErrorString(e));
     return KMLL_OK;
 }

@@ -291,7 +291,7 @@ constexpr int kHEpiWarps = 8;
 constexpr int kHThreads = (2 + kHEpiWarps) * 32;  // warp 0: TMA, warp 1: MMA, warps 2..9: epilogue
 
 struct GemmBf16Params {
-    int rows, K, T, n_block, stages, row_tiles, tiles;
+    int rows, K, T, n_block, stages, row_tiles, x_tiles, tiles;
     void* out;
     int out_bf16, ldo, silu_rows;
     const float* residual;
@@ -337,7 +337,7 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
         if (lane == 0) {
             int it = 0;
             for (int tile = blockIdx.x; ok && tile < p.tiles; tile += gridDim.x) {
-                const int row0 = (tile % p.row_tiles) * kHRows, t0 = (tile / p.row_tiles) * p.n_block;
+                const int row0 = (tile / p.x_tiles) * kHRows, t0 = (tile % p.x_tiles) * p.n_block;
 #pragma unroll 1
                 for (int kt = 0; kt < KT; ++kt, ++it) {
                     const int s = it % stages, use = it / stages;
@@ -377,7 +377,7 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
         int n = 0;
         for (int tile = blockIdx.x; tile < p.tiles; tile += gridDim.x, ++n) {
             const int buf = n & 1;
-            const int row0 = (tile % p.row_tiles) * kHRows, t0 = (tile / p.row_tiles) * p.n_block;
+            const int row0 = (tile / p.x_tiles) * kHRows, t0 = (tile % p.x_tiles) * p.n_block;
             if (!mbar_wait<true>(&acc_full[buf], (uint32_t)(n >> 1) & 1u)) ok = false;
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
@@ -486,7 +486,8 @@ int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g) {
         if (best_cost < 0 || cost < best_cost) { best = nb; best_cost = cost; }
     }
     p.n_block = best;
-    const long long tiles = (long long)p.row_tiles * ((g.T + best - 1) / best);
+    p.x_tiles = (g.T + best - 1) / best;  // walked fastest: the blocks at work share their weight rows, and x stays in L2
+    const long long tiles = (long long)p.row_tiles * p.x_tiles;
     if (tiles > 0x3fffffff) return fail(KMLL_ERR_UNSUPPORTED, "bf16_gemm: too many tiles");
     p.tiles = (int)tiles;
     const size_t stage = (size_t)kHRows * 128 + (size_t)p.n_block * 128;

@@ -48,10 +48,11 @@ def main():
     ap.add_argument("--cols", type=int, default=4096)
     ap.add_argument("--mats", type=int, default=8)
     ap.add_argument("--reps", type=int, default=10)
-    ap.add_argument("--suite", default="", choices=["", "decode", "chain4096", "micro", "gemm_sweep"],
-                    help="decode: every batch-1 operator shape of a Mistral-7B-architecture step; chain4096: 4096x4096 matvec + residual + "
+    ap.add_argument("--suite", default="", choices=["", "decode", "chain4096", "micro", "gemm_sweep", "layered"],
+                    help="layered: the kernels of the layered decoders beside their like kernels, and whole decoders; decode: every batch-1 operator shape of a Mistral-7B-architecture step; chain4096: 4096x4096 matvec + residual + "
                          "RMSNorm in both formats; micro: RMSNorm / SwiGLU / RoPE / row softmax over B in {1,16,64}, bf16; gemm_sweep: "
                          "M in {1,16,64,256,2048} x four (N,K), W4-G128")
+    ap.add_argument("--only", default="", help="layered: only the lines of one part (matvec, mixer decode, gemm, mixer prompt, rows, decoder)")
     ap.add_argument("--shards", type=int, default=1, help="gemm_sweep: time one rank's share of every matrix when its N output rows are split over this "
                                                            "many GPUs (column-parallel: disjoint output blocks, no collective)")
     ap.add_argument("--profile", action="store_true", help="bracket one graph replay with cudaProfilerStart/Stop")
@@ -70,6 +71,8 @@ def main():
         return suite_micro(a.reps)
     if a.suite == "gemm_sweep":
         return suite_gemm_sweep(a.reps, shards=a.shards)
+    if a.suite == "layered":
+        return suite_layered(a.reps, only=a.only)
     run_one(a)
 
 
@@ -201,6 +204,202 @@ def suite_gemm_sweep(reps, cpu=None, shards=1):
                    cpu_us=cpu("gemm_w4", m=m, n=n, k=k) if cpu else None)
             del ws, calls
             torch.cuda.empty_cache()
+
+
+# ---- layered decoders ---------------------------------------------------------------------------------------------------
+# mixer sizes that resemble real layers of the given width
+LAYERED_SIZES = {4096: dict(ff=14336, lightning=(32, 128, 128), retention=(16, 256, 256), latent=dict(heads=32, dim=128, rot=64, vdim=128, rank=512)),
+                 2048: dict(ff=8192, lightning=(16, 128, 128), retention=(8, 256, 256), latent=dict(heads=16, dim=128, rot=64, vdim=128, rank=512))}
+LAYERED_WINDOW = 4096
+
+
+def layered_decoder(width, layers, max_seq_len, vocab=32000):
+    """Random-weight decoder whose layers cycle through lightning, latent attention and retention."""
+    from . import runtime as rt
+    from .pefisun import layered_config
+    z = LAYERED_SIZES[width]
+    la = z["latent"]
+
+    def layer(i):
+        kind = ("lightning", "latent_attention", "retention")[i % 3]
+        if kind == "latent_attention":
+            m = {"heads": la["heads"], "dim": la["dim"], "rot_dim": la["rot"], "vdim": la["vdim"], "kv_rank": la["rank"], "scale": (la["dim"] + la["rot"]) ** -0.5,
+                 "mask": {"size": LAYERED_WINDOW}, "rot": {"base": 1e4, "dims": la["rot"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        else:
+            h, dk, dv = z["lightning" if kind == "lightning" else "retention"]
+            m = {"heads": h, "dim": dk, "vdim": dv, "decay": [1.0 - 2.0 ** (-4 - 6 * j / h) for j in range(h)]}
+            if kind == "retention":
+                m["rot"] = {"base": 1e4, "dims": dk}
+        return {"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": z["ff"]}}
+
+    cfg = layered_config({"width": width, "vocab": vocab, "max_positions": max_seq_len, "norm": {"eps": 1e-5}, "layers": [layer(i) for i in range(layers)]})
+    dec = rt.LayeredDecoder(cfg)
+    dec.init_random(7, 0.02)
+    return dec
+
+
+def time_decoder(dec, prompt_len, steps, prefill_reps=3):
+    """(decode ms per token at context prompt_len, prefill ms): CUDA events, after warm-up."""
+    import numpy as np
+    prompt = np.random.default_rng(3).integers(0, dec.cfg.vocab_size, prompt_len)
+    dec.prefill(prompt)
+    dec.prefill(prompt)
+    e = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+    best = None
+    for _ in range(prefill_reps):
+        torch.cuda.synchronize()
+        e[0].record()
+        dec.prefill(prompt)
+        e[1].record()
+        torch.cuda.synchronize()
+        t = e[0].elapsed_time(e[1])
+        best = t if best is None else min(best, t)
+    dec.enqueue_steps(4)
+    torch.cuda.synchronize()
+    e[0].record()
+    dec.enqueue_steps(steps)
+    e[1].record()
+    torch.cuda.synchronize()
+    return e[0].elapsed_time(e[1]) / steps, best
+
+
+def suite_layered(reps, cpu=None, only="", context=2048):
+    """The kernels of the layered decoders beside the like kernels of the uniform decoder (RS-I8 and W4-G128 weights, f32 KV
+    cache) at equal sizes, then whole decoders of equal width and layer count: decode at context 2048, 2048-token prompt.
+    Inputs of a line together exceed L2.  frac_hbm / frac_tensor: of the copy bandwidth / bf16 peak."""
+    from . import runtime as rt
+    gen = torch.Generator(device="cuda").manual_seed(5)
+
+    def bf(*shape, std=1.0):
+        return (torch.randn(shape, generator=gen, device="cuda") * std).to(torch.bfloat16)
+
+    def want(name):
+        return not only or only in name
+
+    def copies(nbytes):
+        return max(2, min(48, int(300e6 // nbytes) + 1))
+
+    n = context
+    table = {r: torch.randn((n + 64, r // 2, 2), generator=gen, device="cuda") for r in (64, 256)}
+    pos = torch.tensor([n, 0, 0, 0], dtype=torch.int32, device="cuda")
+    for width, z in LAYERED_SIZES.items():
+        ff, la = z["ff"], z["latent"]
+        h, dk, dv = z["lightning"]
+        rh, rdk, rdv = z["retention"]
+        # ---- one row of x
+        coef = bf(4)
+        shapes = [("norm + stacked q k v gate", 2 * h * (dk + dv), width, "norm"), ("norm + up", ff, width, "norm"), ("polynorm + down", width, ff, "poly"),
+                  ("gate + output projection", width, h * dv, "gate"), ("norm + lm_head", 32000, width, "norm")]
+        for name, rows, cols, kind in shapes:
+            if not want("matvec"):
+                continue
+            ws = [bf(rows, cols, std=0.02) for _ in range(copies(rows * cols * 2))]
+            x, y, g, nw = torch.randn(cols, device="cuda"), torch.empty(rows, device="cuda"), torch.randn(cols, device="cuda"), bf(cols)
+            res = torch.randn(rows, device="cuda")
+            call = {"norm": lambda w: ops.linear_bf16(x, w, norm_weight=nw, norm_offset=1.0, eps=1e-5, out=y),
+                    "poly": lambda w: ops.polynorm_linear_bf16(x, coef, 1e-5, w, residual=res, out=y),
+                    "gate": lambda w: ops.gated_linear_bf16(x, g, w, 1e-5, head_len=dv, residual=res, out=y)}[kind]
+            us = time_graph([lambda w=w: call(w) for w in ws], reps)
+            report(f"matvec {name} {rows}x{cols} [bf16]", us, rows * cols * 2 + 4 * cols + 4 * rows)
+            del ws
+            for fmt in ("i8", "w4p"):
+                ws = [_weight(fmt, rows, cols) for _ in range(copies(rows * cols // 2))]
+                like = (lambda w: ops.linear_residual(x, w, res, out=y)) if kind != "norm" else (lambda w: ops.linear(x, w, out=y))
+                us = time_graph([lambda w=w: like(w) for w in ws], reps)
+                report(f"matvec {rows}x{cols} [{fmt}] (like kernel)", us, weight_bytes(fmt, rows, cols) + 4 * cols + 4 * rows)
+                del ws
+        # ---- mixers, one token
+        if want("mixer decode"):
+            for name, hh, d, v, rot in (("lightning", h, dk, dv, 0), ("retention", rh, rdk, rdv, rdk)):
+                sb = hh * d * v * 4
+                states = [torch.randn(hh * d * v, device="cuda") for _ in range(copies(2 * sb))]
+                pw = ops.decay_powers([1.0 - 2.0 ** (-4 - 6 * j / hh) for j in range(hh)])
+                x, out = torch.randn((1, 2 * hh * (d + v)), device="cuda") * 0.1, torch.empty((1, hh * v), device="cuda")
+                us = time_graph([lambda s=s: ops.linear_attention(x, hh, d, v, pw, s, pos, rot, table.get(rot), 0.1, None, out) for s in states], reps)
+                report(f"mixer decode {name} {hh}x{d}x{v}", us, 2 * sb + 4 * hh * (2 * d + 2 * v))
+                del states
+            H, D, R, V, K = la["heads"], la["dim"], la["rot"], la["vdim"], la["rank"]
+            caches = [bf(n + 64, K + R, std=0.5) for _ in range(48)]
+            wu = [bf(H * (D + V), K, std=0.05) for _ in range(copies(H * (D + V) * K * 2))]
+            x, out = torch.randn(H * (D + R) + K + R, device="cuda"), torch.empty(H * V, device="cuda")
+            ws = ops.latent_attention_workspace(H, K, R, LAYERED_WINDOW, n + 64)
+            lnorm = bf(K)
+            us = time_graph([lambda c=c, i=i: ops.latent_attention_decode(x, H, D, R, V, K, LAYERED_WINDOW, 0.07, 1e-5, lnorm, wu[i % len(wu)], table[R], pos, c, ws,
+                                                                          out) for i, c in enumerate(caches)], reps)
+            report(f"mixer decode latent attention (3 launches) {H} heads, context {n}", us, n * (K + R) * 2 + H * (D + V) * K * 2)
+            del caches, wu
+            ms, nq = n + 64, width // 128
+            nkv = nq // 4
+            q, wsp, o2 = torch.randn(nq * 128, device="cuda"), ops.single_query_attention_workspace(nq, 128, ms), torch.empty(nq * 128, device="cuda")
+            kv = [(torch.randn(ms * nkv * 128, device="cuda"), torch.randn(ms * nkv * 128, device="cuda")) for _ in range(24)]
+            us = time_graph([lambda c=c: ops.single_query_attention(q, c[0], c[1], n, ms, nq, nkv, 128, out=o2, workspace=wsp) for c in kv], reps)
+            report(f"decode attention {nq}/{nkv} heads x 128, f32 cache, context {n} (like kernel)", us, 2 * n * nkv * 128 * 4)
+            del kv
+        # ---- prompt
+        T = n
+        if want("gemm"):
+            for name, rows, cols in (("stacked q k v gate", 2 * h * (dk + dv), width), ("up", ff, width), ("down", width, ff), ("output projection", width, h * dv)):
+                ws = [bf(rows, cols, std=0.02) for _ in range(4)]
+                x, y = bf(T, cols), torch.empty((T, rows), dtype=torch.bfloat16, device="cuda")
+                us = time_graph([lambda w=w: ops.linear_batched_bf16(x, w, out=y) for w in ws], reps)
+                report(f"gemm {name} {T}x{rows}x{cols} [bf16]", us, 2 * (rows * cols + T * cols + T * rows), flops=2.0 * T * rows * cols)
+                del ws
+                for fmt in ("i8", "w4"):
+                    ws = [_weight(fmt, rows, cols) for _ in range(4)]
+                    xf, yf, sc = x.float(), torch.empty((T, rows), device="cuda"), ops.linear_batched_workspace(T, cols)
+                    us = time_graph([lambda w=w: ops.linear_batched(xf, w, T, cols, rows, out=yf, workspace=sc) for w in ws], reps)
+                    report(f"gemm {T}x{rows}x{cols} [{fmt}] (like kernel)", us, weight_bytes(fmt, rows, cols) + 4 * T * (rows + cols), flops=2.0 * T * rows * cols)
+                    del ws, xf, yf, sc
+                torch.cuda.empty_cache()
+        if want("mixer prompt"):
+            for name, hh, d, v, rot in (("lightning", h, dk, dv, 0), ("retention", rh, rdk, rdv, rdk)):
+                xs = [bf(T, 2 * hh * (d + v), std=0.2) for _ in range(4)]
+                pw = ops.decay_powers([1.0 - 2.0 ** (-4 - 6 * j / hh) for j in range(hh)])
+                st, out, sc = torch.zeros(hh * d * v, device="cuda"), torch.empty((T, hh * v), device="cuda"), ops.linear_attention_scratch(T, hh, d, v)
+                us = time_graph([lambda x=x: ops.linear_attention(x, hh, d, v, pw, st, 0, rot, table.get(rot), 0.1, sc, out) for x in xs], reps)
+                fl = 2.0 * hh * T * (2 * d * v + 32.5 * (d + v))  # state in and out, and on average 32.5 tokens of the chunk
+                report(f"mixer prompt {name} (3 launches) {T} tokens, {hh}x{d}x{v}", us, T * hh * (2 * d * 2 + v * 2 + v * 4), flops=fl)
+                del xs
+            H, D, R, V, K = la["heads"], la["dim"], la["rot"], la["vdim"], la["rank"]
+            x, cache, ex, out = bf(T, H * (D + R) + K + R), bf(T, K + R, std=0.5), bf(T, H * (D + V), std=0.5), torch.empty((T, H * V), device="cuda")
+            us = time_graph([lambda: ops.latent_attention_prefill(x, 0, H, D, R, V, K, LAYERED_WINDOW, 0.07, table[R], cache, ex, 0, out)] * 4, reps)
+            report(f"mixer prompt latent attention {T} tokens, {H} heads", us, T * (H * (D + R) + K + R + H * (D + V)) * 2 + T * H * V * 4, flops=1.0 * H * T * T * (D + R + V))
+        if want("rows"):
+            xs = [bf(T, ff) for _ in range(4)]
+            os_ = torch.empty_like(xs[0])
+            us = time_graph([lambda x=x: ops.polynorm_rows_bf16(x, coef, 1e-5, out=os_) for x in xs], reps)
+            report(f"rows polynorm [{T},{ff}] bf16", us, 4 * T * ff)
+            us = time_graph([lambda x=x: ops.softmax_rows(x, out=os_) for x in xs], reps) if ff <= 8192 else None
+            if us:
+                report(f"rows softmax [{T},{ff}] bf16 (like kernel)", us, 4 * T * ff)
+            del xs
+        torch.cuda.empty_cache()
+        # ---- whole decoders
+        if want("decoder"):
+            layers, hbm = 12, peak_hbm_gbs()[0]
+            dec = layered_decoder(width, layers, n + 256)
+            ms, pf = time_decoder(dec, n, max(16, reps))
+            wb = dec.weight_bytes - (32000 + n + 256) * width * 2
+            nst = sum(1 for i in range(layers) if i % 3 != 1)
+            sb = sum(2 * 4 * (h * dk * dv if i % 3 == 0 else rh * rdk * rdv) for i in range(layers) if i % 3 != 1)
+            cb = (layers - nst) * n * (la["rank"] + la["rot"]) * 2
+            print(json.dumps({"op": f"decoder layered {width} wide, {layers} layers", "decode_ms": round(ms, 4), "decode_tokens_per_s": round(1e3 / ms, 1),
+                              "launches_per_step": dec.launches_per_step, "step_frac_hbm": round((wb + sb + cb) / ms / 1e6 / hbm, 3), "prefill_ms": round(pf, 3),
+                              "prefill_tokens_per_s": round(n / pf * 1e3)}), flush=True)
+            dec.close()
+            heads = width // 128
+            for name, fmt in (("rs_i8", rt.FORMAT_RS_I8), ("w4g128", rt.FORMAT_W4G128)):
+                cfg = rt.DecoderConfig(n_layers=layers, dim=width, n_heads=heads, n_kv_heads=heads // 4, head_dim=128, hidden_dim=ff, vocab_size=32000, max_seq_len=n + 256,
+                                       rope_theta=1e6, norm_eps=1e-5, format=fmt)
+                dec = rt.Decoder(cfg)
+                dec.init_random(7, 0.02)
+                ms, pf = time_decoder(dec, n, max(16, reps))
+                wb = cfg.linear_elements() * (1 if fmt == rt.FORMAT_RS_I8 else 0.515625) + layers * 2 * n * (heads // 4) * 128 * 4
+                print(json.dumps({"op": f"decoder uniform {width} wide, {layers} layers, {name} (closest model)", "decode_ms": round(ms, 4),
+                                  "decode_tokens_per_s": round(1e3 / ms, 1), "launches_per_step": dec.launches_per_step, "step_frac_hbm": round(wb / ms / 1e6 / hbm, 3),
+                                  "prefill_ms": round(pf, 3), "prefill_tokens_per_s": round(n / pf * 1e3)}), flush=True)
+                dec.close()
+                torch.cuda.empty_cache()
 
 
 def run_decode_batch(a):

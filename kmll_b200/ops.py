@@ -561,3 +561,83 @@ def top_k_f32(logits, k: int):
     values = torch.zeros(k, dtype=torch.float32, device=logits.device)
     check(load().kmll_top_k_f32(_stream(), _p(_f32(logits, "logits")), logits.numel(), k, _p(tokens), _p(values)))
     return tokens, values
+
+
+# ---- operators of the layered decoders (bf16 weights [rows, cols], cols a multiple of 8) ------------------------------------
+def _pitch(w: torch.Tensor) -> int:
+    if w.dtype != torch.bfloat16 or w.dim() != 2 or w.shape[1] % 8:
+        raise KmllError(-2, "bf16 weights must be [rows, cols] with cols a multiple of 8")
+    return w.shape[1]
+
+
+def linear_bf16(x, w, norm_weight=None, norm_offset: float = 0.0, eps: float = 0.0, residual=None, silu_rows: int = 0, out=None):
+    out = torch.empty(w.shape[0], dtype=torch.float32, device=w.device) if out is None else out
+    check(load().kmll_linear_bf16(_stream(), _p(_f32(x, "x")), _p(w), _pitch(w), w.shape[0], w.shape[1], _p(norm_weight), norm_offset, eps, _p(residual),
+                                  silu_rows, _p(out)))
+    return out
+
+
+def polynorm_linear_bf16(x, coef, eps: float, w, residual=None, out=None):
+    out = torch.empty(w.shape[0], dtype=torch.float32, device=w.device) if out is None else out
+    check(load().kmll_polynorm_linear_bf16(_stream(), _p(_f32(x, "x")), _p(coef), eps, _p(w), _pitch(w), w.shape[0], w.shape[1], _p(residual), _p(out)))
+    return out
+
+
+def gated_linear_bf16(x, gate, w, eps: float, norm_weight=None, head_len: int = 0, sigmoid: bool = False, residual=None, out=None):
+    out = torch.empty(w.shape[0], dtype=torch.float32, device=w.device) if out is None else out
+    check(load().kmll_gated_linear_bf16(_stream(), _p(_f32(x, "x")), _p(norm_weight), head_len, eps, _p(_f32(gate, "gate")), 1 if sigmoid else 0, _p(w), _pitch(w),
+                                        w.shape[0], w.shape[1], _p(residual), _p(out)))
+    return out
+
+
+def linear_batched_bf16(x, w, residual=None, out=None, out_bf16: bool = False):
+    """x [batch, cols] bf16 (tensor cores) or f32 (CUDA cores, f32 throughout)."""
+    f32 = x.dtype == torch.float32
+    if out is None:
+        out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.bfloat16 if out_bf16 else torch.float32, device=w.device)
+    check(load().kmll_linear_batched_bf16(_stream(), _p(x), 1 if f32 else 0, x.shape[1], x.shape[0], _p(w), _pitch(w), w.shape[0], w.shape[1], _p(residual),
+                                          _p(out), 1 if out.dtype == torch.bfloat16 else 0))
+    return out
+
+
+def polynorm_rows_bf16(x, coef, eps: float, out=None):
+    out = torch.empty_like(x) if out is None else out
+    check(load().kmll_polynorm_rows_bf16(_stream(), _p(x), x.shape[0], x.shape[1], _p(coef), eps, _p(out)))
+    return out
+
+
+def decay_powers(decay, device="cuda") -> torch.Tensor:
+    """[heads, 129]: the powers 0 .. 128 of every head's decay."""
+    return torch.tensor([[float(d) ** i for i in range(129)] for d in decay], dtype=torch.float32, device=device)
+
+
+def linear_attention_scratch(tokens: int, heads: int, dk: int, dv: int, device="cuda") -> torch.Tensor:
+    return torch.empty(load().kmll_linear_attention_scratch_floats(tokens, heads, dk, dv), dtype=torch.float32, device=device)
+
+
+def linear_attention(qkv, heads: int, dk: int, dv: int, powers, state, position=0, rot: int = 0, table=None, key_scale: float = 1.0, scratch=None, out=None):
+    """qkv [tokens, ld]: q | k | v | ...; position: an int, or an int32 tensor on the device."""
+    tokens, ld = qkv.shape
+    out = torch.empty((tokens, heads * dv), dtype=torch.float32, device=qkv.device) if out is None else out
+    dev = isinstance(position, torch.Tensor)
+    check(load().kmll_linear_attention(_stream(), _p(qkv), 1 if qkv.dtype == torch.float32 else 0, ld, 0, heads * dk, 2 * heads * dk, tokens, heads, dk, dv, rot,
+                                       _p(table), 0 if dev else position, _p(position) if dev else None, key_scale, _p(powers), _p(state), _p(scratch), _p(out)))
+    return out
+
+
+def latent_attention_workspace(heads: int, rank: int, rot: int, window: int, max_seq: int, device="cuda") -> torch.Tensor:
+    return torch.empty(load().kmll_latent_attention_workspace_floats(heads, rank, rot, window, max_seq), dtype=torch.float32, device=device)
+
+
+def latent_attention_decode(x, heads, dim, rot, vdim, rank, window, scale, eps, latent_norm, w_uk_uv, table, position, cache, workspace, out=None):
+    out = torch.empty(heads * vdim, dtype=torch.float32, device=x.device) if out is None else out
+    check(load().kmll_latent_attention_decode(_stream(), _p(_f32(x, "x")), heads, dim, rot, vdim, rank, window, scale, eps, _p(latent_norm), _p(w_uk_uv),
+                                              _pitch(w_uk_uv), _p(table), _p(position), _p(cache), cache.shape[1], cache.shape[0], _p(workspace), _p(out)))
+    return out
+
+
+def latent_attention_prefill(x, position, heads, dim, rot, vdim, rank, window, scale, table, cache, expanded, first, out=None):
+    out = torch.empty((x.shape[0], heads * vdim), dtype=torch.float32, device=x.device) if out is None else out
+    check(load().kmll_latent_attention_prefill(_stream(), _p(x), x.shape[1], x.shape[0], position, heads, dim, rot, vdim, rank, window, scale, _p(table), _p(cache),
+                                               cache.shape[1], cache.shape[0], _p(expanded), expanded.shape[1], first, _p(out)))
+    return out

@@ -293,7 +293,7 @@ def test_far_keys_and_chunk_edges(cuda, dtype, kind):
     layer = retention(2, 16, 24, decay=decay, rot=2, base=1e9) if kind == "retention" else lightning(2, 24, 16, decay=decay)
     cfg, T = beacon(layer, 2.0)
     m = Model(cfg, dtype, tensors=T)
-    for distance in (1, 62, 63, 64, 65, 128, 300):
+    for distance in (1, 63, 64, 65, 127, 128, 129, 300):
         n = distance + 6
         tokens = placed(n, [4], [4 + distance])
         want = m.oracle(tokens)

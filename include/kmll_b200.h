@@ -374,9 +374,12 @@ int kmll_polynorm_linear_bf16(kmll_stream_t stream, const float* x, const uint16
 int kmll_gated_linear_bf16(kmll_stream_t stream, const float* x, const uint16_t* norm_weight, int head_len, float eps, const float* gate, int gate_sigmoid,
                            const uint16_t* w, int pitch, int rows, int cols, const float* residual, float* y);
 /* out[batch, rows] = x[batch, cols] W^T (+ residual f32 [batch, rows]): x_f32 = 0: x bf16 at pitch ldx (a multiple of 8), tensor
- * cores, out f32 or (out_bf16) bf16; x_f32 = 1: f32 operands, f32 arithmetic on the CUDA cores. */
+ * cores, out f32 or (out_bf16) bf16; x_f32 = 1: f32 operands, f32 arithmetic on the CUDA cores.  workspace (optional):
+ * kmll_linear_batched_bf16_workspace_bytes() bytes whose first 512 are zero before the first call (each call leaves them so);
+ * with it few rows of x are cut along K over more blocks. */
+size_t kmll_linear_batched_bf16_workspace_bytes(void);
 int kmll_linear_batched_bf16(kmll_stream_t stream, const void* x, int x_f32, int ldx, int batch, const uint16_t* w, int pitch, int rows, int cols,
-                             const float* residual, void* out, int out_bf16);
+                             const float* residual, void* workspace, void* out, int out_bf16);
 int kmll_polynorm_rows_bf16(kmll_stream_t stream, const uint16_t* x, int batch, int dim, const uint16_t* coef, float eps, uint16_t* out);
 /* Linear attention S <- decay S + k v^T, o = S^T q over `tokens` rows of `in` (pitch ld; q, k, v at their column offsets, head by
  * head), from position `position` (or *position_device).  rot > 0: the first rot entries of q and k are rotated with

@@ -239,7 +239,11 @@ struct Bf16Gemm {
     int out_bf16, ldo;
     const float* residual;  // [T, ldo] f32 or null; may be `out`
     int silu_rows;
+    float* partial;          // optional scratch of kGemmPartialFloats floats and
+    unsigned int* counters;  // 74 zeroed counters: up to kGemmSplitRows rows of x may be cut along K
 };
+constexpr int kGemmSplitRows = 256;
+constexpr size_t kGemmPartialFloats = (size_t)148 * 256 * 128;
 int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g);
 
 // ---- row operators of the layered decoders (layered_rows.cu) -----------------------------------------------------------

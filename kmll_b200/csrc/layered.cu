@@ -62,6 +62,8 @@ struct Layered {
     int rows = 0;
     std::vector<void*> row_allocs;
     float *x = nullptr, *o = nullptr, *lin = nullptr;
+    float* gemm_partial = nullptr;        // scratch of the projections over few rows
+    unsigned int* gemm_counters = nullptr;
     void *a = nullptr, *p = nullptr, *z = nullptr;
     int* want = nullptr;
     void* expanded = nullptr;
@@ -171,6 +173,11 @@ int create(Decoder* d, const kmll_layered_config& c, const kmll_layer_spec* spec
     KMLL_TRY(dalloc(d, &L->held, L->state_floats));
     KMLL_CUDA(cudaMemset(L->states, 0, L->state_floats * 4));
     d->kv_bytes += L->state_floats * 4;
+    if (!c.compute_f32) {
+        KMLL_TRY(dalloc(d, &L->gemm_partial, kGemmPartialFloats));
+        KMLL_TRY(dalloc(d, &L->gemm_counters, (size_t)74));
+        KMLL_CUDA(cudaMemset(L->gemm_counters, 0, 74 * 4));
+    }
     KMLL_TRY(dalloc(d, &L->logits, (size_t)c.vocab_size));
     KMLL_TRY(dalloc(d, &L->saved_logits, (size_t)c.vocab_size));
     KMLL_TRY(dalloc(d, &L->counter, (size_t)4));
@@ -312,6 +319,7 @@ int gemm(const Layered* L, cudaStream_t s, const void* x, int ldx, int T, const 
     g.w = w; g.rows = rows; g.ldw = ldw;
     g.out = out; g.out_bf16 = !(out_f32 || L->cfg.compute_f32); g.ldo = ldo;
     g.residual = residual; g.silu_rows = silu_rows;
+    g.partial = L->gemm_partial; g.counters = L->gemm_counters;
     return bf16_gemm(s, g);
 }
 

@@ -43,13 +43,19 @@ int kmll_gated_linear_bf16(kmll_stream_t s, const float* x, const uint16_t* norm
     return bf16_matvec(as_stream(s), v);
 }
 
+size_t kmll_linear_batched_bf16_workspace_bytes(void) { return 512 + kGemmPartialFloats * 4; }
+
 int kmll_linear_batched_bf16(kmll_stream_t s, const void* x, int x_f32, int ldx, int batch, const uint16_t* w, int pitch, int rows, int cols,
-                             const float* residual, void* out, int out_bf16) {
+                             const float* residual, void* workspace, void* out, int out_bf16) {
     KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(out);
     Bf16Gemm g;
     memset(&g, 0, sizeof(g));
     g.x = x; g.x_f32 = x_f32; g.ldx = ldx; g.T = batch; g.K = cols; g.w = w; g.rows = rows; g.ldw = pitch; g.out = out; g.out_bf16 = out_bf16; g.ldo = rows;
     g.residual = residual;
+    if (workspace != nullptr) {
+        g.counters = static_cast<unsigned int*>(workspace);
+        g.partial = static_cast<float*>(workspace) + 128;
+    }
     return bf16_gemm(as_stream(s), g);
 }
 

@@ -9,6 +9,8 @@
 
 #include <cuda.h>
 
+#include <algorithm>
+
 namespace kmll {
 
 // ---- one row of x -------------------------------------------------------------------------------------------------------
@@ -285,16 +287,19 @@ int bf16_matvec(cudaStream_t stream, const Bf16Matvec& a) {
 // N side, so a warp's stores of one row of x are 32 consecutive outputs.  Both operands come by TMA (128-byte swizzle, columns
 // beyond K zero-filled); persistent blocks walk the tiles, two accumulators in tensor memory let the epilogue of a tile
 // overlap the MMAs of the next.  Tensor maps cover this GPU's memory only, no multicast; every wait is bounded and a time-out
-// raises the device status word.
+// raises the device status word.  Few tiles with a long K are cut into K pieces, one block each; the block that arrives last adds
+// the partial tiles in the order of the pieces.
 constexpr int kHRows = 128, kHMaxN = 256, kHKT = 64;
 constexpr int kHEpiWarps = 8;
 constexpr int kHThreads = (2 + kHEpiWarps) * 32;  // warp 0: TMA, warp 1: MMA, warps 2..9: epilogue
 
 struct GemmBf16Params {
-    int rows, K, T, n_block, stages, row_tiles, x_tiles, tiles;
+    int rows, K, T, n_block, stages, row_tiles, x_tiles, tiles, ksplit;
     void* out;
     int out_bf16, ldo, silu_rows;
     const float* residual;
+    float* partial;          // ksplit > 1 (one item per block): [tiles][ksplit][n_block][128]
+    unsigned int* counters;  // [tiles], zero between launches
 };
 
 __host__ __device__ constexpr uint32_t gemm_idesc_bf16(int m, int n) {
@@ -312,8 +317,9 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
     uint64_t* acc_full = empty + stages;  // [2]
     uint64_t* acc_free = acc_full + 2;    // [2]
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_free + 2);
+    __shared__ unsigned int s_last;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int KT = (p.K + kHKT - 1) / kHKT;
+    const int KT = (p.K + kHKT - 1) / kHKT, kt_per = (KT + p.ksplit - 1) / p.ksplit, items = p.tiles * p.ksplit;
 
     if (tid == 0) {
         for (int s = 0; s < stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
@@ -336,10 +342,11 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
     if (warp == 0) {
         if (lane == 0) {
             int it = 0;
-            for (int tile = blockIdx.x; ok && tile < p.tiles; tile += gridDim.x) {
+            for (int item = blockIdx.x; ok && item < items; item += gridDim.x) {
+                const int tile = item / p.ksplit, kt0 = (item % p.ksplit) * kt_per, kt1 = min(kt0 + kt_per, KT);
                 const int row0 = (tile / p.x_tiles) * kHRows, t0 = (tile % p.x_tiles) * p.n_block;
 #pragma unroll 1
-                for (int kt = 0; kt < KT; ++kt, ++it) {
+                for (int kt = kt0; kt < kt1; ++kt, ++it) {
                     const int s = it % stages, use = it / stages;
                     if (use > 0 && !mbar_wait<false>(&empty[s], (uint32_t)(use - 1) & 1u)) { ok = false; break; }
                     const uint32_t st = smem_base + (uint32_t)s * stage_bytes;
@@ -352,20 +359,20 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
     } else if (warp == 1) {
         if (lane == 0) {
             int it = 0, n = 0;
-            for (int tile = blockIdx.x; ok && tile < p.tiles; tile += gridDim.x, ++n) {
-                const int buf = n & 1;
+            for (int item = blockIdx.x; ok && item < items; item += gridDim.x, ++n) {
+                const int buf = n & 1, kt0 = (item % p.ksplit) * kt_per, kt1 = min(kt0 + kt_per, KT);
                 if (n >= 2 && !mbar_wait<false>(&acc_free[buf], (uint32_t)((n >> 1) - 1) & 1u)) { ok = false; break; }
                 tcgen05_fence_after();
                 const uint32_t acc = tmem_base + (uint32_t)buf * 256u;
 #pragma unroll 1
-                for (int kt = 0; kt < KT; ++kt, ++it) {
+                for (int kt = kt0; kt < kt1; ++kt, ++it) {
                     const int s = it % stages, use = it / stages;
                     if (!mbar_wait<false>(&full[s], (uint32_t)use & 1u)) { ok = false; break; }
                     tcgen05_fence_after();
                     const uint32_t st = smem_base + (uint32_t)s * stage_bytes;
 #pragma unroll
                     for (int ks = 0; ks < kHKT / 16; ++ks)
-                        gemm_mma_f16(acc, gemm_smem_desc(st + ks * 32), gemm_smem_desc(st + a_bytes + ks * 32), idesc, (kt > 0 || ks > 0) ? 1u : 0u);
+                        gemm_mma_f16(acc, gemm_smem_desc(st + ks * 32), gemm_smem_desc(st + a_bytes + ks * 32), idesc, (kt > kt0 || ks > 0) ? 1u : 0u);
                     umma_commit(&empty[s]);
                 }
                 if (ok) umma_commit(&acc_full[buf]);
@@ -374,9 +381,17 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
     } else {
         const int q = warp & 3, half = (warp - 2) >> 2;  // lane quarter this warp may read; which half of the columns
         const int rl = q * 32 + lane;
+        auto finish = [&](int t, int row, float v, bool act) {
+            const size_t o = (size_t)t * p.ldo + row;
+            if (act) v = act_silu(v);
+            if (p.residual != nullptr) v += p.residual[o];
+            if (p.out_bf16) static_cast<uint16_t*>(p.out)[o] = f32_to_bf16_bits(v);
+            else static_cast<float*>(p.out)[o] = v;
+        };
         int n = 0;
-        for (int tile = blockIdx.x; tile < p.tiles; tile += gridDim.x, ++n) {
-            const int buf = n & 1;
+        for (int item = blockIdx.x; item < items; item += gridDim.x, ++n) {
+            const int buf = n & 1, tile = item / p.ksplit;
+            float* const part = p.ksplit > 1 ? p.partial + (size_t)item * p.n_block * kHRows : nullptr;
             const int row0 = (tile / p.x_tiles) * kHRows, t0 = (tile % p.x_tiles) * p.n_block;
             if (!mbar_wait<true>(&acc_full[buf], (uint32_t)(n >> 1) & 1u)) ok = false;
             ok = __all_sync(0xffffffffu, ok);
@@ -396,20 +411,42 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                    const int t = t0 + c0 + j;
-                    if (live && t < p.T) {
-                        const size_t o = (size_t)t * p.ldo + row;
-                        float v = __uint_as_float(d[j]);
-                        if (act) v = act_silu(v);
-                        if (p.residual != nullptr) v += p.residual[o];
-                        if (p.out_bf16) static_cast<uint16_t*>(p.out)[o] = f32_to_bf16_bits(v);
-                        else static_cast<float*>(p.out)[o] = v;
-                    }
+                    if (part != nullptr) part[(size_t)(c0 + j) * kHRows + rl] = __uint_as_float(d[j]);
+                    else if (live && t0 + c0 + j < p.T) finish(t0 + c0 + j, row, __uint_as_float(d[j]), act);
                 }
             }
             tcgen05_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&acc_free[buf]);
+            if (part != nullptr) {  // (this block's only item)
+                __threadfence();
+                asm volatile("bar.sync 1, %0;" ::"n"(kHEpiWarps * 32) : "memory");
+                if (tid == 64) s_last = atomicAdd(&p.counters[tile], 1u) == (unsigned)p.ksplit - 1u ? 1u : 0u;
+                asm volatile("bar.sync 1, %0;" ::"n"(kHEpiWarps * 32) : "memory");
+                if (s_last != 0u) {
+                    __threadfence();
+                    const float* base = p.partial + (size_t)tile * p.ksplit * p.n_block * kHRows;
+                    const int cols = min(p.n_block, p.T - t0);
+                    const size_t piece = (size_t)p.n_block * kHRows;
+                    for (int i = tid - 64; i < cols * (kHRows / 4); i += kHEpiWarps * 32) {
+                        const int r = (i & (kHRows / 4 - 1)) * 4, c = i / (kHRows / 4);
+                        const float* src = base + (size_t)c * kHRows + r;
+                        float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                        for (int z0 = 0; z0 < p.ksplit; z0 += 8) {  // eight pieces in flight
+                            float4 x[8];
+#pragma unroll
+                            for (int z = 0; z < 8; ++z)
+                                x[z] = z0 + z < p.ksplit ? __ldcg(reinterpret_cast<const float4*>(src + (size_t)(z0 + z) * piece)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+                            for (int z = 0; z < 8; ++z) { v[0] += x[z].x; v[1] += x[z].y; v[2] += x[z].z; v[3] += x[z].w; }
+                        }
+#pragma unroll
+                        for (int e = 0; e < 4; ++e)
+                            if (row0 + r + e < p.rows) finish(t0 + c, row0 + r + e, v[e], row0 + r + e < p.silu_rows);
+                    }
+                    if (tid == 64) p.counters[tile] = 0u;
+                }
+            }
         }
     }
     __syncwarp();
@@ -477,12 +514,12 @@ int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g) {
     p.rows = g.rows; p.K = g.K; p.T = g.T;
     p.out = g.out; p.out_bf16 = g.out_bf16; p.ldo = g.ldo; p.residual = g.residual; p.silu_rows = g.silu_rows;
     p.row_tiles = (g.rows + kHRows - 1) / kHRows;
-    // rows of x per tile: the size whose rounds over 148 SMs cost least (a round costs about its n_block columns)
+    // rows of x per tile: the size whose rounds over 148 SMs cost least (measured with K = 4096: 24 us at 64 rows, 32 at 256)
     const int nmax = g.T >= kHMaxN ? kHMaxN : (g.T + 15) / 16 * 16;
     int best = nmax;
     long long best_cost = -1;
     for (int nb = nmax; nb >= 64 || nb == nmax; nb -= 16) {
-        const long long tiles = (long long)p.row_tiles * ((g.T + nb - 1) / nb), cost = (tiles + 147) / 148 * (nb + 16);
+        const long long tiles = (long long)p.row_tiles * ((g.T + nb - 1) / nb), cost = (tiles + 147) / 148 * (600 + nb);
         if (best_cost < 0 || cost < best_cost) { best = nb; best_cost = cost; }
     }
     p.n_block = best;
@@ -490,6 +527,17 @@ int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g) {
     const long long tiles = (long long)p.row_tiles * p.x_tiles;
     if (tiles > 0x3fffffff) return fail(KMLL_ERR_UNSUPPORTED, "bf16_gemm: too many tiles");
     p.tiles = (int)tiles;
+    p.ksplit = 1;
+    if (g.partial != nullptr && g.T <= kGemmSplitRows && p.tiles <= 74) {  // at least eight k-tiles per piece
+        const int KT = (g.K + kHKT - 1) / kHKT;
+        const int want = std::min({148 / p.tiles, KT / 8, 16});
+        if (want > 1) {
+            const int per = (KT + want - 1) / want;
+            p.ksplit = (KT + per - 1) / per;  // (no empty piece)
+            p.partial = g.partial;
+            p.counters = g.counters;
+        }
+    }
     const size_t stage = (size_t)kHRows * 128 + (size_t)p.n_block * 128;
     p.stages = (int)((220 * 1024) / stage);
     if (p.stages > 8) p.stages = 8;
@@ -501,7 +549,7 @@ int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g) {
                             CU_TENSOR_MAP_SWIZZLE_128B));
     cudaError_t e = allow_all_dynamic_smem(linear_gemm_bf16_kernel);
     if (e == cudaSuccess)
-        e = launch(linear_gemm_bf16_kernel, dim3(p.tiles < 148 ? p.tiles : 148), dim3(kHThreads), smem, stream, true, p, map_w, map_x);
+        e = launch(linear_gemm_bf16_kernel, dim3(p.tiles * p.ksplit < 148 ? p.tiles * p.ksplit : 148), dim3(kHThreads), smem, stream, true, p, map_w, map_x);
     if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "linear_gemm_bf16: %s", cudaGetErrorString(e));
     return KMLL_OK;
 }

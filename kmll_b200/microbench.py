@@ -350,6 +350,18 @@ def suite_layered(reps, cpu=None, only="", context=2048):
                     us = time_graph([lambda w=w: ops.linear_batched(xf, w, T, cols, rows, out=yf, workspace=sc) for w in ws], reps)
                     report(f"gemm {T}x{rows}x{cols} [{fmt}] (like kernel)", us, weight_bytes(fmt, rows, cols) + 4 * T * (rows + cols), flops=2.0 * T * rows * cols)
                     del ws, xf, yf, sc
+                for m in (16, 64):  # short portions: a weight stream
+                    ws = [bf(rows, cols, std=0.02) for _ in range(copies(rows * cols * 2))]
+                    xm, ym, sc = bf(m, cols), torch.empty((m, rows), dtype=torch.bfloat16, device="cuda"), ops.linear_batched_bf16_workspace()
+                    us = time_graph([lambda w=w: ops.linear_batched_bf16(xm, w, out=ym, workspace=sc) for w in ws], reps)
+                    report(f"gemm {name} {m}x{rows}x{cols} [bf16]", us, 2 * (rows * cols + m * cols + m * rows), flops=2.0 * m * rows * cols)
+                    del ws
+                    for fmt in ("i8", "w4"):
+                        ws = [_weight(fmt, rows, cols) for _ in range(copies(rows * cols // 2))]
+                        xf, yf, sc = xm.float(), torch.empty((m, rows), device="cuda"), ops.linear_batched_workspace(m, cols)
+                        us = time_graph([lambda w=w: ops.linear_batched(xf, w, m, cols, rows, out=yf, workspace=sc) for w in ws], reps)
+                        report(f"gemm {m}x{rows}x{cols} [{fmt}] (like kernel)", us, weight_bytes(fmt, rows, cols) + 4 * m * (rows + cols), flops=2.0 * m * rows * cols)
+                        del ws, xf, yf, sc
                 torch.cuda.empty_cache()
         if want("mixer prompt"):
             for name, hh, d, v, rot in (("lightning", h, dk, dv, 0), ("retention", rh, rdk, rdv, rdk)):

@@ -590,13 +590,17 @@ def gated_linear_bf16(x, gate, w, eps: float, norm_weight=None, head_len: int = 
     return out
 
 
-def linear_batched_bf16(x, w, residual=None, out=None, out_bf16: bool = False):
+def linear_batched_bf16_workspace(device="cuda") -> torch.Tensor:
+    return torch.zeros(load().kmll_linear_batched_bf16_workspace_bytes() // 4, dtype=torch.float32, device=device)
+
+
+def linear_batched_bf16(x, w, residual=None, out=None, out_bf16: bool = False, workspace=None):
     """x [batch, cols] bf16 (tensor cores) or f32 (CUDA cores, f32 throughout)."""
     f32 = x.dtype == torch.float32
     if out is None:
         out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.bfloat16 if out_bf16 else torch.float32, device=w.device)
     check(load().kmll_linear_batched_bf16(_stream(), _p(x), 1 if f32 else 0, x.shape[1], x.shape[0], _p(w), _pitch(w), w.shape[0], w.shape[1], _p(residual),
-                                          _p(out), 1 if out.dtype == torch.bfloat16 else 0))
+                                          _p(workspace), _p(out), 1 if out.dtype == torch.bfloat16 else 0))
     return out
 
 

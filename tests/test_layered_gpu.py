@@ -449,3 +449,48 @@ def test_uniform_decoder_extends_by_decode_steps(cuda):
         ref.prefill(t[:n])
         np.testing.assert_allclose(row, ref.next_logits_to_host(), atol=2e-3)
     dec.close()
+
+
+# ---- operators through the C ABI --------------------------------------------------------------------------------------------
+def test_bf16_linear_operators(cuda):
+    import torch
+
+    from kmll_b200 import ops
+    gen = torch.Generator(device="cuda").manual_seed(9)
+
+    def randn(*shape):
+        return torch.randn(shape, generator=gen, device="cuda")
+
+    ws = ops.linear_batched_bf16_workspace()
+    for batch, rows, cols in ((1, 5, 8), (3, 130, 72), (17, 200, 520), (40, 1000, 2056), (64, 128, 4096), (256, 384, 1024), (300, 1300, 320), (700, 96, 64)):
+        w = (randn(rows, cols) / cols ** 0.5).bfloat16()
+        x, res = randn(batch, cols), randn(batch, rows)
+        want = x.bfloat16().double() @ w.double().T + res.double()
+        for workspace in (None, ws, ws):
+            got = ops.linear_batched_bf16(x.bfloat16(), w, residual=res, workspace=workspace)
+            assert float((got.double() - want).abs().max()) <= 2e-5 * cols ** 0.5, (batch, rows, cols)
+        got = ops.linear_batched_bf16(x.bfloat16(), w, out_bf16=True, workspace=ws)
+        assert float((got.double() - (want - res.double())).abs().max()) <= 0.03
+        want = x.double() @ w.double().T + res.double()
+        assert float((ops.linear_batched_bf16(x, w, residual=res).double() - want).abs().max()) <= 1e-5 * cols ** 0.5
+        norm = randn(cols).bfloat16()
+        xd, w0 = x[0].double(), w.double()
+        got = ops.linear_bf16(x[0].contiguous(), w, residual=res[0].contiguous())
+        assert float((got.double() - (w0 @ xd + res[0].double())).abs().max()) <= 1e-5 * cols ** 0.5
+        n = torch.from_numpy(lo.rms_norm_zero_centred(xd.cpu().numpy(), norm.double().cpu().numpy(), 1e-3)).cuda()
+        y = w0 @ n
+        y[:rows // 2] = y[:rows // 2] * torch.sigmoid(y[:rows // 2])
+        got = ops.linear_bf16(x[0].contiguous(), w, norm_weight=norm, norm_offset=1.0, eps=1e-3, silu_rows=rows // 2)
+        assert float((got.double() - y).abs().max()) <= 4e-5 * cols ** 0.5
+        coef = randn(4).bfloat16()
+        n = torch.from_numpy(lo.poly_norm(xd.cpu().numpy(), coef.double().cpu().numpy(), 1e-3)).cuda()
+        got = ops.polynorm_linear_bf16(x[0].contiguous(), coef, 1e-3, w)
+        assert float((got.double() - w0 @ n).abs().max()) <= 6e-5 * cols ** 0.5
+        gate = randn(cols)
+        o = xd.cpu().numpy()
+        n = lo.rms(o.reshape(-1, 8), 1e-3).reshape(-1) * lo.silu(gate.double().cpu().numpy())
+        got = ops.gated_linear_bf16(x[0].contiguous(), gate, w, 1e-3, head_len=8)
+        assert float((got.double() - w0 @ torch.from_numpy(n).cuda()).abs().max()) <= 4e-5 * cols ** 0.5
+        n = lo.rms_norm_plain(o, norm.double().cpu().numpy(), 1e-3) * lo.sigmoid(gate.double().cpu().numpy())
+        got = ops.gated_linear_bf16(x[0].contiguous(), gate, w, 1e-3, norm_weight=norm, sigmoid=True)
+        assert float((got.double() - w0 @ torch.from_numpy(n).cuda()).abs().max()) <= 4e-5 * cols ** 0.5

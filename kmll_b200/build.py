@@ -54,8 +54,10 @@ def build(force: bool = False, verbose: bool = False, ptxas_verbose: bool = Fals
         failed |= p.returncode != 0
     if failed:
         raise RuntimeError("nvcc failed; see output above")
-    link = [nvcc, "-shared", "-o", LIB, *objs, "-Xcompiler", "-fPIC", "-lcudart_static", "-ldl", "-lpthread", "-lrt"]
+    part = LIB + ".part"  # (an interrupted link leaves no half-written library behind)
+    link = [nvcc, "-shared", "-o", part, *objs, "-Xcompiler", "-fPIC", "-lcudart_static", "-ldl", "-lpthread", "-lrt"]
     subprocess.run(link, check=True)
+    os.replace(part, LIB)
     return LIB
 
 

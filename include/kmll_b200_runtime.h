@@ -56,7 +56,23 @@ enum {
     KMLL_T_DKV_NORM = 18,      /* latent attention: [kv_rank] */
     KMLL_T_UK = 19,            /* latent attention: latent -> keys [heads*dim, kv_rank] */
     KMLL_T_UV = 20,            /* latent attention: latent -> values [heads*vdim, kv_rank] */
-    KMLL_T_ACT = 21            /* PolyNorm coefficients a, b, c, e [4] */
+    KMLL_T_ACT = 21,           /* PolyNorm coefficients a, b, c, e [4] */
+    KMLL_T_ATTENTION_NORM_BIAS = 22, /* [dim], layer norms */
+    KMLL_T_FFN_NORM_BIAS = 23,
+    KMLL_T_FINAL_NORM_BIAS = 24,     /* (layer = -1) */
+    KMLL_T_EMBED_NORM = 25,          /* norm of the embedding [dim] (layer = -1) */
+    KMLL_T_EMBED_NORM_BIAS = 26,     /* (layer = -1) */
+    KMLL_T_DECAY_DOWN = 27,    /* gated linear attention: [decay_rank, dim] */
+    KMLL_T_DECAY_UP = 28,      /* [heads*dim_k, decay_rank] */
+    KMLL_T_DECAY_BIAS = 29,    /* [heads*dim_k] */
+    KMLL_T_DECAY_LOG = 30,     /* [heads], KMLL_DECAY_SOFTPLUS */
+    KMLL_T_BETA = 31,          /* delta rule: write strength [heads, dim] */
+    KMLL_T_Q_CONV = 32,        /* short convolutions [channels, conv], the current token's tap last */
+    KMLL_T_K_CONV = 33,
+    KMLL_T_V_CONV = 34,
+    KMLL_T_GATE_DOWN = 35,     /* low-rank output gate: [gate_rank, dim] */
+    KMLL_T_GATE_UP = 36,       /* [heads*vdim, gate_rank] */
+    KMLL_T_BESIDE = 64         /* added to a mixer's tensor id: that tensor of the layer's second mixer */
 };
 
 /* TextConfig of kmll (crates/inference/src/model.rs:271-366) reduced to what the decoder path uses. */
@@ -167,16 +183,30 @@ size_t kmll_decoder_resident_bytes(kmll_decoder_t dec);
 
 /* ---- layered decoders ----------------------------------------------------------------------------------------------
  * A decoder over a list of layer descriptions with bf16 weights: pre-norm layers (x += mixer(norm(x)), x += feed_forward(
- * norm(x))) whose mixers are latent attention or linear attention with a fixed decay per head, in any order and with sizes of
- * their own.  The handle is an ordinary kmll_decoder_t: prefill, generate_greedy, enqueue_steps, history, step_host, next_top,
- * set_pending, rewind, position, last_hidden, next_logits, set_tensor / get_tensor / init_random, the byte counts and destroy
- * work on it (rewind replays tokens from the nearest remembered state, since a recurrent state cannot be cut back).  No
- * counterpart in kmll.  Not for layered decoders: tensor parallelism, the lockstep batch, archives, prefill_token_loop. */
-enum { KMLL_MIXER_LATENT_ATTENTION = 1, KMLL_MIXER_LINEAR_ATTENTION = 2 };
-enum { KMLL_ACT_NONE = 0, KMLL_ACT_SILU = 1, KMLL_ACT_SIGMOID = 2 };
-enum { KMLL_MLP_NONE = 0, KMLL_MLP_POLYNORM = 1 };
-/* norm of a linear-attention output ahead of its gate */
-enum { KMLL_OUT_NORM_PER_HEAD = 0 /* each head over its own root mean square, no weight */, KMLL_OUT_NORM_JOINT = 1 /* all heads together, weighted */ };
+ * norm(x))) in any order and with sizes of their own.  The mixers are latent attention, grouped softmax attention, linear
+ * attention with a fixed decay per head, and linear attention with a decay per key channel and token (optionally with the delta
+ * rule); a layer may hold two of them side by side.  The handle is an ordinary kmll_decoder_t: prefill, generate_greedy,
+ * enqueue_steps, history, step_host, next_top, set_pending, rewind, position, last_hidden, next_logits, set_tensor / get_tensor /
+ * init_random, the byte counts and destroy work on it (rewind replays tokens from the nearest remembered state, since a recurrent
+ * state cannot be cut back).  No counterpart in kmll.  Not for layered decoders: tensor parallelism, the lockstep batch,
+ * archives, prefill_token_loop. */
+enum { KMLL_MIXER_NONE = 0, KMLL_MIXER_LATENT_ATTENTION = 1, KMLL_MIXER_LINEAR_ATTENTION = 2, KMLL_MIXER_ATTENTION = 3, KMLL_MIXER_GATED_LINEAR = 4 };
+enum { KMLL_ACT_NONE = 0, KMLL_ACT_SILU = 1, KMLL_ACT_SIGMOID = 2, KMLL_ACT_GELU_TANH = 3 };
+enum {
+    KMLL_MLP_NONE = 0,
+    KMLL_MLP_POLYNORM = 1, /* W_down polynorm(W_up h) */
+    KMLL_MLP_GATED = 2     /* W_down (mlp_act(W_gate h) * (W_up h)) */
+};
+enum { KMLL_NORM_RMS = 0, KMLL_NORM_LAYER = 1 /* mean taken off, weight and bias */ };
+/* norm of a mixer's output ahead of its gate */
+enum {
+    KMLL_OUT_NORM_PER_HEAD = 0,      /* each head over its own root mean square, no weight */
+    KMLL_OUT_NORM_JOINT = 1,         /* all heads together, weight [heads*vdim] */
+    KMLL_OUT_NORM_HEAD_WEIGHTED = 2, /* each head over its own root mean square, weight [vdim] shared by the heads */
+    KMLL_OUT_NORM_NONE = 3
+};
+/* decay of a key channel from z = W_up (W_down h) + bias */
+enum { KMLL_DECAY_LOGISTIC = 1 /* sigmoid(z)^(1 / decay_tau) */, KMLL_DECAY_SOFTPLUS = 2 /* exp(-exp(A_head) softplus(z)) */ };
 
 typedef struct {
     int mixer;       /* KMLL_MIXER_* */
@@ -187,7 +217,7 @@ typedef struct {
      * scores (q . W_uk c + q_rot . k_rot) * score_scale, values W_uv c */
     int kv_rank;
     int rot_dim;     /* even; 0 = no rotated part */
-    int window;      /* > 0: a position sees itself and the window - 1 positions before it; 0: every earlier position */
+    int window;      /* attention, > 0: a position sees itself and the window - 1 positions before it; 0: every earlier position */
     float score_scale;
     /* linear attention: S <- decay S + k v^T, o = S^T q; q, k, v through qkv_act, the first rot_dim entries of q and k rotated,
      * k times key_scale; o normed (out_norm), times gate_act(W_g h) */
@@ -195,7 +225,27 @@ typedef struct {
     int gate_act;    /* KMLL_ACT_SILU / KMLL_ACT_SIGMOID */
     int out_norm;    /* KMLL_OUT_NORM_* */
     float key_scale;
+    /* grouped attention: query head h uses key / value head h / (heads / kv_heads); no rotation */
+    int kv_heads;    /* divides heads; also for gated linear attention: heads of q and k */
+    int chunk;       /* > 0: a position sees the positions of its own chunk only (chunks counted from position 0) */
+    int head_gate;   /* 1: head i's output times gate_act(W_g h)_i, W_g [heads, dim] */
+    float out_scale; /* factor on the mixer's output (1 for none) */
+    /* gated linear attention: S <- diag(alpha) S + k u^T, o = S^T q, one decay alpha per key channel and token */
+    float q_scale;
+    int decay;       /* KMLL_DECAY_* */
+    float decay_tau;
+    int decay_rank;
+    int delta;       /* 0: u = v; 1: u = beta (v - (diag(alpha) S)^T k), beta = sigmoid(W_beta h) per head */
+    int conv;        /* taps of the causal convolution on q, k and v, followed by SiLU; 0: none */
+    float unit_eps;  /* > 0: q and k over sqrt(sum of squares + unit_eps) */
+    int gate_rank;   /* 0: gate W_g h, W_g [heads*vdim, dim]; > 0: W_gate_up (W_gate_down h) */
+} kmll_mixer_spec;
+
+typedef struct {
+    kmll_mixer_spec mixers[2]; /* the second: KMLL_MIXER_NONE, or a mixer beside the first that reads the same normed input; their
+                                  outputs, each times its out_scale, are added */
     int mlp;         /* KMLL_MLP_* */
+    int mlp_act;     /* KMLL_MLP_GATED: KMLL_ACT_SILU / KMLL_ACT_GELU_TANH */
     int ff;          /* feed-forward width */
 } kmll_layer_spec;
 
@@ -207,7 +257,12 @@ typedef struct {
     int position_rows; /* > 0: a learned position vector is added to the embedding (max_seq_len <= position_rows); 0: none */
     float norm_eps;
     float norm_offset; /* layer and final norms multiply by (norm_offset + w): 1 for weights stored around zero, else 0 */
-    int compute_f32;   /* 0: bf16 activations into the tensor-core projections of a prompt, bf16 latent cache; 1: f32 throughout */
+    int compute_f32;   /* 0: bf16 activations into the tensor-core projections of a prompt, bf16 caches; 1: f32 throughout */
+    int norm;          /* KMLL_NORM_*: layer, final and embedding norms */
+    float embed_scale; /* factor on the embedding (ahead of the position vector) */
+    int embed_norm;    /* 1: the embedding is normed */
+    float logit_scale;
+    int tie_output;    /* 1: the logits read the embedding table (no KMLL_T_OUTPUT) */
 } kmll_layered_config;
 
 size_t kmll_layer_spec_bytes(void);

@@ -193,6 +193,18 @@ class ModelWeights:
             raise CheckpointError(f"tensor {info.name} has shape {info.shape}, expected {tuple(shape)}")
         return f.read_tensor(info)
 
+    def shape(self, name: str) -> tuple:
+        return tuple(self.tensor(name)[1].shape)
+
+
+def load_layered(weights: ModelWeights, cfg, names):
+    """A layered decoder with the checkpoint's bf16 tensors; names = [(checkpoint name, layer or -1, tensor id)]."""
+    from . import runtime as rt
+    dec = rt.LayeredDecoder(cfg)
+    for name, layer, tensor in names:
+        dec.set_tensor(layer, tensor, weights.read(name, "BF16", cfg.tensor_shape(layer, tensor)))
+    return dec
+
 
 @dataclass
 class YarnRopeConfig:

@@ -448,20 +448,15 @@ __global__ void prepare_incremental_dyn_kernel(const float* __restrict__ q, cons
 
 __global__ void decode_begin_kernel(const uint16_t* __restrict__ table, int vocab, int dim, DecodeState* state,
                                     uint64_t* __restrict__ history, int history_cap, float* __restrict__ hidden,
-                                    unsigned int* exchange_epoch, const uint16_t* __restrict__ pos_table, uint32_t* token_log) {
+                                    unsigned int* exchange_epoch) {
     pdl_wait();
     const uint64_t packed = state->next_top;
     uint32_t token = (uint32_t)(packed & 0xffffffffull);
     if (token >= (uint32_t)vocab) token = (uint32_t)vocab - 1;
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < dim) {
-        float h = bf16_bits_to_f32(table[(size_t)token * dim + i]);
-        if (pos_table != nullptr) h += bf16_bits_to_f32(pos_table[(size_t)state->position * dim + i]);
-        hidden[i] = h;
-    }
+    if (i < dim) hidden[i] = bf16_bits_to_f32(table[(size_t)token * dim + i]);
     if (i == 0) {
         const int step = state->step;
-        if (token_log != nullptr) token_log[state->position] = token;
         if (step < history_cap) history[step] = packed;
         state->seq_len = state->position + 1;
         if (exchange_epoch != nullptr) *exchange_epoch += 1u;  // numbers the peer-memory exchanges of this step
@@ -519,9 +514,9 @@ int write_kv_row(cudaStream_t stream, const float* x, int position, int token_le
 }
 
 int decode_begin(cudaStream_t stream, const uint16_t* table, int vocab, int dim, DecodeState* state, uint64_t* history,
-                 int history_cap, float* hidden, unsigned int* exchange_epoch, const uint16_t* pos_table, uint32_t* token_log) {
+                 int history_cap, float* hidden, unsigned int* exchange_epoch) {
     cudaError_t e = launch(decode_begin_kernel, dim3((dim + 255) / 256), dim3(256), 0, stream, true, table, vocab, dim, state,
-                           history, history_cap, hidden, exchange_epoch, pos_table, token_log);
+                           history, history_cap, hidden, exchange_epoch);
     if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "decode_begin: %s", cudaGetErrorString(e));
     return KMLL_OK;
 }

@@ -165,11 +165,10 @@ int prepare_prefill_offset(cudaStream_t stream, const float* q, const float* k, 
 int write_kv_row(cudaStream_t stream, const float* x, int position, int token_len, int head_dim, float* cache, int kv_bf16);
 int prefill_attention_launch(cudaStream_t stream, const float* q_batch, const float* k_cache, const float* v_cache, int prompt_len,
                              int n_heads, int n_kv_heads, int head_dim, float* out, int kv_bf16, int window, int tensor_cores);
-// hidden = embedding[state->next_top.token] (+ pos_table[position]); token_log[position] = token; also records next_top into history[state->step] and
+// hidden = embedding[state->next_top.token]; also records next_top into history[state->step] and
 // sets seq_len = position + 1.
 int decode_begin(cudaStream_t stream, const uint16_t* table, int vocab, int dim, DecodeState* state, uint64_t* history,
-                 int history_cap, float* hidden, unsigned int* exchange_epoch = nullptr, const uint16_t* pos_table = nullptr,
-                 uint32_t* token_log = nullptr);
+                 int history_cap, float* hidden, unsigned int* exchange_epoch = nullptr);
 // state->next_top = *packed; position += 1; step += 1.
 int decode_end(cudaStream_t stream, const uint64_t* packed, DecodeState* state);
 
@@ -202,25 +201,45 @@ int linear_batched_form(int form, cudaStream_t stream, int fmt, const float* x, 
                         const float* residual, void* workspace = nullptr, float* gate_tmp = nullptr, float* up_tmp = nullptr);
 size_t linear_batched_workspace_bytes(int batch, int in_dim);
 // ---- bf16 weights (linear_bf16.cuh) ------------------------------------------------------------------------------------
+// Norm of a vector: x / rms(x) * (offset + w), or (kind KMLL_NORM_LAYER) (x - mean) / sqrt(variance + eps) * (offset + w) + b.
+struct NormArgs {
+    int kind;
+    const uint16_t* w;
+    const uint16_t* b;   // KMLL_NORM_LAYER
+    float offset, eps;
+};
+// One mixer's output inside the vector that its layer's output projection reads: columns [begin, begin + cols), normed per
+// `norm` (KMLL_OUT_NORM_*; heads of head_len), times act(gate), times scale.  Entry i takes gate value i / gate_len.
+struct GateSegment {
+    int begin, cols, head_len;
+    int norm;
+    const uint16_t* norm_w;  // JOINT: [cols]; HEAD_WEIGHTED: [head_len]
+    const void* gate;        // null: no gate
+    int gate_len, act;
+    float scale, eps;
+};
+constexpr int kMaxSegments = 2;
 // What happens to the vector x ahead of a projection:
-//   PRO_RMSNORM   x / rms(x) * (norm_offset + norm_w)
+//   PRO_NORM      `norm`
 //   PRO_POLYNORM  a N(x) + b N(x^2) + c N(x^3) + e with coef = (a, b, c, e), N = division by the root mean square
-//   PRO_GATED     x / rms (over all of x times norm_w, or per head_len entries when norm_w is null) * gate_act(gate)
-enum { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_POLYNORM = 2, PRO_GATED = 3 };
+//   PRO_GATED     `seg`: the normed, gated and scaled outputs of the mixers; columns outside every segment are zeros
+enum { PRO_PLAIN = 0, PRO_NORM = 1, PRO_POLYNORM = 2, PRO_GATED = 3 };
 constexpr int kMatvecMaxBlocks = 4096;  // partial arg-max entries a caller provides
 struct Bf16Matvec {
     const uint16_t* w;   // [rows, ldw] bf16
     int rows, K, ldw;
     const float* x;      // [K]
     int pro;
-    float eps, norm_offset;
-    const uint16_t* norm_w;
+    float eps;           // PRO_POLYNORM
+    NormArgs norm;
     const uint16_t* coef;
-    const float* gate;
-    int gate_act, head_len;
+    GateSegment seg[kMaxSegments];
+    int n_seg;
     float* y;            // [rows]
     const float* residual;
     int silu_rows;       // rows below this index go through SiLU
+    int pair_act;        // not 0: rows 2 i and 2 i + 1 are a gate and its value, y[i] = act(gate) * value
+    float out_scale;     // factor on every result (ahead of the residual)
     // arg-max over the rows (packed != null): partials of kMatvecMaxBlocks entries, a zeroed counter; state != null: the decode
     // step ends here (next_top, position, step)
     uint32_t* part_tok;
@@ -239,6 +258,8 @@ struct Bf16Gemm {
     int out_bf16, ldo;
     const float* residual;  // [T, ldo] f32 or null; may be `out`
     int silu_rows;
+    int pair_act;            // as in Bf16Matvec: out is [T, rows / 2]
+    float out_scale;
     float* partial;          // optional scratch of kGemmPartialFloats floats and
     unsigned int* counters;  // 74 zeroed counters: up to kGemmSplitRows rows of x may be cut along K
 };
@@ -247,14 +268,28 @@ constexpr size_t kGemmPartialFloats = (size_t)148 * 256 * 128;
 int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g);
 
 // ---- row operators of the layered decoders (layered_rows.cu) -----------------------------------------------------------
-int embed_rows(cudaStream_t stream, const uint16_t* table, const uint16_t* pos_table, int vocab, int dim, const uint32_t* tokens, int pos0, int T, float* x);
+// x = norm(embed[token] * scale + pos_table[position]) (pos_table, norm.w null: without).  Rows of a prompt: `tokens` from position
+// pos0.  Decode step (state given): the pending token, recorded in token_log and history, seq_len = position + 1.
+struct EmbedArgs {
+    const uint16_t *table, *pos_table;
+    int vocab, dim, ld;  // ld: pitch of `table`
+    float scale;
+    NormArgs norm;
+    const uint32_t* tokens;
+    int pos0, T;
+    float* x;            // [T, dim]
+    DecodeState* state;
+    uint64_t* history;
+    int history_cap;
+    uint32_t* token_log;
+};
+int embed_rows(cudaStream_t stream, const EmbedArgs& a);
 // out[t] = x[row[t]] normed (row null: t); out_f32 selects the type of out
-int norm_rows(cudaStream_t stream, const float* x, int dim, const int* row, int T, const uint16_t* w, float offset, float eps, int out_f32, void* out, int ldo);
+int norm_rows(cudaStream_t stream, const float* x, int dim, const int* row, int T, const NormArgs& norm, int out_f32, void* out, int ldo);
 int polynorm_rows(cudaStream_t stream, const void* z, int f32, int ldz, int n, int T, const uint16_t* coef, float eps, void* out, int ldo);
-int gated_rows(cudaStream_t stream, const float* o, int ldi, int n, int T, const uint16_t* norm_w, int head_len, float eps, const void* gate, int f32,
-               int ldg, int gate_act, void* out, int ldo);
-// rows of f32 -> bf16 or f32 at another pitch
-int convert_rows(cudaStream_t stream, const float* x, int ldi, int n, int T, int out_f32, void* out, int ldo);
+// columns [seg.begin, seg.begin + seg.cols) of o [T, ldi] f32 -> the same columns of out, zeros up to column `end`; the gate has
+// rows of ldg elements, f32 or bf16
+int gated_rows(cudaStream_t stream, const float* o, int ldi, int T, const GateSegment& seg, int gate_f32, int ldg, int end, int out_f32, void* out, int ldo);
 // table[p][i] = magnitude * (cos, sin)(p * freq[i]), evaluated in f64
 int rotation_table(cudaStream_t stream, const double* freqs, int half, int positions, double magnitude, float2* table);
 
@@ -271,7 +306,8 @@ struct LinearAttnArgs {
     float key_scale;
     const float* powers; // [heads][kLinChunk + 1]: decay^0 .. decay^kLinChunk
     float* state;        // [heads, dk, dv] f32
-    float* out;          // [T, heads * dv] f32
+    float* out;          // [T, ldo] f32
+    int ldo;
     float* scratch;      // linear_attention_scratch_floats()
 };
 size_t linear_attention_scratch_floats(int T, int heads, int dk, int dv);
@@ -294,7 +330,8 @@ struct LatentArgs {
     int pos0;
     void* cache;             // [max_seq, pitch]: normed latent at 0, rotated key part at kr_off; f32 or bf16
     int cache_f32, pitch, kr_off, max_seq;
-    float* out;              // [T, heads * vdim] f32
+    float* out;              // [T, ldo] f32
+    int ldo;
     float* work;             // decode: latent_decode_work_floats()
     unsigned int* counters;  // decode: [heads] zeros
     void* expanded;          // prompt in bf16: keys and values of every visible position [rows, ldx]
@@ -308,6 +345,67 @@ bool latent_decode_ok(const LatentArgs& a);
 int latent_attention_decode(cudaStream_t stream, const LatentArgs& a);  // T = 1, bf16 cache; writes the cache row itself
 bool latent_prefill_ok(const LatentArgs& a);
 int latent_attention_prefill(cudaStream_t stream, const LatentArgs& a); // after latent_write_cache and the expansion
+
+// ---- grouped softmax attention (grouped_attention.cu) --------------------------------------------------------------------
+// Query head h uses key / value head h / (heads / kv_heads).  A position sees itself and the earlier positions of its window
+// (the last `window` positions), of its chunk (positions are cut into chunks of `chunk` from 0), or all of them (both 0).
+struct GroupedArgs {
+    const void* in;      // [T, ld]: q at q_off, k at k_off, v at v_off, head by head
+    int in_f32, ld, q_off, k_off, v_off;
+    int T, heads, kv_heads, dim, vdim, window, chunk;
+    float scale;
+    const DecodeState* at;  // position of the first token: at->position, or pos0 when null
+    int pos0;
+    void* cache;         // [max_seq, pitch]: keys of dimp entries per head, then values of vdimp; f32 or bf16
+    int cache_f32, pitch, dimp, vdimp, max_seq;
+    float* out;          // [T, ldo] f32
+    int ldo;
+    float* work;         // decode: grouped_decode_work_floats()
+    unsigned int* counters;  // decode: kGroupedMaxTiles zeros, left so
+};
+constexpr int kGroupedMaxTiles = 1024;
+int grouped_write_cache(cudaStream_t stream, const GroupedArgs& a);
+int grouped_attention_plain(cudaStream_t stream, const GroupedArgs& a);   // any size, f32 arithmetic, after grouped_write_cache
+size_t grouped_decode_work_floats(int heads, int kv_heads, int vdim);
+bool grouped_decode_ok(const GroupedArgs& a);
+int grouped_attention_decode(cudaStream_t stream, const GroupedArgs& a);  // T = 1, bf16 cache; writes the cache row itself
+bool grouped_prefill_ok(const GroupedArgs& a);
+int grouped_attention_prefill(cudaStream_t stream, const GroupedArgs& a); // bf16, after grouped_write_cache
+
+// ---- linear attention with a decay per key channel and token (gated_linear.cu) -------------------------------------------
+//   S <- diag(alpha) S + k u^T, o = S^T q;  u = v, or (delta) beta (v - (diag(alpha) S)^T k)
+// alpha from z = W_up a (+ bias): sigmoid(z)^(1 / tau) or exp(-exp(A_head) softplus(z)).  q, k and v go through a causal
+// convolution of `taps` taps and SiLU (taps 0: neither), q and k are made unit vectors when unit_eps > 0, q is scaled.
+struct GatedLinearArgs {
+    const void* in;      // [T, ld]: q, k (kv_heads x dk), v (heads x dv), a (rank), logits of beta (heads), gate factor (gate_rank)
+    int in_f32, ld, q_off, k_off, v_off, a_off, b_off, g_off;
+    int T, heads, kv_heads, dk, dv;
+    int decay;           // KMLL_DECAY_*
+    float inv_tau;
+    int rank, ldu;
+    const uint16_t* up;  // [heads * dk, ldu]
+    const uint16_t* bias;    // [heads * dk] or null
+    const uint16_t* a_log;   // [heads], KMLL_DECAY_SOFTPLUS
+    int delta;
+    int taps;
+    const uint16_t* conv;    // [q | k | v channels][taps]
+    float* ring;             // [taps][channels]: projected inputs of the last `taps` positions, slot = position % taps
+    float unit_eps, q_scale;
+    int gate_rank, ldg;      // low-rank output gate: gate = W_gate g (gate_rank 0: none here)
+    const uint16_t* gate_up; // [heads * dv, ldg]
+    float* gate;             // [T, heads * dv] f32 (step form)
+    const DecodeState* at;
+    int pos0;
+    float* state;        // [heads, dk, dv] f32
+    float* out;          // [T, ldo] f32
+    int ldo;
+    float* scratch;      // chunked form: gated_chunk_scratch_floats()
+};
+constexpr int kMaxConvTaps = 16;
+int gated_linear_steps(cudaStream_t stream, const GatedLinearArgs& a);    // token after token in f32 (decode; prompts in f32)
+bool gated_linear_chunked_ok(const GatedLinearArgs& a);
+size_t gated_chunk_scratch_floats(int T, int heads, int dk, int dv, int delta);
+int gated_linear_chunked(cudaStream_t stream, const GatedLinearArgs& a);  // bf16 inputs: chunks on the tensor cores; without the gate
 
 // Deterministic merge of per-rank packed results: higher logit wins, ties -> lower token.
 int merge_packed_top1(cudaStream_t stream, const uint64_t* packed_all, int n, uint64_t* packed_out);

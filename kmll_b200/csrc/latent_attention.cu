@@ -110,7 +110,7 @@ __global__ void __launch_bounds__(kPlainWarps * 32) latent_plain_kernel(const La
         float s = 0.0f;
         for (int r = lane; r < a.rank; r += 32) s = fmaf(bf16_bits_to_f32(u[r]), qa[r], s);
         s = warp_sum(s);
-        if (lane == 0) a.out[(size_t)t * a.heads * a.vdim + (size_t)h * a.vdim + v] = s;
+        if (lane == 0) a.out[(size_t)t * a.ldo + (size_t)h * a.vdim + v] = s;
     }
 }
 
@@ -631,7 +631,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a)
         }
     }
     const float inv_a = 1.0f / l_run[0], inv_b = 1.0f / l_run[1];
-    const size_t ldo = (size_t)a.heads * a.vdim;
+    const size_t ldo = (size_t)a.ldo;
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i)
 #pragma unroll

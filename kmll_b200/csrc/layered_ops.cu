@@ -9,7 +9,7 @@ namespace {
 Bf16Matvec base(const float* x, const uint16_t* w, int pitch, int rows, int cols, const float* residual, float* y) {
     Bf16Matvec v;
     memset(&v, 0, sizeof(v));
-    v.x = x; v.w = w; v.ldw = pitch; v.rows = rows; v.K = cols; v.residual = residual; v.y = y;
+    v.x = x; v.w = w; v.ldw = pitch; v.rows = rows; v.K = cols; v.residual = residual; v.y = y; v.out_scale = 1.0f;
     return v;
 }
 int up8(int v) { return (v + 7) & ~7; }
@@ -22,7 +22,7 @@ int kmll_linear_bf16(kmll_stream_t s, const float* x, const uint16_t* w, int pit
     KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(y);
     Bf16Matvec v = base(x, w, pitch, rows, cols, residual, y);
     v.silu_rows = silu_rows;
-    if (norm_weight != nullptr) { v.pro = PRO_RMSNORM; v.norm_w = norm_weight; v.norm_offset = norm_offset; v.eps = eps; }
+    if (norm_weight != nullptr) { v.pro = PRO_NORM; v.norm = NormArgs{KMLL_NORM_RMS, norm_weight, nullptr, norm_offset, eps}; }
     return bf16_matvec(as_stream(s), v);
 }
 
@@ -39,7 +39,10 @@ int kmll_gated_linear_bf16(kmll_stream_t s, const float* x, const uint16_t* norm
     KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(gate); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(y);
     KMLL_REQUIRE(norm_weight != nullptr || (head_len > 0 && cols > 0 && cols % head_len == 0), "gated_linear_bf16: %d columns are not heads of %d", cols, head_len);
     Bf16Matvec v = base(x, w, pitch, rows, cols, residual, y);
-    v.pro = PRO_GATED; v.norm_w = norm_weight; v.head_len = head_len; v.eps = eps; v.gate = gate; v.gate_act = gate_sigmoid ? KMLL_ACT_SIGMOID : KMLL_ACT_SILU;
+    v.pro = PRO_GATED;
+    v.n_seg = 1;
+    v.seg[0] = GateSegment{0, cols, norm_weight != nullptr ? cols : head_len, norm_weight != nullptr ? KMLL_OUT_NORM_JOINT : KMLL_OUT_NORM_PER_HEAD, norm_weight, gate, 1,
+                           gate_sigmoid ? KMLL_ACT_SIGMOID : KMLL_ACT_SILU, 1.0f, eps};
     return bf16_matvec(as_stream(s), v);
 }
 
@@ -51,7 +54,7 @@ int kmll_linear_batched_bf16(kmll_stream_t s, const void* x, int x_f32, int ldx,
     Bf16Gemm g;
     memset(&g, 0, sizeof(g));
     g.x = x; g.x_f32 = x_f32; g.ldx = ldx; g.T = batch; g.K = cols; g.w = w; g.rows = rows; g.ldw = pitch; g.out = out; g.out_bf16 = out_bf16; g.ldo = rows;
-    g.residual = residual;
+    g.residual = residual; g.out_scale = 1.0f;
     if (workspace != nullptr) {
         g.counters = static_cast<unsigned int*>(workspace);
         g.partial = static_cast<float*>(workspace) + 128;
@@ -78,7 +81,7 @@ int kmll_linear_attention(kmll_stream_t s, const void* in, int in_f32, int ld, i
     a.in = in; a.in_f32 = in_f32; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.T = tokens; a.heads = heads; a.dk = dk; a.dv = dv; a.rot = rot;
     a.table = reinterpret_cast<const float2*>(table);
     a.at = reinterpret_cast<const DecodeState*>(position_device);  // (the position is its first field)
-    a.pos0 = position; a.key_scale = key_scale; a.powers = powers; a.state = state; a.scratch = scratch; a.out = out;
+    a.pos0 = position; a.key_scale = key_scale; a.powers = powers; a.state = state; a.scratch = scratch; a.out = out; a.ldo = heads * dv;
     return scratch != nullptr ? linear_attention_chunked(as_stream(s), a) : linear_attention_recurrent(as_stream(s), a);
 }
 
@@ -90,7 +93,7 @@ static LatentArgs latent_base(int heads, int dim, int rot, int vdim, int rank, i
     a.heads = heads; a.dim = dim; a.rot = rot; a.vdim = vdim; a.rank = rank; a.window = window; a.scale = scale;
     a.table = reinterpret_cast<const float2*>(table);
     a.cache = const_cast<uint16_t*>(cache); a.pitch = pitch; a.kr_off = up8(rank); a.max_seq = max_seq;
-    a.out = out;
+    a.out = out; a.ldo = heads * vdim;
     return a;
 }
 

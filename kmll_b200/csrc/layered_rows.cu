@@ -1,17 +1,12 @@
 // Row operators of the layered decoders' prompt path: what stands between two projections, one block per row, f32 arithmetic,
 // result in the type the next projection reads.  (A decode step runs the same steps as prologues of bf16_matvec_kernel.)
-#include "internal.cuh"
+#include "activations.cuh"
 
 namespace kmll {
 
 namespace {
 
 constexpr int kRowThreads = 256;
-
-__device__ inline float silu_f(float z) { return z / (1.0f + expf(-z)); }
-__device__ inline float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ inline float gate_f(float z, int act) { return act == KMLL_ACT_SILU ? silu_f(z) : act == KMLL_ACT_SIGMOID ? sigmoid_f(z) : z; }
-__device__ inline float inv_rms_f(float sum_sq, int n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
 
 template <bool F32>
 __device__ inline float load1(const void* p, size_t i) {
@@ -56,38 +51,105 @@ __device__ inline void storev(void* p, size_t i, const float (&v)[V]) {
     }
 }
 
-__global__ void embed_rows_kernel(const uint16_t* __restrict__ table, const uint16_t* __restrict__ pos_table, int vocab, int dim,
-                                  const uint32_t* __restrict__ tokens, int pos0, float* __restrict__ x) {
+// One block per row; entry i of a row is always held by the same thread.
+__global__ void __launch_bounds__(1024) embed_rows_kernel(const EmbedArgs a) {
+    __shared__ float scratch[96];
     pdl_wait();
     const int t = blockIdx.x;
-    uint32_t token = tokens[t];
-    if (token >= (uint32_t)vocab) token = (uint32_t)vocab - 1;
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        float v = bf16_bits_to_f32(table[(size_t)token * dim + i]);
-        if (pos_table != nullptr) v += bf16_bits_to_f32(pos_table[(size_t)(pos0 + t) * dim + i]);
-        x[(size_t)t * dim + i] = v;
+    int pos = a.pos0 + t;
+    uint32_t token;
+    if (a.state != nullptr) {
+        const uint64_t packed = a.state->next_top;
+        token = (uint32_t)(packed & 0xffffffffull);
+        if (token >= (uint32_t)a.vocab) token = (uint32_t)a.vocab - 1;
+        pos = a.state->position;
+        if (threadIdx.x == 0) {
+            const int step = a.state->step;
+            a.token_log[pos] = token;
+            if (step < a.history_cap) a.history[step] = packed;
+            a.state->seq_len = pos + 1;
+        }
+    } else {
+        token = a.tokens[t];
+        if (token >= (uint32_t)a.vocab) token = (uint32_t)a.vocab - 1;
+    }
+    const uint16_t* e = a.table + (size_t)token * a.ld;
+    const uint16_t* p = a.pos_table != nullptr ? a.pos_table + (size_t)pos * a.dim : nullptr;
+    float* x = a.x + (size_t)t * a.dim;
+    auto value = [&](int i) {
+        float v = bf16_bits_to_f32(e[i]) * a.scale;
+        if (p != nullptr) v += bf16_bits_to_f32(p[i]);
+        return v;
+    };
+    if (a.norm.w == nullptr) {
+        for (int i = threadIdx.x; i < a.dim; i += blockDim.x) x[i] = value(i);
+        return;
+    }
+    float s = 0.0f, q = 0.0f;
+    int n = 0;
+    for (int i = threadIdx.x; i < a.dim; i += blockDim.x) {
+        const float v = value(i);
+        s += v;
+        q += v * v;
+        ++n;
+    }
+    float mean = 0.0f, inv;
+    if (a.norm.kind == KMLL_NORM_LAYER) {
+        Moments m{(float)n, n > 0 ? s / (float)n : 0.0f, 0.0f};
+        for (int i = threadIdx.x; i < a.dim; i += blockDim.x) {
+            const float v = value(i) - m.mean;
+            m.dev += v * v;
+        }
+        m = block_moments(m, scratch);
+        mean = m.mean;
+        inv = inv_rms(m.dev, a.dim, a.norm.eps);
+    } else {
+        inv = inv_rms(block_sum(q, scratch), a.dim, a.norm.eps);
+    }
+    for (int i = threadIdx.x; i < a.dim; i += blockDim.x) {
+        float v = (value(i) - mean) * inv * (a.norm.offset + bf16_bits_to_f32(a.norm.w[i]));
+        if (a.norm.kind == KMLL_NORM_LAYER) v += bf16_bits_to_f32(a.norm.b[i]);
+        x[i] = v;
     }
 }
 
-template <bool OUT32, int V>
-__global__ void __launch_bounds__(kRowThreads) norm_rows_kernel(const float* __restrict__ x, int dim, const int* __restrict__ row,
-                                                                const uint16_t* __restrict__ w, float offset, float eps, void* out, int ldo) {
-    __shared__ float scratch[40];
+template <bool LAYER, bool OUT32, int V>
+__global__ void __launch_bounds__(kRowThreads) norm_rows_kernel(const float* __restrict__ x, int dim, const int* __restrict__ row, const NormArgs norm, void* out,
+                                                                int ldo) {
+    __shared__ float scratch[96];
     pdl_wait();
     const int t = blockIdx.x;
     const float* xr = x + (size_t)(row != nullptr ? row[t] : t) * dim;
-    float s = 0.0f, v[V], g[V];
+    float s = 0.0f, mean = 0.0f, inv, v[V], g[V], b[V];
+    int n = 0;
     for (int i = threadIdx.x * V; i < dim; i += kRowThreads * V) {
         loadv<true, V>(xr, i, v);
 #pragma unroll
-        for (int e = 0; e < V; ++e) s += v[e] * v[e];
+        for (int e = 0; e < V; ++e) s += LAYER ? v[e] : v[e] * v[e];
+        n += V;
     }
-    const float inv = inv_rms_f(block_sum(s, scratch), dim, eps);
+    if (LAYER) {
+        Moments m{(float)n, n > 0 ? s / (float)n : 0.0f, 0.0f};
+        for (int i = threadIdx.x * V; i < dim; i += kRowThreads * V) {
+            loadv<true, V>(xr, i, v);
+#pragma unroll
+            for (int e = 0; e < V; ++e) m.dev += (v[e] - m.mean) * (v[e] - m.mean);
+        }
+        m = block_moments(m, scratch);
+        mean = m.mean;
+        inv = inv_rms(m.dev, dim, norm.eps);
+    } else {
+        inv = inv_rms(block_sum(s, scratch), dim, norm.eps);
+    }
     for (int i = threadIdx.x * V; i < dim; i += kRowThreads * V) {
         loadv<true, V>(xr, i, v);
-        loadv<false, V>(w, i, g);
+        loadv<false, V>(norm.w, i, g);
+        if (LAYER) loadv<false, V>(norm.b, i, b);
 #pragma unroll
-        for (int e = 0; e < V; ++e) v[e] *= inv * (offset + g[e]);
+        for (int e = 0; e < V; ++e) {
+            v[e] = (v[e] - mean) * inv * (norm.offset + g[e]);
+            if (LAYER) v[e] += b[e];
+        }
         storev<OUT32, V>(out, (size_t)t * ldo + i, v);
     }
 }
@@ -112,8 +174,8 @@ __global__ void __launch_bounds__(kRowThreads) polynorm_rows_kernel(const void* 
     s1 = block_sum(s1, scratch);
     s2 = block_sum(s2, scratch);
     s3 = block_sum(s3, scratch);
-    const float c1 = bf16_bits_to_f32(coef[0]) * inv_rms_f(s1, n, eps), c2 = bf16_bits_to_f32(coef[1]) * inv_rms_f(s2, n, eps),
-                c3 = bf16_bits_to_f32(coef[2]) * inv_rms_f(s3, n, eps), c0 = bf16_bits_to_f32(coef[3]);
+    const float c1 = bf16_bits_to_f32(coef[0]) * inv_rms(s1, n, eps), c2 = bf16_bits_to_f32(coef[1]) * inv_rms(s2, n, eps),
+                c3 = bf16_bits_to_f32(coef[2]) * inv_rms(s3, n, eps), c0 = bf16_bits_to_f32(coef[3]);
     for (int i = threadIdx.x * V; i < n; i += kRowThreads * V) {
         loadv<F32, V>(z, zr + i, v);
 #pragma unroll
@@ -122,60 +184,76 @@ __global__ void __launch_bounds__(kRowThreads) polynorm_rows_kernel(const void* 
     }
 }
 
-// o normed (per head without weight, or over the whole row with norm_w), times gate_act(gate)
-template <bool F32, int V>
-__global__ void __launch_bounds__(kRowThreads) gated_rows_kernel(const float* __restrict__ o, int ldi, int n, const uint16_t* __restrict__ norm_w,
-                                                                 int head_len, float eps, const void* __restrict__ gate, int ldg, int gate_act,
-                                                                 void* out, int ldo) {
+// one segment of a mixer's output: normed, times act(gate), times its scale; zeros behind it up to column `end`
+template <bool GATE32, bool OUT32, int V>
+__global__ void __launch_bounds__(kRowThreads) gated_rows_kernel(const float* __restrict__ o, int ldi, const GateSegment seg, int ldg, int end, void* out, int ldo) {
     __shared__ float scratch[40];
     pdl_wait();
-    const float* orow = o + (size_t)blockIdx.x * ldi;
-    const size_t gr = (size_t)blockIdx.x * ldg, outr = (size_t)blockIdx.x * ldo;
+    const float* orow = o + (size_t)blockIdx.x * ldi + seg.begin;
+    const size_t gr = (size_t)blockIdx.x * ldg, outr = (size_t)blockIdx.x * ldo + seg.begin;
+    const int n = seg.cols, len = seg.head_len;
     float v[V], g[V], w[V];
-    if (norm_w != nullptr) {
-        float s = 0.0f;
-        for (int i = threadIdx.x * V; i < n; i += kRowThreads * V) {
-            loadv<true, V>(orow, i, v);
+    for (int i = n + threadIdx.x; i < end - seg.begin; i += kRowThreads) store1<OUT32>(out, outr + i, 0.0f);
+    auto gates = [&](int i) {  // of entries i .. i + V - 1 (one head, when heads share a gate)
+        if (seg.gate == nullptr) {
 #pragma unroll
-            for (int e = 0; e < V; ++e) s += v[e] * v[e];
+            for (int e = 0; e < V; ++e) g[e] = seg.scale;
+        } else if (seg.gate_len == 1) {
+            loadv<GATE32, V>(seg.gate, gr + i, g);
+#pragma unroll
+            for (int e = 0; e < V; ++e) g[e] = seg.scale * apply_act(g[e], seg.act);
+        } else {
+            const float f = seg.scale * apply_act(load1<GATE32>(seg.gate, gr + i / seg.gate_len), seg.act);
+#pragma unroll
+            for (int e = 0; e < V; ++e) g[e] = f;
         }
-        const float inv = inv_rms_f(block_sum(s, scratch), n, eps);
+    };
+    if (seg.norm == KMLL_OUT_NORM_JOINT || seg.norm == KMLL_OUT_NORM_NONE) {
+        float inv = 1.0f;
+        if (seg.norm == KMLL_OUT_NORM_JOINT) {
+            float s = 0.0f;
+            for (int i = threadIdx.x * V; i < n; i += kRowThreads * V) {
+                loadv<true, V>(orow, i, v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) s += v[e] * v[e];
+            }
+            inv = inv_rms(block_sum(s, scratch), n, seg.eps);
+        }
         for (int i = threadIdx.x * V; i < n; i += kRowThreads * V) {
             loadv<true, V>(orow, i, v);
-            loadv<F32, V>(gate, gr + i, g);
-            loadv<false, V>(norm_w, i, w);
+            gates(i);
+            if (seg.norm == KMLL_OUT_NORM_JOINT) {
+                loadv<false, V>(seg.norm_w, i, w);
 #pragma unroll
-            for (int e = 0; e < V; ++e) v[e] *= inv * w[e] * gate_f(g[e], gate_act);
-            storev<F32, V>(out, outr + i, v);
+                for (int e = 0; e < V; ++e) v[e] *= inv * w[e];
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] *= g[e];
+            storev<OUT32, V>(out, outr + i, v);
         }
         return;
     }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int h0 = warp * head_len; h0 < n; h0 += (kRowThreads / 32) * head_len) {  // a warp per head
+    for (int h0 = warp * len; h0 < n; h0 += (kRowThreads / 32) * len) {  // a warp per head
         float s = 0.0f;
-        for (int i = lane * V; i < head_len; i += 32 * V) {
+        for (int i = lane * V; i < len; i += 32 * V) {
             loadv<true, V>(orow, h0 + i, v);
 #pragma unroll
             for (int e = 0; e < V; ++e) s += v[e] * v[e];
         }
-        const float inv = inv_rms_f(warp_sum(s), head_len, eps);
-        for (int i = lane * V; i < head_len; i += 32 * V) {
+        const float inv = inv_rms(warp_sum(s), len, seg.eps);
+        for (int i = lane * V; i < len; i += 32 * V) {
             loadv<true, V>(orow, h0 + i, v);
-            loadv<F32, V>(gate, gr + h0 + i, g);
+            gates(h0 + i);
+            if (seg.norm == KMLL_OUT_NORM_HEAD_WEIGHTED) {
+                loadv<false, V>(seg.norm_w, i, w);
 #pragma unroll
-            for (int e = 0; e < V; ++e) v[e] *= inv * gate_f(g[e], gate_act);
-            storev<F32, V>(out, outr + h0 + i, v);
+                for (int e = 0; e < V; ++e) v[e] *= w[e];
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] *= inv * g[e];
+            storev<OUT32, V>(out, outr + h0 + i, v);
         }
-    }
-}
-
-template <bool OUT32, int V>
-__global__ void __launch_bounds__(kRowThreads) convert_rows_kernel(const float* __restrict__ x, int ldi, int n, void* out, int ldo) {
-    pdl_wait();
-    float v[V];
-    for (int i = threadIdx.x * V; i < n; i += kRowThreads * V) {
-        loadv<true, V>(x, (size_t)blockIdx.x * ldi + i, v);
-        storev<OUT32, V>(out, (size_t)blockIdx.x * ldo + i, v);
     }
 }
 
@@ -203,14 +281,19 @@ bool aligned(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) 
         return KMLL_OK;                                                                          \
     } while (0)
 
-int embed_rows(cudaStream_t stream, const uint16_t* table, const uint16_t* pos_table, int vocab, int dim, const uint32_t* tokens, int pos0, int T, float* x) {
-    KMLL_ROWS_CHECK(launch(embed_rows_kernel, dim3(T), dim3(256), 0, stream, true, table, pos_table, vocab, dim, tokens, pos0, x), "embed_rows");
+int embed_rows(cudaStream_t stream, const EmbedArgs& a) {
+    const int threads = a.dim >= 1024 ? 1024 : (a.dim + 31) / 32 * 32;
+    KMLL_ROWS_CHECK(launch(embed_rows_kernel, dim3(a.T), dim3(threads), 0, stream, true, a), "embed_rows");
 }
 
-int norm_rows(cudaStream_t stream, const float* x, int dim, const int* row, int T, const uint16_t* w, float offset, float eps, int out_f32, void* out, int ldo) {
-    const bool v4 = by4({dim, ldo}) && aligned(x, 16) && aligned(w, 8) && aligned(out, 16);
-    auto k = out_f32 ? (v4 ? norm_rows_kernel<true, 4> : norm_rows_kernel<true, 1>) : (v4 ? norm_rows_kernel<false, 4> : norm_rows_kernel<false, 1>);
-    KMLL_ROWS_CHECK(launch(k, dim3(T), dim3(kRowThreads), 0, stream, true, x, dim, row, w, offset, eps, out, ldo), "norm_rows");
+int norm_rows(cudaStream_t stream, const float* x, int dim, const int* row, int T, const NormArgs& norm, int out_f32, void* out, int ldo) {
+    const bool v4 = by4({dim, ldo}) && aligned(x, 16) && aligned(norm.w, 8) && aligned(out, 16) && (norm.b == nullptr || aligned(norm.b, 8));
+    void (*k)(const float*, int, const int*, const NormArgs, void*, int) = nullptr;
+    if (norm.kind == KMLL_NORM_LAYER)
+        k = out_f32 ? (v4 ? norm_rows_kernel<true, true, 4> : norm_rows_kernel<true, true, 1>) : (v4 ? norm_rows_kernel<true, false, 4> : norm_rows_kernel<true, false, 1>);
+    else
+        k = out_f32 ? (v4 ? norm_rows_kernel<false, true, 4> : norm_rows_kernel<false, true, 1>) : (v4 ? norm_rows_kernel<false, false, 4> : norm_rows_kernel<false, false, 1>);
+    KMLL_ROWS_CHECK(launch(k, dim3(T), dim3(kRowThreads), 0, stream, true, x, dim, row, norm, out, ldo), "norm_rows");
 }
 
 int polynorm_rows(cudaStream_t stream, const void* z, int f32, int ldz, int n, int T, const uint16_t* coef, float eps, void* out, int ldo) {
@@ -219,17 +302,16 @@ int polynorm_rows(cudaStream_t stream, const void* z, int f32, int ldz, int n, i
     KMLL_ROWS_CHECK(launch(k, dim3(T), dim3(kRowThreads), 0, stream, true, z, ldz, n, coef, eps, out, ldo), "polynorm_rows");
 }
 
-int gated_rows(cudaStream_t stream, const float* o, int ldi, int n, int T, const uint16_t* norm_w, int head_len, float eps, const void* gate, int f32,
-               int ldg, int gate_act, void* out, int ldo) {
-    const bool v4 = by4({n, ldi, ldg, ldo, head_len}) && aligned(o, 16) && aligned(gate, 16) && aligned(out, 16) && (norm_w == nullptr || aligned(norm_w, 8));
-    auto k = f32 ? (v4 ? gated_rows_kernel<true, 4> : gated_rows_kernel<true, 1>) : (v4 ? gated_rows_kernel<false, 4> : gated_rows_kernel<false, 1>);
-    KMLL_ROWS_CHECK(launch(k, dim3(T), dim3(kRowThreads), 0, stream, true, o, ldi, n, norm_w, head_len, eps, gate, ldg, gate_act, out, ldo), "gated_rows");
-}
-
-int convert_rows(cudaStream_t stream, const float* x, int ldi, int n, int T, int out_f32, void* out, int ldo) {
-    const bool v4 = by4({n, ldi, ldo}) && aligned(x, 16) && aligned(out, 16);
-    auto k = out_f32 ? (v4 ? convert_rows_kernel<true, 4> : convert_rows_kernel<true, 1>) : (v4 ? convert_rows_kernel<false, 4> : convert_rows_kernel<false, 1>);
-    KMLL_ROWS_CHECK(launch(k, dim3(T), dim3(kRowThreads), 0, stream, true, x, ldi, n, out, ldo), "convert_rows");
+int gated_rows(cudaStream_t stream, const float* o, int ldi, int T, const GateSegment& seg, int gate_f32, int ldg, int end, int out_f32, void* out, int ldo) {
+    const bool v4 = by4({seg.begin, seg.cols, ldi, ldo}) && (seg.norm == KMLL_OUT_NORM_JOINT || (seg.norm == KMLL_OUT_NORM_NONE && seg.gate_len == 1) || by4({seg.head_len})) &&
+                    (seg.gate == nullptr || (seg.gate_len == 1 ? by4({ldg}) && aligned(seg.gate, 16) : by4({seg.gate_len}))) && aligned(o, 16) && aligned(out, 16) &&
+                    (seg.norm_w == nullptr || aligned(seg.norm_w, 8));
+    void (*k)(const float*, int, const GateSegment, int, int, void*, int) = nullptr;
+    if (gate_f32)
+        k = out_f32 ? (v4 ? gated_rows_kernel<true, true, 4> : gated_rows_kernel<true, true, 1>) : (v4 ? gated_rows_kernel<true, false, 4> : gated_rows_kernel<true, false, 1>);
+    else
+        k = out_f32 ? (v4 ? gated_rows_kernel<false, true, 4> : gated_rows_kernel<false, true, 1>) : (v4 ? gated_rows_kernel<false, false, 4> : gated_rows_kernel<false, false, 1>);
+    KMLL_ROWS_CHECK(launch(k, dim3(T), dim3(kRowThreads), 0, stream, true, o, ldi, seg, ldg, end, out, ldo), "gated_rows");
 }
 
 int rotation_table(cudaStream_t stream, const double* freqs, int half, int positions, double magnitude, float2* table) {

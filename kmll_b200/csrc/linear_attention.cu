@@ -101,7 +101,7 @@ __global__ void __launch_bounds__(256) linear_recurrent_kernel(const LinearAttnA
             float sum = 0.0f;
 #pragma unroll
             for (int w = 0; w < 8; ++w) sum += red[w * 32 + tid];
-            a.out[(size_t)t * a.heads * a.dv + (size_t)h * a.dv + c] = sum;
+            a.out[(size_t)t * a.ldo + (size_t)h * a.dv + c] = sum;
         }
         // (the next token's q and k overwrite nothing that is still read: all reads of them lie before the barrier above;
         // `red` is rewritten only after the next barrier)
@@ -135,7 +135,7 @@ constexpr int kC = kLinChunk, kB = 64, kCThreads = 128, kPS = 64 + 8;  // kPS: p
 struct ChunkArgs {
     const uint16_t *qh, *ql, *kh, *kl, *v;  // rows of ldq / ldv elements, heads hq / hv apart; ql, kl null: exact
     int ldq, hq, ldv, hv;
-    int T, heads, dk, dv, dvp, chunks;
+    int T, heads, dk, dv, dvp, chunks, ldo;
     float key_scale;                        // still to be applied (1 once it is in the planes)
     const float* powers;
     float* state;
@@ -489,8 +489,8 @@ __global__ void __launch_bounds__(kCThreads) linear_chunk_outputs_kernel(const C
             }
         }
     }
-    const size_t ldo = (size_t)a.heads * a.dv;
-    const bool v2 = (a.dv & 1) == 0;
+    const size_t ldo = (size_t)a.ldo;
+    const bool v2 = ((a.dv | a.ldo) & 1) == 0;
 #pragma unroll
     for (int i = 0; i < VT / 8; ++i)
 #pragma unroll
@@ -571,7 +571,7 @@ int linear_attention_chunked(cudaStream_t stream, const LinearAttnArgs& a) {
     ChunkArgs c;
     memset(&c, 0, sizeof(c));
     c.T = a.T; c.heads = a.heads; c.dk = a.dk; c.dv = a.dv; c.dvp = dvp; c.chunks = (a.T + kC - 1) / kC;
-    c.powers = a.powers; c.state = a.state; c.out = a.out;
+    c.powers = a.powers; c.state = a.state; c.out = a.out; c.ldo = a.ldo;
     float* f = a.scratch;
     c.kv = f;
     c.sh = reinterpret_cast<uint16_t*>(f + m.kv);

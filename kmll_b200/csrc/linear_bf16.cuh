@@ -11,6 +11,8 @@
 
 #include <algorithm>
 
+#include "activations.cuh"
+
 namespace kmll {
 
 // ---- one row of x -------------------------------------------------------------------------------------------------------
@@ -25,12 +27,6 @@ constexpr int kVThreads = kVWarps * 32;
 constexpr int kVRows = 16;     // rows whose sums a warp holds in registers
 constexpr int kVDepth = 8;     // 16-byte copies in flight per lane (64 KB per block, two blocks per SM)
 constexpr int kVPiece = 256;   // columns per warp and step
-
-__device__ inline float act_silu(float z) { return z / (1.0f + expf(-z)); }
-__device__ inline float act_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ inline float apply_act(float z, int act) { return act == KMLL_ACT_SILU ? act_silu(z) : act == KMLL_ACT_SIGMOID ? act_sigmoid(z) : z; }
-// 1 / root mean square with eps inside the root
-__device__ inline float inv_rms(float sum_sq, int n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
 
 // index of column k in the staged vector: two planes, so that the 16-byte reads of a warp are free of bank conflicts
 __device__ inline int vec_slot(int k, int half) { return ((k >> 2) & 1) * half + ((k >> 3) << 2) + (k & 3); }
@@ -54,7 +50,7 @@ __device__ inline void block_sum3(float (&v)[3], float* scratch) {
 
 struct MatvecArgs {
     Bf16Matvec a;
-    int half, kpieces, rows_cap, n_heads;
+    int half, kpieces, rows_cap, n_heads;  // n_heads: of all segments
     int off_x, off_part, off_head;  // byte offsets in shared memory (the ring is at 0)
 };
 
@@ -66,7 +62,8 @@ __global__ void __launch_bounds__(kVThreads, 2) bf16_matvec_kernel(const MatvecA
     float* const xs = reinterpret_cast<float*>(vsmem + p.off_x);
     float* const part = reinterpret_cast<float*>(vsmem + p.off_part);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int r0 = (int)((long long)blockIdx.x * a.rows / gridDim.x), r1 = (int)((long long)(blockIdx.x + 1) * a.rows / gridDim.x);
+    const int unit = a.pair_act != 0 ? 2 : 1, units = a.rows / unit;
+    const int r0 = unit * (int)((long long)blockIdx.x * units / gridDim.x), r1 = unit * (int)((long long)(blockIdx.x + 1) * units / gridDim.x);
     const int nrows = r1 - r0, ngroups = (nrows + kVRows - 1) / kVRows;
     const int mine = p.kpieces > warp ? (p.kpieces - warp + kVWarps - 1) / kVWarps : 0;  // pieces of this warp
     const uint32_t ring = smem_u32(vsmem) + (uint32_t)tid * 16u;
@@ -88,15 +85,32 @@ __global__ void __launch_bounds__(kVThreads, 2) bf16_matvec_kernel(const MatvecA
     pdl_wait();
     // ---- x -> shared memory through the prologue; columns K .. are zeros
     const int kpad = p.kpieces * kVPiece;
-    if (a.pro == PRO_RMSNORM) {
+    if (a.pro == PRO_NORM && a.norm.kind == KMLL_NORM_LAYER) {
+        float s = 0.0f;
+        int n = 0;
+        for (int k = tid; k < kpad; k += kVThreads) {
+            const float v = k < a.K ? a.x[k] : 0.0f;
+            if (k < a.K) { s += v; ++n; }
+            xs[vec_slot(k, p.half)] = v;
+        }
+        Moments m{(float)n, n > 0 ? s / (float)n : 0.0f, 0.0f};
+        for (int k = tid; k < a.K; k += kVThreads) {
+            const float v = xs[vec_slot(k, p.half)] - m.mean;
+            m.dev += v * v;
+        }
+        m = block_moments(m, scratch);
+        const float inv = inv_rms(m.dev, a.K, a.norm.eps);
+        for (int k = tid; k < a.K; k += kVThreads)
+            xs[vec_slot(k, p.half)] = (xs[vec_slot(k, p.half)] - m.mean) * inv * (a.norm.offset + bf16_bits_to_f32(a.norm.w[k])) + bf16_bits_to_f32(a.norm.b[k]);
+    } else if (a.pro == PRO_NORM) {
         float s = 0.0f;
         for (int k = tid; k < kpad; k += kVThreads) {
             const float v = k < a.K ? a.x[k] : 0.0f;
             s += v * v;
             xs[vec_slot(k, p.half)] = v;
         }
-        const float inv = inv_rms(block_sum(s, scratch), a.K, a.eps);
-        for (int k = tid; k < a.K; k += kVThreads) xs[vec_slot(k, p.half)] *= inv * (a.norm_offset + bf16_bits_to_f32(a.norm_w[k]));
+        const float inv = inv_rms(block_sum(s, scratch), a.K, a.norm.eps);
+        for (int k = tid; k < a.K; k += kVThreads) xs[vec_slot(k, p.half)] *= inv * (a.norm.offset + bf16_bits_to_f32(a.norm.w[k]));
     } else if (a.pro == PRO_POLYNORM) {
         float s[3] = {0.0f, 0.0f, 0.0f};
         for (int k = tid; k < kpad; k += kVThreads) {
@@ -114,31 +128,63 @@ __global__ void __launch_bounds__(kVThreads, 2) bf16_matvec_kernel(const MatvecA
             xs[vec_slot(k, p.half)] = ((c3 * v + c2) * v + c1) * v + c0;
         }
     } else if (a.pro == PRO_GATED) {
-        float s = 0.0f;
+        float s[kMaxSegments] = {};
         for (int k = tid; k < kpad; k += kVThreads) {
             const float v = k < a.K ? a.x[k] : 0.0f;
-            s += v * v;
+#pragma unroll
+            for (int j = 0; j < kMaxSegments; ++j)
+                if (j < a.n_seg && k >= a.seg[j].begin && k < a.seg[j].begin + a.seg[j].cols) s[j] += v * v;
             xs[vec_slot(k, p.half)] = v;
         }
-        if (a.norm_w != nullptr) {  // one norm over all heads, weighted
-            const float inv = inv_rms(block_sum(s, scratch), a.K, a.eps);
-            for (int k = tid; k < a.K; k += kVThreads)
-                xs[vec_slot(k, p.half)] *= inv * bf16_bits_to_f32(a.norm_w[k]) * apply_act(a.gate[k], a.gate_act);
-        } else {  // every head over its own root mean square
-            float* const hinv = reinterpret_cast<float*>(vsmem + p.off_head);
-            __syncthreads();
-            for (int h = warp; h < p.n_heads; h += kVWarps) {
-                float t = 0.0f;
-                for (int i = lane; i < a.head_len; i += 32) {
-                    const float v = xs[vec_slot(h * a.head_len + i, p.half)];
-                    t += v * v;
+        float* const hinv = reinterpret_cast<float*>(vsmem + p.off_head);  // one entry per head of the segments that norm by head
+        int heads0 = 0;
+        float joint[kMaxSegments] = {};
+        __syncthreads();
+#pragma unroll
+        for (int j = 0; j < kMaxSegments; ++j) {
+            if (j >= a.n_seg) break;
+            const GateSegment& g = a.seg[j];
+            if (g.norm == KMLL_OUT_NORM_JOINT) {
+                joint[j] = inv_rms(block_sum(s[j], scratch), g.cols, g.eps);
+            } else if (g.norm != KMLL_OUT_NORM_NONE) {
+                const int nh = g.cols / g.head_len;
+                for (int h = warp; h < nh; h += kVWarps) {
+                    float t = 0.0f;
+                    for (int i = lane; i < g.head_len; i += 32) {
+                        const float v = xs[vec_slot(g.begin + h * g.head_len + i, p.half)];
+                        t += v * v;
+                    }
+                    t = warp_sum(t);
+                    if (lane == 0) hinv[heads0 + h] = inv_rms(t, g.head_len, g.eps);
                 }
-                t = warp_sum(t);
-                if (lane == 0) hinv[h] = inv_rms(t, a.head_len, a.eps);
+                heads0 += nh;
             }
-            __syncthreads();
-            for (int k = tid; k < a.K; k += kVThreads) xs[vec_slot(k, p.half)] *= hinv[k / a.head_len] * apply_act(a.gate[k], a.gate_act);
         }
+        __syncthreads();
+        heads0 = 0;
+        int covered = 0;
+#pragma unroll
+        for (int j = 0; j < kMaxSegments; ++j) {
+            if (j >= a.n_seg) break;
+            const GateSegment& g = a.seg[j];
+            for (int k = covered + tid; k < g.begin; k += kVThreads) xs[vec_slot(k, p.half)] = 0.0f;
+            covered = g.begin + g.cols;
+            const float* const gate = static_cast<const float*>(g.gate);
+            for (int i = tid; i < g.cols; i += kVThreads) {
+                float f = g.scale;
+                if (g.norm == KMLL_OUT_NORM_JOINT) {
+                    f *= joint[j] * bf16_bits_to_f32(g.norm_w[i]);
+                } else if (g.norm != KMLL_OUT_NORM_NONE) {
+                    const int h = i / g.head_len;
+                    f *= hinv[heads0 + h];
+                    if (g.norm == KMLL_OUT_NORM_HEAD_WEIGHTED) f *= bf16_bits_to_f32(g.norm_w[i - h * g.head_len]);
+                }
+                if (gate != nullptr) f *= apply_act(gate[g.gate_len == 1 ? i : i / g.gate_len], g.act);
+                xs[vec_slot(g.begin + i, p.half)] *= f;
+            }
+            if (g.norm == KMLL_OUT_NORM_PER_HEAD || g.norm == KMLL_OUT_NORM_HEAD_WEIGHTED) heads0 += g.cols / g.head_len;
+        }
+        for (int k = covered + tid; k < a.K; k += kVThreads) xs[vec_slot(k, p.half)] = 0.0f;
     } else {
         for (int k = tid; k < kpad; k += kVThreads) xs[vec_slot(k, p.half)] = k < a.K ? a.x[k] : 0.0f;
     }
@@ -193,11 +239,24 @@ __global__ void __launch_bounds__(kVThreads, 2) bf16_matvec_kernel(const MatvecA
     const int nw = p.kpieces < kVWarps ? p.kpieces : kVWarps;
     float best = -INFINITY;
     uint32_t best_row = 0xffffffffu;
+    if (a.pair_act != 0) {
+        for (int r = 2 * tid; r < nrows; r += 2 * kVThreads) {
+            float gate = 0.0f, v = 0.0f;
+            for (int w = 0; w < nw; ++w) {
+                const float2 t = *reinterpret_cast<const float2*>(part + w * p.rows_cap + r);
+                gate += t.x;
+                v += t.y;
+            }
+            a.y[(r0 + r) >> 1] = apply_act(gate, a.pair_act) * v;
+        }
+        return;
+    }
     for (int r = tid; r < nrows; r += kVThreads) {
         float v = 0.0f;
         for (int w = 0; w < nw; ++w) v += part[w * p.rows_cap + r];
         const int row = r0 + r;
         if (row < a.silu_rows) v = act_silu(v);
+        v *= a.out_scale;
         if (a.residual != nullptr) v += a.residual[row];
         a.y[row] = v;
         if (top1_better(v, (uint32_t)row, best, best_row)) { best = v; best_row = (uint32_t)row; }
@@ -261,7 +320,10 @@ int bf16_matvec(cudaStream_t stream, const Bf16Matvec& a) {
     p.a = a;
     p.kpieces = (a.K + kVPiece - 1) / kVPiece;
     p.half = p.kpieces * kVPiece / 2;
-    p.n_heads = (a.pro == PRO_GATED && a.norm_w == nullptr) ? (a.K + a.head_len - 1) / a.head_len : 0;
+    if (a.pair_act != 0 && ((a.rows & 1) != 0 || a.packed != nullptr || a.residual != nullptr)) return fail(KMLL_ERR_SHAPE, "bf16_matvec: %d rows are not pairs", a.rows);
+    p.n_heads = 0;
+    for (int j = 0; a.pro == PRO_GATED && j < a.n_seg; ++j)
+        if (a.seg[j].norm == KMLL_OUT_NORM_PER_HEAD || a.seg[j].norm == KMLL_OUT_NORM_HEAD_WEIGHTED) p.n_heads += a.seg[j].cols / a.seg[j].head_len;
     const size_t ring = (size_t)kVDepth * kVThreads * 16, xbytes = (size_t)p.kpieces * kVPiece * 4, hbytes = ((size_t)p.n_heads * 4 + 15) & ~(size_t)15;
     p.off_x = (int)ring;
     p.off_head = (int)(ring + xbytes);
@@ -270,7 +332,8 @@ int bf16_matvec(cudaStream_t stream, const Bf16Matvec& a) {
     int grid = a.rows / 4 < 148 ? (a.rows + 3) / 4 : 148;
     size_t smem = 0;
     for (;; grid += 148) {
-        p.rows_cap = ((a.rows + grid - 1) / grid + kVRows - 1) / kVRows * kVRows;
+        const int unit = a.pair_act != 0 ? 2 : 1;
+        p.rows_cap = (unit * ((a.rows / unit + grid - 1) / grid) + kVRows - 1) / kVRows * kVRows;
         smem = ring + xbytes + hbytes + (size_t)kVWarps * p.rows_cap * 4;
         if (smem <= 220 * 1024) break;
         if (p.rows_cap <= kVRows) return fail(KMLL_ERR_UNSUPPORTED, "bf16_matvec: in_dim %d does not fit in shared memory", a.K);
@@ -296,7 +359,8 @@ constexpr int kHThreads = (2 + kHEpiWarps) * 32;  // warp 0: TMA, warp 1: MMA, w
 struct GemmBf16Params {
     int rows, K, T, n_block, stages, row_tiles, x_tiles, tiles, ksplit;
     void* out;
-    int out_bf16, ldo, silu_rows;
+    int out_bf16, ldo, silu_rows, pair_act;
+    float out_scale;
     const float* residual;
     float* partial;          // ksplit > 1 (one item per block): [tiles][ksplit][n_block][128]
     unsigned int* counters;  // [tiles], zero between launches
@@ -384,6 +448,7 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
         auto finish = [&](int t, int row, float v, bool act) {
             const size_t o = (size_t)t * p.ldo + row;
             if (act) v = act_silu(v);
+            v *= p.out_scale;
             if (p.residual != nullptr) v += p.residual[o];
             if (p.out_bf16) static_cast<uint16_t*>(p.out)[o] = f32_to_bf16_bits(v);
             else static_cast<float*>(p.out)[o] = v;
@@ -411,8 +476,12 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                    if (part != nullptr) part[(size_t)(c0 + j) * kHRows + rl] = __uint_as_float(d[j]);
-                    else if (live && t0 + c0 + j < p.T) finish(t0 + c0 + j, row, __uint_as_float(d[j]), act);
+                    if (part != nullptr) {
+                        part[(size_t)(c0 + j) * kHRows + rl] = __uint_as_float(d[j]);
+                    } else if (p.pair_act != 0) {  // even lanes hold the gate, odd lanes its value
+                        const float v = __shfl_xor_sync(0xffffffffu, __uint_as_float(d[j]), 1);
+                        if (live && (lane & 1) == 0 && t0 + c0 + j < p.T) finish(t0 + c0 + j, row >> 1, apply_act(__uint_as_float(d[j]), p.pair_act) * v, false);
+                    } else if (live && t0 + c0 + j < p.T) finish(t0 + c0 + j, row, __uint_as_float(d[j]), act);
                 }
             }
             tcgen05_fence_before();
@@ -440,9 +509,15 @@ __global__ void __launch_bounds__(kHThreads, 1) linear_gemm_bf16_kernel(const Ge
 #pragma unroll
                             for (int z = 0; z < 8; ++z) { v[0] += x[z].x; v[1] += x[z].y; v[2] += x[z].z; v[3] += x[z].w; }
                         }
+                        if (p.pair_act != 0) {
 #pragma unroll
-                        for (int e = 0; e < 4; ++e)
-                            if (row0 + r + e < p.rows) finish(t0 + c, row0 + r + e, v[e], row0 + r + e < p.silu_rows);
+                            for (int e = 0; e < 4; e += 2)
+                                if (row0 + r + e < p.rows) finish(t0 + c, (row0 + r + e) >> 1, apply_act(v[e], p.pair_act) * v[e + 1], false);
+                        } else {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e)
+                                if (row0 + r + e < p.rows) finish(t0 + c, row0 + r + e, v[e], row0 + r + e < p.silu_rows);
+                        }
                     }
                     if (tid == 64) p.counters[tile] = 0u;
                 }
@@ -484,6 +559,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const Bf16Gemm g) {
         }
         __syncthreads();
     }
+    float* const out = static_cast<float*>(g.out);
+    if (g.pair_act != 0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int t = t0 + ty * 4 + i, row = r0 + tx * 4 + j;
+                if (t < g.T && row < g.rows) out[(size_t)t * g.ldo + (row >> 1)] = apply_act(acc[i][j], g.pair_act) * acc[i][j + 1];
+            }
+        return;
+    }
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -492,15 +578,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const Bf16Gemm g) {
             if (t < g.T && row < g.rows) {
                 float v = acc[i][j];
                 if (row < g.silu_rows) v = act_silu(v);
+                v *= g.out_scale;
                 const size_t o = (size_t)t * g.ldo + row;
                 if (g.residual != nullptr) v += g.residual[o];
-                static_cast<float*>(g.out)[o] = v;
+                out[o] = v;
             }
         }
 }
 
 int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g) {
     if (g.T <= 0 || g.rows <= 0 || g.K <= 0 || g.ldw < g.K || g.ldx < g.K) return fail(KMLL_ERR_SHAPE, "bf16_gemm: T %d, rows %d, K %d", g.T, g.rows, g.K);
+    if (g.pair_act != 0 && ((g.rows & 1) != 0 || g.residual != nullptr)) return fail(KMLL_ERR_SHAPE, "bf16_gemm: %d rows are not pairs", g.rows);
     if (g.x_f32) {
         if (g.out_bf16) return fail(KMLL_ERR_UNSUPPORTED, "bf16_gemm: f32 activations give f32 results");
         cudaError_t e = launch(gemm_f32_kernel, dim3((g.rows + 63) / 64, (g.T + 63) / 64), dim3(256), 0, stream, true, g);
@@ -513,6 +601,7 @@ int bf16_gemm(cudaStream_t stream, const Bf16Gemm& g) {
     memset(&p, 0, sizeof(p));
     p.rows = g.rows; p.K = g.K; p.T = g.T;
     p.out = g.out; p.out_bf16 = g.out_bf16; p.ldo = g.ldo; p.residual = g.residual; p.silu_rows = g.silu_rows;
+    p.pair_act = g.pair_act; p.out_scale = g.out_scale;
     p.row_tiles = (g.rows + kHRows - 1) / kHRows;
     // rows of x per tile: the size whose rounds over 148 SMs cost least (measured with K = 4096: 24 us at 64 rows, 32 at 256)
     const int nmax = g.T >= kHMaxN ? kHMaxN : (g.T + 15) / 16 * 16;

@@ -7,7 +7,7 @@ import json
 import math
 
 from . import runtime as rt
-from .checkpoint import CheckpointError, ModelWeights, YarnRopeConfig
+from .checkpoint import CheckpointError, ModelWeights, YarnRopeConfig, load_layered
 
 
 def inverse_frequencies(dims: int, base: float, yarn: YarnRopeConfig | None = None):
@@ -106,12 +106,7 @@ def tensor_names(config: dict):
 
 
 def load(model_dir: str, config: dict, max_seq_len: int | None = None, compute_f32: bool = False) -> rt.LayeredDecoder:
-    cfg = layered_config(config, max_seq_len, compute_f32)
-    weights = ModelWeights(model_dir)
-    dec = rt.LayeredDecoder(cfg)
-    for name, layer, tensor in tensor_names(config):
-        dec.set_tensor(layer, tensor, weights.read(name, "BF16", cfg.tensor_shape(layer, tensor)))
-    return dec
+    return load_layered(ModelWeights(model_dir), layered_config(config, max_seq_len, compute_f32), tensor_names(config))
 
 
 def load_dir(model_dir: str, **kw) -> rt.LayeredDecoder:

@@ -7,10 +7,11 @@ import os
 
 from . import pefisun
 from . import runtime as rt
+from . import somopel
 from .checkpoint import CheckpointError, load_decoder
 
 # architecture -> loader(model_dir, config, max_seq_len, compute_f32)
-ARCHITECTURES = {"Pefisun": pefisun.load}
+ARCHITECTURES = {"Pefisun": pefisun.load, "Somopel": somopel.load}
 
 
 def read_config(model_dir: str) -> dict:

@@ -20,10 +20,15 @@ FORMAT_BF16 = 2  # layered decoders
 
 T_ATTENTION_NORM, T_WQ, T_WK, T_WV, T_WO, T_FFN_NORM, T_W1, T_W3, T_W2, T_FINAL_NORM, T_EMBEDDING, T_OUTPUT, T_Q_NORM, T_K_NORM = range(14)
 T_POSITION, T_GATE, T_MIX_NORM, T_DKV, T_DKV_NORM, T_UK, T_UV, T_ACT = range(14, 22)  # layered decoders
-MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION = 1, 2
-ACT_NONE, ACT_SILU, ACT_SIGMOID = range(3)
-MLP_NONE, MLP_POLYNORM = range(2)
-OUT_NORM_PER_HEAD, OUT_NORM_JOINT = range(2)
+(T_ATTENTION_NORM_BIAS, T_FFN_NORM_BIAS, T_FINAL_NORM_BIAS, T_EMBED_NORM, T_EMBED_NORM_BIAS, T_DECAY_DOWN, T_DECAY_UP, T_DECAY_BIAS, T_DECAY_LOG, T_BETA,
+ T_Q_CONV, T_K_CONV, T_V_CONV, T_GATE_DOWN, T_GATE_UP) = range(22, 37)
+T_BESIDE = 64  # added to a tensor id: the layer's second mixer
+MIXER_NONE, MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION, MIXER_ATTENTION, MIXER_GATED_LINEAR = range(5)
+ACT_NONE, ACT_SILU, ACT_SIGMOID, ACT_GELU_TANH = range(4)
+MLP_NONE, MLP_POLYNORM, MLP_GATED = range(3)
+NORM_RMS, NORM_LAYER = range(2)
+OUT_NORM_PER_HEAD, OUT_NORM_JOINT, OUT_NORM_HEAD_WEIGHTED, OUT_NORM_NONE = range(4)
+DECAY_LOGISTIC, DECAY_SOFTPLUS = 1, 2
 
 
 class _Config(C.Structure):
@@ -237,14 +242,21 @@ class Decoder:
         return int(self._lib.kmll_decoder_resident_bytes(self._h))
 
 
-class _LayerSpec(C.Structure):
+class _MixerSpec(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("mixer", "heads", "dim", "vdim", "kv_rank", "rot_dim", "window")] + [("score_scale", C.c_float)] + \
-               [(n, C.c_int) for n in ("qkv_act", "gate_act", "out_norm")] + [("key_scale", C.c_float), ("mlp", C.c_int), ("ff", C.c_int)]
+               [(n, C.c_int) for n in ("qkv_act", "gate_act", "out_norm")] + [("key_scale", C.c_float)] + \
+               [(n, C.c_int) for n in ("kv_heads", "chunk", "head_gate")] + [("out_scale", C.c_float), ("q_scale", C.c_float), ("decay", C.c_int)] + \
+               [("decay_tau", C.c_float)] + [(n, C.c_int) for n in ("decay_rank", "delta", "conv")] + [("unit_eps", C.c_float), ("gate_rank", C.c_int)]
+
+
+class _LayerSpec(C.Structure):
+    _fields_ = [("mixers", _MixerSpec * 2), ("mlp", C.c_int), ("mlp_act", C.c_int), ("ff", C.c_int)]
 
 
 class _LayeredConfig(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("n_layers", "dim", "vocab_size", "max_seq_len", "position_rows")] + \
-               [("norm_eps", C.c_float), ("norm_offset", C.c_float), ("compute_f32", C.c_int)]
+               [("norm_eps", C.c_float), ("norm_offset", C.c_float), ("compute_f32", C.c_int), ("norm", C.c_int), ("embed_scale", C.c_float),
+                ("embed_norm", C.c_int), ("logit_scale", C.c_float), ("tie_output", C.c_int)]
 
 
 @dataclass
@@ -255,8 +267,8 @@ class Rotation:
 
 
 @dataclass
-class LayerSpec:
-    """One layer of a layered decoder (kmll_layer_spec); unused fields keep their defaults."""
+class MixerSpec:
+    """One mixer of a layer (kmll_mixer_spec); unused fields keep their defaults."""
     mixer: int
     heads: int
     dim: int
@@ -269,14 +281,81 @@ class LayerSpec:
     gate_act: int = ACT_SILU
     out_norm: int = OUT_NORM_PER_HEAD
     key_scale: float = 1.0
+    kv_heads: int = 0
+    chunk: int = 0
+    head_gate: int = 0
+    out_scale: float = 1.0
+    q_scale: float = 1.0
+    decay_kind: int = 0          # gated linear attention: DECAY_*
+    decay_tau: float = 1.0
+    decay_rank: int = 0
+    delta: int = 0
+    conv: int = 0
+    unit_eps: float = 0.0
+    gate_rank: int = 0
+    rotation: Rotation | None = None  # needed when rot_dim > 0
+    decay: list | None = None         # per head, linear attention with a fixed decay
+
+    def _mixer(self) -> _MixerSpec:
+        return _MixerSpec(self.mixer, self.heads, self.dim, self.vdim, self.kv_rank, self.rot_dim, self.window, self.score_scale, self.qkv_act,
+                          self.gate_act, self.out_norm, self.key_scale, self.kv_heads, self.chunk, self.head_gate, self.out_scale, self.q_scale,
+                          self.decay_kind, self.decay_tau, self.decay_rank, self.delta, self.conv, self.unit_eps, self.gate_rank)
+
+    def tensor_shapes(self, width: int) -> dict:
+        """tensor id -> shape of the tensors this mixer has."""
+        k, v, g, d, dv = self.heads * self.dim, self.heads * self.vdim, self.kv_heads or self.heads, self.dim, self.vdim
+        out = {T_WO: (width, v)}
+        if self.mixer == MIXER_LATENT_ATTENTION:
+            out.update({T_WQ: (k + self.heads * self.rot_dim, width), T_DKV: (self.kv_rank + self.rot_dim, width), T_DKV_NORM: (self.kv_rank,),
+                        T_UK: (k, self.kv_rank), T_UV: (v, self.kv_rank)})
+        elif self.mixer == MIXER_ATTENTION:
+            out.update({T_WQ: (k, width), T_WK: (g * d, width), T_WV: (g * dv, width)})
+            if self.head_gate:
+                out[T_GATE] = (self.heads, width)
+        else:
+            gated = self.mixer == MIXER_GATED_LINEAR
+            nk = g * d if gated else k
+            out.update({T_WQ: (nk, width), T_WK: (nk, width), T_WV: (v, width)})
+            if self.out_norm in (OUT_NORM_JOINT, OUT_NORM_HEAD_WEIGHTED):
+                out[T_MIX_NORM] = (v if self.out_norm == OUT_NORM_JOINT else dv,)
+            if gated and self.gate_rank:
+                out.update({T_GATE_DOWN: (self.gate_rank, width), T_GATE_UP: (v, self.gate_rank)})
+            else:
+                out[T_GATE] = (v, width)
+            if gated:
+                out.update({T_DECAY_DOWN: (self.decay_rank, width), T_DECAY_UP: (k, self.decay_rank), T_DECAY_BIAS: (k,)})
+                if self.decay_kind == DECAY_SOFTPLUS:
+                    out[T_DECAY_LOG] = (self.heads,)
+                if self.delta:
+                    out[T_BETA] = (self.heads, width)
+                if self.conv:
+                    out.update({T_Q_CONV: (nk, self.conv), T_K_CONV: (nk, self.conv), T_V_CONV: (v, self.conv)})
+        return out
+
+
+@dataclass
+class LayerSpec(MixerSpec):
+    """One layer of a layered decoder (kmll_layer_spec): its mixer, perhaps a second one beside it, and its feed-forward."""
     mlp: int = MLP_NONE
     ff: int = 0
-    rotation: Rotation | None = None  # needed when rot_dim > 0
-    decay: list | None = None         # per head, linear attention
+    mlp_act: int = ACT_NONE
+    beside: MixerSpec | None = None
 
     def _c(self) -> _LayerSpec:
-        return _LayerSpec(self.mixer, self.heads, self.dim, self.vdim, self.kv_rank, self.rot_dim, self.window, self.score_scale, self.qkv_act,
-                          self.gate_act, self.out_norm, self.key_scale, self.mlp, self.ff)
+        second = self.beside._mixer() if self.beside is not None else _MixerSpec()
+        return _LayerSpec((_MixerSpec * 2)(self._mixer(), second), self.mlp, self.mlp_act, self.ff)
+
+    def layer_shapes(self, width: int, norm: int) -> dict:
+        """tensor id -> shape of every tensor of the layer."""
+        out = {T_ATTENTION_NORM: (width,), **self.tensor_shapes(width)}
+        if self.beside is not None:
+            out.update({T_BESIDE + t: s for t, s in self.beside.tensor_shapes(width).items()})
+        if self.mlp != MLP_NONE:
+            out.update({T_FFN_NORM: (width,), T_W3: (self.ff, width), T_W2: (width, self.ff)})
+            out.update({T_W1: (self.ff, width)} if self.mlp == MLP_GATED else {T_ACT: (4,)})
+        if norm == NORM_LAYER:
+            out.update({b: out[t] for t, b in ((T_ATTENTION_NORM, T_ATTENTION_NORM_BIAS), (T_FFN_NORM, T_FFN_NORM_BIAS)) if t in out})
+        return out
 
 
 @dataclass
@@ -289,23 +368,29 @@ class LayeredConfig:
     norm_eps: float = 1.0e-5
     norm_offset: float = 0.0  # 1.0: norm weights are stored around zero
     compute_f32: bool = False
+    norm: int = NORM_RMS
+    embed_scale: float = 1.0
+    embed_norm: bool = False
+    logit_scale: float = 1.0
+    tie_output: bool = False  # the logits read the embedding table
 
     format = FORMAT_BF16
 
     def _c(self) -> _LayeredConfig:
         return _LayeredConfig(len(self.layers), self.dim, self.vocab_size, self.max_seq_len, self.position_rows, self.norm_eps, self.norm_offset,
-                              1 if self.compute_f32 else 0)
+                              1 if self.compute_f32 else 0, self.norm, self.embed_scale, 1 if self.embed_norm else 0, self.logit_scale,
+                              1 if self.tie_output else 0)
 
     def tensor_shape(self, layer: int, tensor: int):
+        if layer != -1:
+            return self.layers[layer].layer_shapes(self.dim, self.norm)[tensor]
         d, v = self.dim, self.vocab_size
-        if layer == -1:
-            return {T_EMBEDDING: (v, d), T_POSITION: (self.position_rows, d), T_FINAL_NORM: (d,), T_OUTPUT: (v, d)}[tensor]
-        s = self.layers[layer]
-        latent = s.mixer == MIXER_LATENT_ATTENTION
-        return {T_ATTENTION_NORM: (d,), T_FFN_NORM: (d,), T_WQ: (s.heads * (s.dim + (s.rot_dim if latent else 0)), d), T_WK: (s.heads * s.dim, d),
-                T_WV: (s.heads * s.vdim, d), T_GATE: (s.heads * s.vdim, d), T_MIX_NORM: (s.heads * s.vdim,), T_WO: (d, s.heads * s.vdim),
-                T_DKV: (s.kv_rank + s.rot_dim, d), T_DKV_NORM: (s.kv_rank,), T_UK: (s.heads * s.dim, s.kv_rank), T_UV: (s.heads * s.vdim, s.kv_rank),
-                T_W3: (s.ff, d), T_W2: (d, s.ff), T_ACT: (4,)}[tensor]
+        return {T_EMBEDDING: (v, d), T_POSITION: (self.position_rows, d), T_OUTPUT: (v, d)}.get(tensor, (d,))
+
+    def weight_elements(self) -> int:
+        """Weights that a decode step streams: every matrix of the layers and the output matrix."""
+        per_layer = sum(int(np.prod(s)) for l in self.layers for s in l.layer_shapes(self.dim, self.norm).values() if len(s) == 2)
+        return per_layer + self.vocab_size * self.dim
 
 
 class LayeredDecoder(Decoder):
@@ -333,7 +418,10 @@ class LayeredDecoder(Decoder):
 
     def set_tensor(self, layer: int, tensor: int, values: np.ndarray, scales=None) -> None:
         """bf16 bit patterns (uint16)."""
-        shape = self.cfg.tensor_shape(layer, tensor)
+        try:
+            shape = self.cfg.tensor_shape(layer, tensor)
+        except (KeyError, IndexError):
+            raise KmllError(-2, f"layer {layer} has no tensor {tensor}") from None
         if values.dtype != np.uint16 or tuple(values.shape) != tuple(shape):
             raise KmllError(-2, f"tensor {tensor} of layer {layer}: {values.dtype} {values.shape}, expected uint16 {shape}")
         super().set_tensor(layer, tensor, values)
@@ -401,5 +489,5 @@ def unpack_top1(packed: int):
     return int(token), float(logit)
 
 
-__all__ = ["Decoder", "LayeredDecoder", "BatchDecoder", "DecoderConfig", "LayeredConfig", "LayerSpec", "Rotation", "KmllError", "FORMAT_RS_I8",
+__all__ = ["Decoder", "LayeredDecoder", "BatchDecoder", "DecoderConfig", "LayeredConfig", "LayerSpec", "MixerSpec", "Rotation", "KmllError", "FORMAT_RS_I8",
            "FORMAT_W4G128", "FORMAT_BF16", "unpack_top1"]

@@ -142,8 +142,13 @@ def test_struct_mirrors_match_the_library():
     assert handle.kmll_layer_spec_bytes() == C.sizeof(rt._LayerSpec)
     assert handle.kmll_layered_config_bytes() == C.sizeof(rt._LayeredConfig)
     s = rt.LayerSpec(mixer=1, heads=2, dim=3, vdim=4, kv_rank=5, rot_dim=6, window=7, score_scale=0.5, qkv_act=1, gate_act=2, out_norm=1, key_scale=0.25,
-                     mlp=1, ff=9)._c()
-    assert [getattr(s, n) for n, _ in rt._LayerSpec._fields_] == [1, 2, 3, 4, 5, 6, 7, 0.5, 1, 2, 1, 0.25, 1, 9]
+                     mlp=1, ff=9, mlp_act=3)._c()
+    first = [getattr(s.mixers[0], n) for n, _ in rt._MixerSpec._fields_]
+    assert first[:12] == [1, 2, 3, 4, 5, 6, 7, 0.5, 1, 2, 1, 0.25] and (s.mlp, s.ff, s.mlp_act, s.mixers[1].mixer) == (1, 9, 3, rt.MIXER_NONE)
+    s = rt.LayerSpec(3, 2, 3, 4, beside=rt.MixerSpec(4, 6, 7, 8, kv_heads=3, chunk=9, head_gate=1, out_scale=0.5, q_scale=0.25, decay_kind=2, decay_tau=4.0,
+                                                     decay_rank=10, delta=1, conv=11, unit_eps=0.125, gate_rank=12))._c()
+    second = [getattr(s.mixers[1], n) for n, _ in rt._MixerSpec._fields_]
+    assert s.mixers[0].mixer == 3 and second[:4] == [4, 6, 7, 8] and second[12:] == [3, 9, 1, 0.5, 0.25, 2, 4.0, 10, 1, 11, 0.125, 12]
 
 
 @pytest.mark.parametrize("change", [dict(heads=0), dict(rot_dim=3), dict(mixer=7), dict(mixer=rt.MIXER_LINEAR_ATTENTION, rot_dim=8, dim=4), dict(kv_rank=0),

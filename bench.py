@@ -263,7 +263,7 @@ def run_suite(args):
     """The operator suites of kmll_b200.microbench with the CPU port of each operator timed beside it."""
     from kmll_b200 import microbench as mb
     cpu = None if args.no_cpu else cpu_operator_us
-    {"chain4096": mb.suite_chain4096, "micro": mb.suite_micro, "gemm_sweep": mb.suite_gemm_sweep, "layered": mb.suite_layered}[args.suite](args.suite_reps, cpu)
+    {"chain4096": mb.suite_chain4096, "micro": mb.suite_micro, "gemm_sweep": mb.suite_gemm_sweep, "layered": mb.suite_layered, "somopel": mb.suite_somopel}[args.suite](args.suite_reps, cpu)
 
 
 def workload_config(n_gpus):
@@ -622,9 +622,10 @@ def main():
     ap.add_argument("--no-batch16", action="store_true", help="skip the batch-16 leg")
     ap.add_argument("--no-rsi8", action="store_true", help="skip the RS-I8 (the reference's own format) decode leg")
     ap.add_argument("--no-kvbf16", action="store_true", help="skip the leg that keeps the KV cache in bf16")
-    ap.add_argument("--suite", default="", choices=["", "chain4096", "micro", "gemm_sweep", "layered"],
+    ap.add_argument("--suite", default="", choices=["", "chain4096", "micro", "gemm_sweep", "layered", "somopel"],
                     help="instead of the decode bench: one operator suite of kmll_b200.microbench, CPU port timed beside each line (layered: the kernels "
-                         "and decode / prompt throughput of the layered decoders beside the uniform decoder, no CPU port)")
+                         "and decode / prompt throughput of the layered decoders beside the uniform decoder; somopel: those of the Somopel design "
+                         "beside the other layered design; both without a CPU port)")
     ap.add_argument("--suite-reps", type=int, default=20)
     ap.add_argument("--profile", nargs="?", const="decode", default=None, choices=["decode", "batch16"],
                     help="bracket the timed batch-1 decode loop (default) or the timed batch-16 loop with cudaProfilerStart/Stop (for ncu --profile-from-start off)")

@@ -283,6 +283,47 @@ int kmll_decoder_reset(kmll_decoder_t dec, kmll_stream_t stream);
  * detaches); parity checks. */
 int kmll_layered_tap(kmll_decoder_t dec, float* residual_device);
 
+/* Operators of the layered decoders that take a mixer description (more of them in kmll_b200.h).
+ *
+ * y = W norm(x) * out_scale, one row of x in f32; norm: KMLL_NORM_*, norm_weight null: none.  pair_act != 0: rows 2 i and 2 i + 1
+ * of w are a gate and its value, y[i] = pair_act(gate) * value (rows / 2 results). */
+int kmll_normed_linear_bf16(kmll_stream_t stream, const float* x, const uint16_t* w, int pitch, int rows, int cols, int norm, const uint16_t* norm_weight,
+                            const uint16_t* norm_bias, float eps, int pair_act, float out_scale, float* y);
+/* The same pairs for a batch of rows: out [batch, rows / 2] in the type of x (workspace as for kmll_linear_batched_bf16). */
+int kmll_pair_linear_batched_bf16(kmll_stream_t stream, const void* x, int x_f32, int ldx, int batch, const uint16_t* w, int pitch, int rows, int cols,
+                                  int pair_act, void* workspace, void* out);
+/* rows [batch, dim] f32 normed into bf16 */
+int kmll_norm_rows_bf16(kmll_stream_t stream, const float* x, int batch, int dim, int norm, const uint16_t* weight, const uint16_t* bias, float eps, uint16_t* out);
+/* y = W z (+ residual) for one row, where z is the outputs of one or two mixers side by side in x [cols] (the second from the next
+ * multiple of 8 on): each normed, gated and scaled as its description says.  gates: f32, one pointer per mixer (null: none), heads
+ * or heads*vdim values. */
+int kmll_mixer_output_linear_bf16(kmll_stream_t stream, const kmll_mixer_spec* mixers, int n_mixers, const float* x, const uint16_t* const* norm_weights,
+                                  const float* const* gates, float eps, const uint16_t* w, int pitch, int rows, int cols, const float* residual, float* y);
+/* Grouped attention over a cache [max_seq, pitch] (f32 or bf16): keys of every key / value head, each padded to a multiple of 8
+ * entries (zeros), then the values likewise.  in [tokens, ld]: q, k, v at their column offsets.  The tokens' cache rows are
+ * written, then every position they see is attended.  One token at *position_device with a workspace: the decode form (f32 input,
+ * bf16 cache); bf16 input and cache: the prompt form; else plain f32 arithmetic.  workspace: _workspace_bytes() bytes whose first
+ * 4096 are zero before the first call (each call leaves them so). */
+size_t kmll_grouped_attention_workspace_bytes(const kmll_mixer_spec* mixer);
+int kmll_grouped_attention(kmll_stream_t stream, const kmll_mixer_spec* mixer, const void* in, int in_f32, int ld, int q_off, int k_off, int v_off, int tokens,
+                           int position, const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, void* workspace, float* out, int ldo);
+/* Gated linear attention.  in [tokens, ld]: q, k, v, the decay factor (decay_rank), the logits of beta (heads) and the gate factor
+ * (gate_rank) at offsets[0 .. 5].  conv [q | k | v channels][taps]; ring [taps][channels] f32 holds the inputs of earlier
+ * positions.  state [heads, dim, vdim] f32 and ring are updated.  scratch == null: token after token in f32, the low-rank gate goes
+ * to gate [tokens, heads*vdim]; else (bf16 input, dim up to 128, 4 or more tokens) chunks of 64 tokens on the tensor cores,
+ * _scratch_floats() floats, no gate. */
+typedef struct {
+    const uint16_t *decay_up; /* [heads*dim, decay_pitch] */
+    int decay_pitch;
+    const uint16_t *decay_bias, *decay_log, *conv;
+    const uint16_t *gate_up;  /* [heads*vdim, gate_pitch] */
+    int gate_pitch;
+} kmll_gated_linear_weights;
+size_t kmll_gated_linear_scratch_floats(const kmll_mixer_spec* mixer, int tokens);
+int kmll_gated_linear_attention(kmll_stream_t stream, const kmll_mixer_spec* mixer, const kmll_gated_linear_weights* weights, const void* in, int in_f32, int ld,
+                                const int* offsets, int tokens, int position, const int* position_device, float* state, float* ring, float* scratch, float* gate,
+                                float* out, int ldo);
+
 /* ---- on-disk archive of the quantized linear weights ---------------------------------------------------------
  * The directory layout of kmll's quantization export, so an archive written by either side loads on the other:
  *   manifest.json with "quantization": "row-symmetric-int8-with-f32-row-scales" (crates/inference/src/model.rs:9047-9053),

@@ -130,4 +130,121 @@ int kmll_latent_attention_prefill(kmll_stream_t s, const uint16_t* in, int ld, i
     return latent_attention_prefill(as_stream(s), a);
 }
 
+int kmll_normed_linear_bf16(kmll_stream_t s, const float* x, const uint16_t* w, int pitch, int rows, int cols, int norm, const uint16_t* norm_weight,
+                            const uint16_t* norm_bias, float eps, int pair_act, float out_scale, float* y) {
+    KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(y);
+    if (norm == KMLL_NORM_LAYER && norm_weight != nullptr) KMLL_REQUIRE_PTR(norm_bias);
+    Bf16Matvec v = base(x, w, pitch, rows, cols, nullptr, y);
+    v.pair_act = pair_act;
+    v.out_scale = out_scale;
+    if (norm_weight != nullptr) { v.pro = PRO_NORM; v.norm = NormArgs{norm, norm_weight, norm_bias, 0.0f, eps}; }
+    return bf16_matvec(as_stream(s), v);
+}
+
+int kmll_pair_linear_batched_bf16(kmll_stream_t s, const void* x, int x_f32, int ldx, int batch, const uint16_t* w, int pitch, int rows, int cols, int pair_act,
+                                  void* workspace, void* out) {
+    KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(out);
+    KMLL_REQUIRE(pair_act != KMLL_ACT_NONE, "pair_linear_batched: no activation");
+    Bf16Gemm g;
+    memset(&g, 0, sizeof(g));
+    g.x = x; g.x_f32 = x_f32; g.ldx = ldx; g.T = batch; g.K = cols; g.w = w; g.rows = rows; g.ldw = pitch; g.out = out; g.out_bf16 = !x_f32; g.ldo = rows / 2;
+    g.pair_act = pair_act; g.out_scale = 1.0f;
+    if (workspace != nullptr) {
+        g.counters = static_cast<unsigned int*>(workspace);
+        g.partial = static_cast<float*>(workspace) + 128;
+    }
+    return bf16_gemm(as_stream(s), g);
+}
+
+int kmll_norm_rows_bf16(kmll_stream_t s, const float* x, int batch, int dim, int norm, const uint16_t* weight, const uint16_t* bias, float eps, uint16_t* out) {
+    KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(weight); KMLL_REQUIRE_PTR(out);
+    KMLL_REQUIRE(batch > 0 && dim > 0, "norm_rows: bad shape");
+    if (norm == KMLL_NORM_LAYER) KMLL_REQUIRE_PTR(bias);
+    return norm_rows(as_stream(s), x, dim, nullptr, batch, NormArgs{norm, weight, bias, 0.0f, eps}, 0, out, dim);
+}
+
+int kmll_mixer_output_linear_bf16(kmll_stream_t s, const kmll_mixer_spec* mixers, int n_mixers, const float* x, const uint16_t* const* norm_weights,
+                                  const float* const* gates, float eps, const uint16_t* w, int pitch, int rows, int cols, const float* residual, float* y) {
+    KMLL_REQUIRE_PTR(mixers); KMLL_REQUIRE_PTR(x); KMLL_REQUIRE_PTR(norm_weights); KMLL_REQUIRE_PTR(gates); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(y);
+    KMLL_REQUIRE(n_mixers == 1 || n_mixers == 2, "mixer_output_linear: %d mixers", n_mixers);
+    Bf16Matvec v = base(x, w, pitch, rows, cols, residual, y);
+    v.pro = PRO_GATED;
+    v.n_seg = n_mixers;
+    int at = 0;
+    for (int i = 0; i < n_mixers; ++i) {
+        const kmll_mixer_spec& m = mixers[i];
+        KMLL_REQUIRE(m.heads > 0 && m.vdim > 0, "mixer_output_linear: bad shape");
+        const bool att = m.mixer == KMLL_MIXER_ATTENTION;
+        v.seg[i] = GateSegment{up8(at), m.heads * m.vdim, m.vdim, att ? KMLL_OUT_NORM_NONE : m.out_norm, norm_weights[i], gates[i], att ? m.vdim : 1, m.gate_act, m.out_scale, eps};
+        if (v.seg[i].norm == KMLL_OUT_NORM_JOINT || v.seg[i].norm == KMLL_OUT_NORM_HEAD_WEIGHTED) KMLL_REQUIRE_PTR(norm_weights[i]);
+        at = v.seg[i].begin + v.seg[i].cols;
+    }
+    KMLL_REQUIRE(at == cols, "mixer_output_linear: the mixers give %d columns, not %d", at, cols);
+    return bf16_matvec(as_stream(s), v);
+}
+
+size_t kmll_grouped_attention_workspace_bytes(const kmll_mixer_spec* m) {
+    if (m == nullptr || m->heads <= 0 || m->vdim <= 0) return 0;
+    return kGroupedMaxTiles * 4 + grouped_decode_work_floats(m->heads, m->kv_heads > 0 ? m->kv_heads : m->heads, m->vdim) * 4;
+}
+
+int kmll_grouped_attention(kmll_stream_t s, const kmll_mixer_spec* m, const void* in, int in_f32, int ld, int q_off, int k_off, int v_off, int tokens, int position,
+                           const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, void* workspace, float* out, int ldo) {
+    KMLL_REQUIRE_PTR(m); KMLL_REQUIRE_PTR(in); KMLL_REQUIRE_PTR(cache); KMLL_REQUIRE_PTR(out);
+    const int g = m->kv_heads > 0 ? m->kv_heads : m->heads;
+    KMLL_REQUIRE(m->heads > 0 && m->heads % g == 0 && m->dim > 0 && m->vdim > 0 && m->window >= 0 && m->chunk >= 0 && tokens > 0 && position >= 0 &&
+                     (position_device != nullptr || position + tokens <= max_seq) && (pitch & 7) == 0 && pitch >= g * (up8(m->dim) + up8(m->vdim)) && ldo >= m->heads * m->vdim,
+                 "grouped_attention: bad shape");
+    GroupedArgs a;
+    memset(&a, 0, sizeof(a));
+    a.in = in; a.in_f32 = in_f32; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off;
+    a.T = tokens; a.heads = m->heads; a.kv_heads = g; a.dim = m->dim; a.vdim = m->vdim; a.window = m->window; a.chunk = m->chunk; a.scale = m->score_scale;
+    a.at = reinterpret_cast<const DecodeState*>(position_device);  // (the position is its first field)
+    a.pos0 = position;
+    a.cache = cache; a.cache_f32 = cache_f32; a.pitch = pitch; a.dimp = up8(m->dim); a.vdimp = up8(m->vdim); a.max_seq = max_seq;
+    a.out = out; a.ldo = ldo;
+    if (workspace != nullptr) {
+        a.counters = static_cast<unsigned int*>(workspace);
+        a.work = static_cast<float*>(workspace) + kGroupedMaxTiles;
+        if (grouped_decode_ok(a)) return grouped_attention_decode(as_stream(s), a);
+    }
+    KMLL_TRY_RC(grouped_write_cache(as_stream(s), a));
+    return position_device == nullptr && grouped_prefill_ok(a) ? grouped_attention_prefill(as_stream(s), a) : grouped_attention_plain(as_stream(s), a);
+}
+
+size_t kmll_gated_linear_scratch_floats(const kmll_mixer_spec* m, int tokens) {
+    return m != nullptr && tokens > 0 ? gated_chunk_scratch_floats(tokens, m->heads, m->dim, m->vdim, m->delta) : 0;
+}
+
+int kmll_gated_linear_attention(kmll_stream_t s, const kmll_mixer_spec* m, const kmll_gated_linear_weights* w, const void* in, int in_f32, int ld, const int* offsets,
+                                int tokens, int position, const int* position_device, float* state, float* ring, float* scratch, float* gate, float* out, int ldo) {
+    KMLL_REQUIRE_PTR(m); KMLL_REQUIRE_PTR(w); KMLL_REQUIRE_PTR(in); KMLL_REQUIRE_PTR(offsets); KMLL_REQUIRE_PTR(state); KMLL_REQUIRE_PTR(out);
+    KMLL_REQUIRE_PTR(w->decay_up);
+    const int g = m->kv_heads > 0 ? m->kv_heads : m->heads;
+    KMLL_REQUIRE(m->heads > 0 && m->heads % g == 0 && m->dim > 0 && m->vdim > 0 && m->decay_rank > 0 && (w->decay_pitch & 7) == 0 && w->decay_pitch >= m->decay_rank &&
+                     m->conv >= 0 && m->conv <= kMaxConvTaps && tokens > 0 && position >= 0 && ldo >= m->heads * m->vdim &&
+                     (m->decay == KMLL_DECAY_SOFTPLUS || (m->decay == KMLL_DECAY_LOGISTIC && m->decay_tau > 0.0f)),
+                 "gated_linear_attention: bad shape");
+    KMLL_REQUIRE(position_device == nullptr || tokens == 1, "gated_linear_attention: a position on the device is for one token");
+    if (m->decay == KMLL_DECAY_SOFTPLUS) KMLL_REQUIRE_PTR(w->decay_log);
+    if (m->conv > 0) { KMLL_REQUIRE_PTR(w->conv); KMLL_REQUIRE_PTR(ring); }
+    GatedLinearArgs a;
+    memset(&a, 0, sizeof(a));
+    a.in = in; a.in_f32 = in_f32; a.ld = ld;
+    a.q_off = offsets[0]; a.k_off = offsets[1]; a.v_off = offsets[2]; a.a_off = offsets[3]; a.b_off = offsets[4]; a.g_off = offsets[5];
+    a.T = tokens; a.heads = m->heads; a.kv_heads = g; a.dk = m->dim; a.dv = m->vdim;
+    a.decay = m->decay; a.inv_tau = m->decay == KMLL_DECAY_LOGISTIC ? 1.0f / m->decay_tau : 0.0f; a.rank = m->decay_rank;
+    a.up = w->decay_up; a.ldu = w->decay_pitch; a.bias = w->decay_bias; a.a_log = w->decay_log;
+    a.delta = m->delta; a.taps = m->conv; a.conv = w->conv; a.ring = ring; a.unit_eps = m->unit_eps; a.q_scale = m->q_scale;
+    a.at = reinterpret_cast<const DecodeState*>(position_device);
+    a.pos0 = position; a.state = state; a.out = out; a.ldo = ldo; a.scratch = scratch;
+    if (scratch != nullptr) return gated_linear_chunked(as_stream(s), a);
+    if (m->gate_rank > 0) {
+        KMLL_REQUIRE_PTR(w->gate_up); KMLL_REQUIRE_PTR(gate);
+        KMLL_REQUIRE((w->gate_pitch & 7) == 0 && w->gate_pitch >= m->gate_rank, "gated_linear_attention: bad gate pitch");
+        a.gate_rank = m->gate_rank; a.gate_up = w->gate_up; a.ldg = w->gate_pitch; a.gate = gate;
+    }
+    return gated_linear_steps(as_stream(s), a);
+}
+
 }  // extern "C"

@@ -48,7 +48,7 @@ def main():
     ap.add_argument("--cols", type=int, default=4096)
     ap.add_argument("--mats", type=int, default=8)
     ap.add_argument("--reps", type=int, default=10)
-    ap.add_argument("--suite", default="", choices=["", "decode", "chain4096", "micro", "gemm_sweep", "layered"],
+    ap.add_argument("--suite", default="", choices=["", "decode", "chain4096", "micro", "gemm_sweep", "layered", "somopel"],
                     help="layered: the kernels of the layered decoders beside their like kernels, and whole decoders; decode: every batch-1 operator shape of a Mistral-7B-architecture step; chain4096: 4096x4096 matvec + residual + "
                          "RMSNorm in both formats; micro: RMSNorm / SwiGLU / RoPE / row softmax over B in {1,16,64}, bf16; gemm_sweep: "
                          "M in {1,16,64,256,2048} x four (N,K), W4-G128")
@@ -73,6 +73,8 @@ def main():
         return suite_gemm_sweep(a.reps, shards=a.shards)
     if a.suite == "layered":
         return suite_layered(a.reps, only=a.only)
+    if a.suite == "somopel":
+        return suite_somopel(a.reps, only=a.only)
     run_one(a)
 
 
@@ -410,6 +412,200 @@ def suite_layered(reps, cpu=None, only="", context=2048):
                 print(json.dumps({"op": f"decoder uniform {width} wide, {layers} layers, {name} (closest model)", "decode_ms": round(ms, 4),
                                   "decode_tokens_per_s": round(1e3 / ms, 1), "launches_per_step": dec.launches_per_step, "step_frac_hbm": round(wb / ms / 1e6 / hbm, 3),
                                   "prefill_ms": round(pf, 3), "prefill_tokens_per_s": round(n / pf * 1e3)}), flush=True)
+                dec.close()
+                torch.cuda.empty_cache()
+
+
+# ---- Somopel ---------------------------------------------------------------------------------------------------------------
+# sizes that resemble real layers of the given width: (heads, kv heads, head size) of the attention, (heads, dim, vdim) of both recurrences
+SOMOPEL_SIZES = {4096: dict(ff=14336, attention=(32, 8, 128), gated=(32, 128, 128), delta=(32, 128, 128), rank=16, delta_rank=128),
+                 2048: dict(ff=8192, attention=(16, 4, 128), gated=(16, 128, 128), delta=(16, 128, 128), rank=16, delta_rank=64)}
+SOMOPEL_CHUNK = 4096
+
+
+def somopel_decoder(width, layers, max_seq_len, vocab=32000, compute_f32=False, chunk=SOMOPEL_CHUNK):
+    """Random-weight decoder whose layers alternate between the parallel mixer and the channel delta rule."""
+    from . import runtime as rt
+    from .somopel import layered_config
+    z = SOMOPEL_SIZES[width]
+    (H, G, D), (gh, gk, gv), (dh, dk, dv) = z["attention"], z["gated"], z["delta"]
+
+    def layer(i):
+        if i % 2 == 0:
+            m = {"left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": chunk}}, "left_scale": 0.9,
+                 "right": {"heads": gh, "dim": gk, "vdim": gv, "tau": 12.0}, "right_scale": 1.1}
+            return {"type": "parallel", "mixer": m, "mlp": {"kind": "dense", "ff": z["ff"]}}
+        return {"type": "channel_delta", "mixer": {"heads": dh, "kv_heads": dh, "dim": dk, "vdim": dv, "conv": 4}, "mlp": {"kind": "dense", "ff": z["ff"]}}
+
+    config = {"width": width, "vocab": vocab, "max_positions": max_seq_len, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "logit_scale": 1.0,
+              "layers": [layer(i) for i in range(layers)]}
+    dec = rt.LayeredDecoder(layered_config(config, lambda name: (z["rank"] if ".right." in name else z["delta_rank"],), compute_f32=compute_f32))
+    dec.init_random(7, 0.02)
+    return dec
+
+
+def suite_somopel(reps, cpu=None, only="", context=2048):
+    """The kernels of the Somopel design beside the like kernels of the closest model (the layered decoder of suite `layered`, at equal
+    sizes; for softmax attention the uniform decoder's), then whole decoders of equal width and layer count: decode at context
+    2048, 2048-token prompt.  Inputs of a line together exceed L2."""
+    from . import runtime as rt
+    gen = torch.Generator(device="cuda").manual_seed(6)
+
+    def bf(*shape, std=1.0):
+        return (torch.randn(shape, generator=gen, device="cuda") * std).to(torch.bfloat16)
+
+    def want(name):
+        return not only or only in name
+
+    def copies(nbytes):
+        return max(2, min(48, int(300e6 // nbytes) + 1))
+
+    n = context
+    pos = torch.tensor([n, 0, 0, 0], dtype=torch.int32, device="cuda")
+    for width, z in SOMOPEL_SIZES.items():
+        ff, (H, G, D), (gh, gk, gv), (dh, dk, dv) = z["ff"], z["attention"], z["gated"], z["delta"]
+        att = rt.MixerSpec(rt.MIXER_ATTENTION, H, D, D, kv_heads=G, score_scale=D ** -0.5, chunk=SOMOPEL_CHUNK, head_gate=1, gate_act=rt.ACT_SIGMOID, out_scale=0.9)
+        gated = rt.MixerSpec(rt.MIXER_GATED_LINEAR, gh, gk, gv, q_scale=gk ** -0.5, decay_kind=rt.DECAY_LOGISTIC, decay_tau=12.0, decay_rank=z["rank"],
+                             out_norm=rt.OUT_NORM_HEAD_WEIGHTED, out_scale=1.1)
+        delta = rt.MixerSpec(rt.MIXER_GATED_LINEAR, dh, dk, dv, q_scale=dk ** -0.5, decay_kind=rt.DECAY_SOFTPLUS, decay_rank=z["delta_rank"], delta=1, conv=4,
+                             unit_eps=1e-6, gate_rank=z["delta_rank"], gate_act=rt.ACT_SIGMOID, out_norm=rt.OUT_NORM_HEAD_WEIGHTED)
+        par_rows, del_rows = (H + 2 * G) * D + H + 2 * gh * (gk + gv) + z["rank"], dh * (2 * dk + dv) + 2 * z["delta_rank"] + dh
+        # ---- one row of x
+        nw, nb = bf(width), bf(width)
+        shapes = [("layer norm + projections of both mixers", par_rows, width, 0), ("layer norm + projections of the delta rule", del_rows, width, 0),
+                  ("layer norm + gelu(gate) up", 2 * ff, width, rt.ACT_GELU_TANH), ("layer norm + logits", 32000, width, 0)]
+        if want("matvec"):
+            x, y = torch.randn(width, device="cuda"), torch.empty(max(32000, 2 * ff, par_rows), device="cuda")
+            for name, rows, cols, act in shapes:
+                ws = [bf(rows, cols, std=0.02) for _ in range(copies(rows * cols * 2))]
+                us = time_graph([lambda w=w: ops.normed_linear_bf16(x, w, rt.NORM_LAYER, nw, nb, 1e-5, act, out=y) for w in ws], reps)
+                report(f"matvec {name} {rows}x{cols}", us, rows * cols * 2 + 4 * cols + 4 * rows)
+                us = time_graph([lambda w=w: ops.linear_bf16(x, w, norm_weight=nw, norm_offset=1.0, eps=1e-5, out=y) for w in ws], reps)
+                report(f"matvec norm + projection {rows}x{cols} (like kernel)", us, rows * cols * 2 + 4 * cols + 4 * rows)
+                del ws
+            cols = H * D + gh * gv
+            ws = [bf(width, cols, std=0.02) for _ in range(copies(width * cols * 2))]
+            o, res, hw = torch.randn(cols, device="cuda"), torch.randn(width, device="cuda"), bf(gv)
+            g0, g1, y1 = torch.randn(H, device="cuda"), torch.randn(gh * gv, device="cuda"), torch.empty(width, device="cuda")
+            gj = torch.randn(cols, device="cuda")
+            us = time_graph([lambda w=w: ops.mixer_output_linear_bf16([att, gated], o, [None, hw], [g0, g1], w, 1e-5, res, y1) for w in ws], reps)
+            report(f"matvec outputs of both mixers + projection {width}x{cols}", us, width * cols * 2 + 4 * cols + 4 * width)
+            us = time_graph([lambda w=w: ops.gated_linear_bf16(o, gj, w, 1e-5, head_len=gv, residual=res, out=y1) for w in ws], reps)
+            report(f"matvec gate + projection {width}x{cols} (like kernel)", us, width * cols * 2 + 4 * cols + 4 * width)
+            ws = [bf(width, ff, std=0.02) for _ in range(copies(width * ff * 2))]
+            xf, coef = torch.randn(ff, device="cuda"), bf(4)
+            us = time_graph([lambda w=w: ops.linear_bf16(xf, w, residual=res, out=y1) for w in ws], reps)
+            report(f"matvec down {width}x{ff}", us, width * ff * 2 + 4 * ff + 4 * width)
+            us = time_graph([lambda w=w: ops.polynorm_linear_bf16(xf, coef, 1e-5, w, residual=res, out=y1) for w in ws], reps)
+            report(f"matvec polynorm + down {width}x{ff} (like kernel)", us, width * ff * 2 + 4 * ff + 4 * width)
+            del ws
+        # ---- mixers, one token
+        aoff, kv = (0, H * D, (H + G) * D), 2 * G * D
+
+        def offsets(m):
+            q, v = (m.kv_heads or m.heads) * m.dim, m.heads * m.vdim
+            return (0, q, 2 * q, 2 * q + v, 2 * q + v + 2 * m.decay_rank, 2 * q + v + m.decay_rank)
+
+        def weights(m, count):
+            return [dict(decay_up=bf(m.heads * m.dim, m.decay_rank, std=0.1), decay_bias=bf(m.heads * m.dim), decay_log=bf(m.heads) if m.delta else None,
+                         conv=bf(m.heads * (2 * m.dim + m.vdim), 4, std=0.5) if m.conv else None,
+                         gate_up=bf(m.heads * m.vdim, m.gate_rank, std=0.1) if m.gate_rank else None) for _ in range(count)]
+
+        def columns(m):
+            return offsets(m)[4] + (m.heads + 7) // 8 * 8
+
+        def extra_bytes(m):
+            return 2 * m.heads * (m.dim * m.decay_rank + m.vdim * m.gate_rank) + (2 + 4) * m.conv * m.heads * (2 * m.dim + m.vdim)
+
+        if want("mixer decode"):
+            caches = [bf(n + 64, kv, std=0.5) for _ in range(48)]
+            x, out, ws = torch.randn((1, (H + 2 * G) * D), device="cuda"), torch.empty((1, H * D), device="cuda"), ops.grouped_attention_workspace(att)
+            us = time_graph([lambda c=c: ops.grouped_attention(att, x, aoff, pos, c, ws, out) for c in caches], reps)
+            report(f"mixer decode attention {H}/{G} heads x {D}, bf16 cache, context {n}", us, n * kv * 2)
+            del caches
+            caches = [(torch.randn((n + 64) * G * D, device="cuda"), torch.randn((n + 64) * G * D, device="cuda")) for _ in range(24)]
+            q, wsp, o2 = torch.randn(H * D, device="cuda"), ops.single_query_attention_workspace(H, D, n + 64), torch.empty(H * D, device="cuda")
+            us = time_graph([lambda c=c: ops.single_query_attention(q, c[0], c[1], n, n + 64, H, G, D, out=o2, workspace=wsp) for c in caches], reps)
+            report(f"mixer decode attention {H}/{G} heads x {D}, f32 cache, context {n} (like kernel)", us, 2 * n * kv * 2)
+            del caches
+            for name, m in (("gated linear", gated), ("delta rule", delta)):
+                sb, cnt = m.heads * m.dim * m.vdim * 4, copies(m.heads * m.dim * m.vdim * 8)
+                states, ws = [torch.randn(m.heads * m.dim * m.vdim, device="cuda") for _ in range(cnt)], weights(m, cnt)
+                x, out = torch.randn((1, columns(m)), device="cuda") * 0.1, torch.empty((1, m.heads * m.vdim), device="cuda")
+                gate = torch.empty(m.heads * m.vdim, device="cuda")
+                rings = [torch.zeros(4 * m.heads * (2 * m.dim + m.vdim), device="cuda") for _ in range(cnt)]
+                us = time_graph([lambda i=i: ops.gated_linear_attention(m, x, offsets(m), pos, states[i], ring=rings[i], gate=gate, out=out, **ws[i]) for i in range(cnt)],
+                                reps)
+                report(f"mixer decode {name} {m.heads}x{m.dim}x{m.vdim}", us, 2 * sb + extra_bytes(m) + 4 * columns(m) + 4 * m.heads * m.vdim)
+            pw = ops.decay_powers([0.99] * gh)
+            xl = torch.randn((1, 2 * gh * (gk + gv)), device="cuda") * 0.1
+            us = time_graph([lambda s=s: ops.linear_attention(xl, gh, gk, gv, pw, s, pos, 0, None, 0.1, None, out) for s in states], reps)
+            report(f"mixer decode lightning {gh}x{gk}x{gv} (like kernel)", us, 2 * sb + 4 * gh * (2 * gk + 2 * gv))
+            del states, ws, rings
+        # ---- prompt
+        T = n
+        if want("gemm"):
+            for rows, cols, act in ((par_rows, width, 0), (2 * ff, width, rt.ACT_GELU_TANH), (width, ff, 0), (width, H * D + gh * gv, 0)):
+                ws = [bf(rows, cols, std=0.02) for _ in range(4)]
+                x, y = bf(T, cols), torch.empty((T, rows), dtype=torch.bfloat16, device="cuda")
+                if act:
+                    yp = torch.empty((T, rows // 2), dtype=torch.bfloat16, device="cuda")
+                    us = time_graph([lambda w=w: ops.pair_linear_batched_bf16(x, w, act, out=yp) for w in ws], reps)
+                    report(f"gemm gelu(gate) up {T}x{rows}x{cols}", us, 2 * (rows * cols + T * cols + T * rows // 2), flops=2.0 * T * rows * cols)
+                us = time_graph([lambda w=w: ops.linear_batched_bf16(x, w, out=y) for w in ws], reps)
+                report(f"gemm {T}x{rows}x{cols}" + (" (like kernel)" if act else ""), us, 2 * (rows * cols + T * cols + T * rows), flops=2.0 * T * rows * cols)
+                del ws, x, y
+        if want("mixer prompt"):
+            caches = [bf(T, kv, std=0.5) for _ in range(4)]
+            xs, out = [bf(T, (H + 2 * G) * D) for _ in range(4)], torch.empty((T, H * D), device="cuda")
+            for chunk in (SOMOPEL_CHUNK, 512):
+                att.chunk = chunk
+                seen = min(chunk, T)
+                us = time_graph([lambda i=i: ops.grouped_attention(att, xs[i], aoff, 0, caches[i], None, out) for i in range(4)], reps)
+                report(f"mixer prompt attention (2 launches) {T} tokens, {H}/{G} heads x {D}, chunk {chunk}", us, T * (H + 2 * G) * D * 2 + T * kv * 2 + T * H * D * 4,
+                       flops=2.0 * H * T * seen * D)
+            att.chunk = SOMOPEL_CHUNK
+            del caches, xs
+            caches = [(torch.randn(T * G * D, device="cuda"), torch.randn(T * G * D, device="cuda")) for _ in range(4)]
+            q = torch.randn(T * H * D, device="cuda")
+            us = time_graph([lambda c=c: ops.prefill_causal_attention(q, c[0], c[1], T, T, H, G, D, out=out.view(-1)) for c in caches], reps)
+            report(f"mixer prompt attention {T} tokens, {H}/{G} heads x {D}, f32 cache (like kernel)", us, T * (H + 2 * G) * D * 4 + T * H * D * 4, flops=2.0 * H * T * T * D)
+            del caches
+            for name, m in (("gated linear", gated), ("delta rule", delta)):
+                xs, ws = [bf(T, columns(m), std=0.2) for _ in range(4)], weights(m, 4)
+                st, out, sc = torch.zeros(m.heads * m.dim * m.vdim, device="cuda"), torch.empty((T, m.heads * m.vdim), device="cuda"), ops.gated_linear_scratch(m, T)
+                ring = torch.zeros(4 * m.heads * (2 * m.dim + m.vdim), device="cuda")
+                us = time_graph([lambda i=i: ops.gated_linear_attention(m, xs[i], offsets(m), 0, st, ring=ring, scratch=sc, out=out, **ws[i]) for i in range(4)], reps)
+                fl = 2.0 * m.heads * T * (2 * m.dim * m.vdim + 32.5 * (m.dim + m.vdim) + (m.dim * m.vdim + 65 * m.dim + 32.5 * m.vdim if m.delta else 0))
+                report(f"mixer prompt {name} ({3 if m.conv else 2} launches) {T} tokens, {m.heads}x{m.dim}x{m.vdim}", us, T * m.heads * (2 * m.dim * 2 + m.vdim * 2 + m.vdim * 4),
+                       flops=fl)
+                del xs, ws, sc
+            xs, sc = [bf(T, 2 * gh * (gk + gv), std=0.2) for _ in range(4)], ops.linear_attention_scratch(T, gh, gk, gv)
+            pw, st = ops.decay_powers([0.99] * gh), torch.zeros(gh * gk * gv, device="cuda")
+            us = time_graph([lambda x=x: ops.linear_attention(x, gh, gk, gv, pw, st, 0, 0, None, 0.1, sc, out) for x in xs], reps)
+            report(f"mixer prompt lightning (3 launches) {T} tokens, {gh}x{gk}x{gv} (like kernel)", us, T * gh * (2 * gk * 2 + gv * 2 + gv * 4),
+                   flops=2.0 * gh * T * (2 * gk * gv + 32.5 * (gk + gv)))
+            del xs, sc
+        if want("rows"):
+            xs, os_ = [torch.randn((T, width), device="cuda") for _ in range(8)], torch.empty((T, width), dtype=torch.bfloat16, device="cuda")
+            us = time_graph([lambda x=x: ops.norm_rows_bf16(x, rt.NORM_LAYER, nw, nb, 1e-5, os_) for x in xs], reps)
+            report(f"rows layer norm [{T},{width}] f32 -> bf16", us, 6 * T * width)
+            us = time_graph([lambda x=x: ops.norm_rows_bf16(x, rt.NORM_RMS, nw, None, 1e-5, os_) for x in xs], reps)
+            report(f"rows rms norm [{T},{width}] f32 -> bf16 (like kernel)", us, 6 * T * width)
+            del xs
+        torch.cuda.empty_cache()
+        # ---- whole decoders
+        if want("decoder"):
+            layers, (hbm, tensor, _) = 12, peak_hbm_gbs()
+            for name, make in (("somopel", somopel_decoder), ("layered", layered_decoder)):
+                dec = make(width, layers, n + 256)
+                ms, pf = time_decoder(dec, n, max(16, reps))
+                elements = dec.cfg.weight_elements()
+                line = {"op": f"decoder {name} {width} wide, {layers} layers" + (" (closest model)" if name == "layered" else ""), "decode_ms": round(ms, 4),
+                        "decode_tokens_per_s": round(1e3 / ms, 1), "launches_per_step": dec.launches_per_step, "weights_gb": round(2e-9 * elements, 3),
+                        "weights_frac_hbm": round(2 * elements / ms / 1e6 / hbm, 3), "prefill_ms": round(pf, 3), "prefill_tokens_per_s": round(n / pf * 1e3),
+                        "prefill_weights_frac_tensor": round(2.0 * n * (elements - 32000 * width) / pf / 1e9 / tensor, 3)}
+                print(json.dumps(line), flush=True)
                 dec.close()
                 torch.cuda.empty_cache()
 

@@ -7,6 +7,7 @@ CUDA stream to libkmll_b200.so.  Nothing here computes on the CPU.
 """
 from __future__ import annotations
 
+import ctypes as C
 from dataclasses import dataclass
 
 import torch
@@ -644,4 +645,81 @@ def latent_attention_prefill(x, position, heads, dim, rot, vdim, rank, window, s
     out = torch.empty((x.shape[0], heads * vdim), dtype=torch.float32, device=x.device) if out is None else out
     check(load().kmll_latent_attention_prefill(_stream(), _p(x), x.shape[1], x.shape[0], position, heads, dim, rot, vdim, rank, window, scale, _p(table), _p(cache),
                                                cache.shape[1], cache.shape[0], _p(expanded), expanded.shape[1], first, _p(out)))
+    return out
+
+
+# ---- operators that take a mixer description (runtime.MixerSpec) ------------------------------------------------------------
+def normed_linear_bf16(x, w, norm: int = 0, norm_weight=None, norm_bias=None, eps: float = 0.0, pair_act: int = 0, out_scale: float = 1.0, out=None):
+    """norm: runtime.NORM_*.  pair_act: rows 2 i and 2 i + 1 of w are a gate and its value."""
+    out = torch.empty(w.shape[0] // (2 if pair_act else 1), dtype=torch.float32, device=w.device) if out is None else out
+    check(load().kmll_normed_linear_bf16(_stream(), _p(_f32(x, "x")), _p(w), _pitch(w), w.shape[0], w.shape[1], norm, _p(norm_weight), _p(norm_bias), eps, pair_act,
+                                         out_scale, _p(out)))
+    return out
+
+
+def pair_linear_batched_bf16(x, w, pair_act: int, workspace=None, out=None):
+    """x [batch, cols] bf16 or f32 -> [batch, rows / 2] of the same type."""
+    out = torch.empty((x.shape[0], w.shape[0] // 2), dtype=x.dtype, device=w.device) if out is None else out
+    check(load().kmll_pair_linear_batched_bf16(_stream(), _p(x), 1 if x.dtype == torch.float32 else 0, x.shape[1], x.shape[0], _p(w), _pitch(w), w.shape[0],
+                                               w.shape[1], pair_act, _p(workspace), _p(out)))
+    return out
+
+
+def norm_rows_bf16(x, norm: int, weight, bias=None, eps: float = 0.0, out=None):
+    out = torch.empty(x.shape, dtype=torch.bfloat16, device=x.device) if out is None else out
+    check(load().kmll_norm_rows_bf16(_stream(), _p(_f32(x, "x")), x.shape[0], x.shape[1], norm, _p(weight), _p(bias), eps, _p(out)))
+    return out
+
+
+def _pointers(tensors):
+    return (C.c_void_p * len(tensors))(*[None if t is None else t.data_ptr() for t in tensors])
+
+
+def mixer_output_linear_bf16(mixers, x, norm_weights, gates, w, eps: float, residual=None, out=None):
+    out = torch.empty(w.shape[0], dtype=torch.float32, device=w.device) if out is None else out
+    specs = [m._mixer() for m in mixers]
+    check(load().kmll_mixer_output_linear_bf16(_stream(), (type(specs[0]) * len(specs))(*specs), len(specs), _p(_f32(x, "x")), _pointers(norm_weights),
+                                               _pointers(gates), eps, _p(w), _pitch(w), w.shape[0], w.shape[1], _p(residual), _p(out)))
+    return out
+
+
+def grouped_attention_workspace(mixer, device="cuda") -> torch.Tensor:
+    return torch.zeros(load().kmll_grouped_attention_workspace_bytes(C.byref(mixer._mixer())) // 4, dtype=torch.float32, device=device)
+
+
+def grouped_attention(mixer, qkv, offsets, position, cache, workspace=None, out=None):
+    """qkv [tokens, ld] f32 or bf16 with q, k, v at `offsets`; position: an int, or an int32 tensor on the device; cache
+    [max_seq, pitch] f32 or bf16 (the tokens' rows are written)."""
+    tokens, ld = qkv.shape
+    out = torch.empty((tokens, mixer.heads * mixer.vdim), dtype=torch.float32, device=qkv.device) if out is None else out
+    dev = isinstance(position, torch.Tensor)
+    check(load().kmll_grouped_attention(_stream(), C.byref(mixer._mixer()), _p(qkv), 1 if qkv.dtype == torch.float32 else 0, ld, *offsets, tokens,
+                                        0 if dev else position, _p(position) if dev else None, _p(cache), 1 if cache.dtype == torch.float32 else 0, cache.shape[1],
+                                        cache.shape[0], _p(workspace), _p(out), out.shape[1]))
+    return out
+
+
+class _GatedLinearWeights(C.Structure):
+    _fields_ = [("decay_up", C.c_void_p), ("decay_pitch", C.c_int), ("decay_bias", C.c_void_p), ("decay_log", C.c_void_p), ("conv", C.c_void_p),
+                ("gate_up", C.c_void_p), ("gate_pitch", C.c_int)]
+
+
+def gated_linear_scratch(mixer, tokens: int, device="cuda") -> torch.Tensor:
+    return torch.empty(load().kmll_gated_linear_scratch_floats(C.byref(mixer._mixer()), tokens), dtype=torch.float32, device=device)
+
+
+def gated_linear_attention(mixer, x, offsets, position, state, decay_up, decay_bias=None, decay_log=None, conv=None, ring=None, gate_up=None, gate=None,
+                           scratch=None, out=None):
+    """x [tokens, ld]: q, k, v, decay factor, logits of beta, gate factor at `offsets` (six columns; unused ones 0)."""
+    tokens, ld = x.shape
+    out = torch.empty((tokens, mixer.heads * mixer.vdim), dtype=torch.float32, device=x.device) if out is None else out
+
+    def ptr(t):
+        return None if t is None else t.data_ptr()
+
+    w = _GatedLinearWeights(ptr(decay_up), decay_up.shape[1], ptr(decay_bias), ptr(decay_log), ptr(conv), ptr(gate_up), 0 if gate_up is None else gate_up.shape[1])
+    dev = isinstance(position, torch.Tensor)
+    check(load().kmll_gated_linear_attention(_stream(), C.byref(mixer._mixer()), C.byref(w), _p(x), 1 if x.dtype == torch.float32 else 0, ld,
+                                             (C.c_int * 6)(*offsets), tokens, 0 if dev else position, _p(position) if dev else None, _p(state), _p(ring), _p(scratch),
+                                             _p(gate), _p(out), out.shape[1]))
     return out

@@ -301,12 +301,10 @@ int kmll_mixer_output_linear_bf16(kmll_stream_t stream, const kmll_mixer_spec* m
                                   const float* const* gates, float eps, const uint16_t* w, int pitch, int rows, int cols, const float* residual, float* y);
 /* Grouped attention over a cache [max_seq, pitch] (f32 or bf16): keys of every key / value head, each padded to a multiple of 8
  * entries (zeros), then the values likewise.  in [tokens, ld]: q, k, v at their column offsets.  The tokens' cache rows are
- * written, then every position they see is attended.  One token at *position_device with a workspace: the decode form (f32 input,
- * bf16 cache); bf16 input and cache: the prompt form; else plain f32 arithmetic.  workspace: _workspace_bytes() bytes whose first
- * 4096 are zero before the first call (each call leaves them so). */
-size_t kmll_grouped_attention_workspace_bytes(const kmll_mixer_spec* mixer);
+ * written, then every position they see is attended.  One token at *position_device: the decode form (f32 input, bf16 cache);
+ * bf16 input and cache: the prompt form; else plain f32 arithmetic. */
 int kmll_grouped_attention(kmll_stream_t stream, const kmll_mixer_spec* mixer, const void* in, int in_f32, int ld, int q_off, int k_off, int v_off, int tokens,
-                           int position, const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, void* workspace, float* out, int ldo);
+                           int position, const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, float* out, int ldo);
 /* Gated linear attention.  in [tokens, ld]: q, k, v, the decay factor (decay_rank), the logits of beta (heads) and the gate factor
  * (gate_rank) at offsets[0 .. 5].  conv [q | k | v channels][taps]; ring [taps][channels] f32 holds the inputs of earlier
  * positions.  state [heads, dim, vdim] f32 and ring are updated.  scratch == null: token after token in f32, the low-rank gate goes

@@ -68,30 +68,75 @@ __device__ inline float dot_row(const uint16_t* w, const float* x, int n) {
 }
 
 // ---- step form ------------------------------------------------------------------------------------------------------------------
-// Block (head, 32 value columns): four warps of eight columns; lane (row lane, column quad) keeps rows rl, rl + 16, .. of four
-// columns in registers for the whole call, so the sums over keys stay inside a warp.
-constexpr int kSThreads = 128, kSCols = 32;
+// Block (head, 32 value columns): eight warps of four columns; a lane keeps rows lane, lane + 32, .. of them in registers for the
+// whole call, so the sums over keys stay inside a warp.  Of a single token's work, everything that does not read its projections
+// (state, low-rank maps, the convolutions over earlier inputs) is done ahead of the dependency wait.
+constexpr int kSThreads = 256, kSCols = 32;
+struct StepLayout {
+    int dkr, rank8, gate8, chans;  // padded sizes; channels a block convolves
+    int off_part, off_maps;        // in floats / bytes: partial convolutions, then the staged maps
+    bool staged;
+    int total;
+};
+__host__ __device__ inline StepLayout step_layout(int dk, int rank, int gate_rank, int taps) {
+    StepLayout l;
+    l.dkr = round_to(dk, 4);
+    l.rank8 = round_to(rank, 8);
+    l.gate8 = round_to(gate_rank, 8);
+    l.chans = 2 * dk + kSCols;
+    l.off_part = 3 * l.dkr + kSCols + l.rank8 + l.gate8;
+    l.off_maps = round_to((l.off_part + (taps > 0 ? 2 * l.chans : 0)) * 4, 16);
+    const int maps = (dk * (l.rank8 + 8) + (gate_rank > 0 ? kSCols * (l.gate8 + 8) : 0)) * 2;
+    l.staged = maps <= 96 * 1024;
+    l.total = l.off_maps + (l.staged ? maps : 0);
+    return l;
+}
 
 template <bool F32, int RP>
 __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinearArgs a) {
-    extern __shared__ __align__(16) float ssm[];  // q | k | decay, [dk] each | v [32] | a [rank] | g [gate_rank], padded
-    const int dkr = round_to(a.dk, 4), rank8 = round_to(a.rank, 8), gate8 = round_to(a.gate_rank, 8);
+    extern __shared__ __align__(16) float ssm[];  // q | k | decay, [dk] each | v [32] | a [rank] | g [gate_rank], padded | ..
+    const StepLayout sl = step_layout(a.dk, a.rank, a.gate_rank, a.taps);
+    const int rank8 = sl.rank8, gate8 = sl.gate8;
     float* const sq = ssm;
-    float* const sk = sq + dkr;
-    float* const sg = sk + dkr;
-    float* const sv = sg + dkr;
+    float* const sk = sq + sl.dkr;
+    float* const sg = sk + sl.dkr;
+    float* const sv = sg + sl.dkr;
     float* const sa = sv + kSCols;
     float* const sgr = sa + rank8;
+    float* const early = ssm + sl.off_part;       // one token: sum over the earlier taps, then the last tap, per channel
+    uint16_t* const maps = reinterpret_cast<uint16_t*>(reinterpret_cast<unsigned char*>(ssm) + sl.off_maps);
     __shared__ float dots[4];  // q.q, k.k, q.k, beta
-    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane & 15;
-    const int col0 = blockIdx.y * kSCols, lc = warp * 8 + (lane >> 4) * 4, c0 = col0 + lc;
+    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int col0 = blockIdx.y * kSCols, lc = warp * 4, c0 = col0 + lc;
     const int per = a.heads / a.kv_heads, hq = h / per, nq = a.kv_heads * a.dk, channels = 2 * nq + a.heads * a.dv;
     float* const S = a.state + (size_t)h * a.dk * a.dv;
-    const bool vec = (a.dv & 3) == 0;
+    const bool vec = (a.dv & 3) == 0, single = a.T == 1;
+    // weights never change; the state's last writer lies more than one launch back, and so does that of the position and the ring
+    const int up_pitch = sl.staged ? rank8 + 8 : a.ldu, gate_pitch = sl.staged ? gate8 + 8 : a.ldg;
+    const uint16_t* up = a.up + (size_t)h * a.dk * a.ldu;
+    const uint16_t* gate_up = a.gate_rank > 0 ? a.gate_up + (size_t)(h * a.dv + col0) * a.ldg : nullptr;
+    if (sl.staged) {
+        const int runs = rank8 / 8;
+        for (int i = tid; i < a.dk * runs; i += kSThreads) {
+            const int d = i / runs, r = (i - d * runs) * 8;
+            cp_async16_to((uint32_t)__cvta_generic_to_shared(maps + d * up_pitch + r), up + (size_t)d * a.ldu + r);
+        }
+        uint16_t* const gm = maps + a.dk * up_pitch;
+        if (a.gate_rank > 0) {
+            const int gruns = gate8 / 8, rows = min(kSCols, a.dv - col0);
+            for (int i = tid; i < rows * gruns; i += kSThreads) {
+                const int c = i / gruns, r = (i - c * gruns) * 8;
+                cp_async16_to((uint32_t)__cvta_generic_to_shared(gm + c * gate_pitch + r), gate_up + (size_t)c * a.ldg + r);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        up = maps;
+        gate_up = gm;
+    }
     float s[RP][4];
 #pragma unroll
-    for (int r = 0; r < RP; ++r) {  // (the state's last writer lies more than one launch back)
-        const int i = rl + r * 16;
+    for (int r = 0; r < RP; ++r) {
+        const int i = lane + r * 32;
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[r][e] = 0.0f;
         if (i < a.dk && c0 < a.dv) {
@@ -105,48 +150,67 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
             }
         }
     }
-    {   // weights never change: towards L2 ahead of the dependency wait
-        const char* up = reinterpret_cast<const char*>(a.up + (size_t)h * a.dk * a.ldu);
-        for (int i = tid * 128; i < a.dk * a.ldu * 2; i += kSThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(up + i));
-        if (a.gate_rank > 0) {
-            const int rows = min(kSCols, a.dv - col0);
-            const char* gu = reinterpret_cast<const char*>(a.gate_up + (size_t)(h * a.dv + col0) * a.ldg);
-            for (int i = tid * 128; i < rows * a.ldg * 2; i += kSThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(gu + i));
+    const int pos0 = a.at != nullptr ? a.at->position : a.pos0;
+    // column of the projection and channel of entry i of q | k | v (v: of this block's columns); false: no such channel
+    auto place = [&](int i, int& col, int& ch) -> bool {
+        if (i < 2 * a.dk) {
+            const int d = i < a.dk ? i : i - a.dk;
+            ch = (i < a.dk ? 0 : nq) + hq * a.dk + d;
+            col = (i < a.dk ? a.q_off : a.k_off) + hq * a.dk + d;
+            return true;
         }
-    }
+        const int c = i - 2 * a.dk;
+        ch = 2 * nq + h * a.dv + col0 + c;
+        col = a.v_off + h * a.dv + col0 + c;
+        return col0 + c < a.dv;
+    };
+    if (single && a.taps > 0)
+        for (int i = tid; i < sl.chans; i += kSThreads) {
+            int col, ch;
+            float y = 0.0f, last = 0.0f;
+            if (place(i, col, ch)) {
+                const uint16_t* w = a.conv + (size_t)ch * a.taps;
+                for (int j = 0; j + 1 < a.taps; ++j) {
+                    const int p = pos0 - (a.taps - 1 - j);
+                    if (p >= 0) y = fmaf(bf16_bits_to_f32(w[j]), a.ring[(size_t)(p % a.taps) * channels + ch], y);
+                }
+                last = bf16_bits_to_f32(w[a.taps - 1]);
+            }
+            early[i] = y;
+            early[sl.chans + i] = last;
+        }
     const float rate = decay_rate(a, h);
-    const int pos0 = a.at != nullptr ? a.at->position : a.pos0;  // (written more than one launch ago)
     pdl_wait();
     for (int t = 0; t < a.T; ++t) {
         const int pos = pos0 + t;
         const size_t row = (size_t)t * a.ld;
         // ---- q, k, v, and the inputs of the low-rank maps
-        const int n_in = 2 * a.dk + kSCols;
-        for (int i = tid; i < n_in + rank8 + gate8; i += kSThreads) {
-            if (i < 2 * a.dk) {
-                const int d = i < a.dk ? i : i - a.dk, ch = (i < a.dk ? 0 : nq) + hq * a.dk + d, col = (i < a.dk ? a.q_off : a.k_off) + hq * a.dk + d;
-                const float y = convolved<F32>(a, t, pos, col, ch, channels);
-                if (i < a.dk) sq[d] = y;
-                else sk[d] = y;
-                if (a.taps > 0 && a.T == 1 && blockIdx.y == 0 && h == hq * per) a.ring[(size_t)(pos % a.taps) * channels + ch] = in_at<F32>(a.in, row + col);
-            } else if (i < n_in) {
-                const int c = i - 2 * a.dk, ch = 2 * nq + h * a.dv + col0 + c, col = a.v_off + h * a.dv + col0 + c;
+        for (int i = tid; i < sl.chans + rank8 + gate8; i += kSThreads) {
+            if (i < sl.chans) {
+                int col, ch;
                 float y = 0.0f;
-                if (col0 + c < a.dv) {
-                    y = convolved<F32>(a, t, pos, col, ch, channels);
-                    if (a.taps > 0 && a.T == 1) a.ring[(size_t)(pos % a.taps) * channels + ch] = in_at<F32>(a.in, row + col);
+                if (place(i, col, ch)) {
+                    if (single && a.taps > 0) {
+                        const float x = in_at<F32>(a.in, col);
+                        y = act_silu(fmaf(early[sl.chans + i], x, early[i]));
+                        if (i >= 2 * a.dk || (blockIdx.y == 0 && h == hq * per)) a.ring[(size_t)(pos % a.taps) * channels + ch] = x;
+                    } else {
+                        y = convolved<F32>(a, t, pos, col, ch, channels);
+                    }
                 }
-                sv[c] = y;
-            } else if (i < n_in + rank8) {
-                const int r = i - n_in;
+                (i < a.dk ? sq : i < 2 * a.dk ? sk - a.dk : sv - 2 * a.dk)[i] = y;
+            } else if (i < sl.chans + rank8) {
+                const int r = i - sl.chans;
                 sa[r] = r < a.rank ? in_at<F32>(a.in, row + a.a_off + r) : 0.0f;
             } else {
-                const int r = i - n_in - rank8;
+                const int r = i - sl.chans - rank8;
                 sgr[r] = r < a.gate_rank ? in_at<F32>(a.in, row + a.g_off + r) : 0.0f;
             }
         }
+        if (warp == 3 && lane == 0) dots[3] = a.delta ? act_sigmoid(in_at<F32>(a.in, row + a.b_off + h)) : 1.0f;
+        if (t == 0 && sl.staged) asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        // ---- decays, norms of q and k, gate
+        // ---- decays (two lanes per channel), norms of q and k, gate (eight lanes per column)
         if (warp < 3) {
             const float* x = warp == 1 ? sk : sq;
             const float* y = warp == 0 ? sq : sk;
@@ -154,21 +218,26 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
             for (int i = lane; i < a.dk; i += 32) d = fmaf(x[i], y[i], d);
             d = warp_sum(d);
             if (lane == 0) dots[warp] = d;
-        } else if (lane == 0) {
-            dots[3] = a.delta ? act_sigmoid(in_at<F32>(a.in, row + a.b_off + h)) : 1.0f;
         }
-        for (int d = tid; d < a.dk; d += kSThreads) {
-            float z = dot_row(a.up + (size_t)(h * a.dk + d) * a.ldu, sa, rank8);
-            if (a.bias != nullptr) z += bf16_bits_to_f32(a.bias[h * a.dk + d]);
-            sg[d] = exp2f(log2_decay(a, z, rate));
+        for (int i0 = 0; i0 < 2 * a.dk; i0 += kSThreads) {
+            const int d = (i0 + tid) >> 1;
+            float z = 0.0f;
+            if (d < a.dk)
+                for (int r = (tid & 1) * 8; r < rank8; r += 16) z += dot_row(up + (size_t)d * up_pitch + r, sa + r, 8);
+            z += __shfl_xor_sync(0xffffffffu, z, 1);
+            if (d < a.dk && (tid & 1) == 0) {
+                if (a.bias != nullptr) z += bf16_bits_to_f32(a.bias[h * a.dk + d]);
+                sg[d] = exp2f(log2_decay(a, z, rate));
+            }
         }
         if (a.gate_rank > 0) {
-            const int c = tid >> 2, part = tid & 3;  // four lanes per column
+            const int c = tid >> 3, part = tid & 7;
             float g = 0.0f;
             if (col0 + c < a.dv)
-                for (int r = part * 8; r < gate8; r += 32) g += dot_row(a.gate_up + (size_t)(h * a.dv + col0 + c) * a.ldg + r, sgr + r, 8);
+                for (int r = part * 8; r < gate8; r += 64) g += dot_row(gate_up + (size_t)c * gate_pitch + r, sgr + r, 8);
             g += __shfl_xor_sync(0xffffffffu, g, 1);
             g += __shfl_xor_sync(0xffffffffu, g, 2);
+            g += __shfl_xor_sync(0xffffffffu, g, 4);
             if (part == 0 && col0 + c < a.dv) a.gate[(size_t)t * a.heads * a.dv + (size_t)h * a.dv + col0 + c] = g;
         }
         __syncthreads();
@@ -179,48 +248,57 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
             fk = 1.0f / sqrtf(dots[1] + a.unit_eps);
         }
         const float qk = dots[2] * fq * fk, beta = dots[3];
-        float kv[4] = {}, qs[4] = {};
+        float sums[8] = {};  // of the decayed state: S^T k, S^T q
 #pragma unroll
         for (int r = 0; r < RP; ++r) {
-            const int i = rl + r * 16;
+            const int i = lane + r * 32;
             if (i < a.dk) {
                 const float g = sg[i], k = sk[i] * fk, q = sq[i] * fq;
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     s[r][e] *= g;
-                    kv[e] = fmaf(k, s[r][e], kv[e]);
-                    qs[e] = fmaf(q, s[r][e], qs[e]);
+                    sums[e] = fmaf(k, s[r][e], sums[e]);
+                    sums[4 + e] = fmaf(q, s[r][e], sums[4 + e]);
                 }
             }
         }
+        // fold eight sums over 32 lanes: lanes keep one half of them in each step; lanes 4 j .. 4 j + 3 end up with sum j
 #pragma unroll
-        for (int off = 1; off < 16; off <<= 1)
+        for (int n = 4, off = 16; n >= 1; n >>= 1, off >>= 1) {
+            const bool high = (lane & off) != 0;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                kv[e] += __shfl_xor_sync(0xffffffffu, kv[e], off);
-                qs[e] += __shfl_xor_sync(0xffffffffu, qs[e], off);
-            }
+            for (int i = 0; i < 4; ++i)
+                if (i < n) {
+                    const float keep = high ? sums[i + n] : sums[i], give = high ? sums[i] : sums[i + n];
+                    sums[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+                }
+        }
+        float all = sums[0];
+        all += __shfl_xor_sync(0xffffffffu, all, 2);
+        all += __shfl_xor_sync(0xffffffffu, all, 1);
         float u[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) u[e] = a.delta ? beta * (sv[lc + e] - kv[e]) : sv[lc + e];
+        for (int e = 0; e < 4; ++e) {
+            const float kv = __shfl_sync(0xffffffffu, all, e * 4);
+            u[e] = a.delta ? beta * (sv[lc + e] - kv) : sv[lc + e];
+        }
+        const float qs = __shfl_sync(0xffffffffu, all, 16 + (lane & 3) * 4);
+        if (lane < 4 && c0 + lane < a.dv)  // S^T q with the token's own write
+            a.out[(size_t)t * a.ldo + (size_t)h * a.dv + c0 + lane] = qs + qk * (lane == 0 ? u[0] : lane == 1 ? u[1] : lane == 2 ? u[2] : u[3]);
 #pragma unroll
         for (int r = 0; r < RP; ++r) {
-            const int i = rl + r * 16;
+            const int i = lane + r * 32;
             if (i < a.dk) {
                 const float k = sk[i] * fk;
 #pragma unroll
                 for (int e = 0; e < 4; ++e) s[r][e] = fmaf(k, u[e], s[r][e]);
             }
         }
-        if (rl < 4) {  // S^T q with the token's own write
-            const float o = rl == 0 ? qs[0] + qk * u[0] : rl == 1 ? qs[1] + qk * u[1] : rl == 2 ? qs[2] + qk * u[2] : qs[3] + qk * u[3];
-            if (c0 + rl < a.dv) a.out[(size_t)t * a.ldo + (size_t)h * a.dv + c0 + rl] = o;
-        }
         if (t + 1 < a.T) __syncthreads();
     }
 #pragma unroll
     for (int r = 0; r < RP; ++r) {
-        const int i = rl + r * 16;
+        const int i = lane + r * 32;
         if (i < a.dk && c0 < a.dv) {
             if (vec) {
                 *reinterpret_cast<float4*>(S + (size_t)i * a.dv + c0) = make_float4(s[r][0], s[r][1], s[r][2], s[r][3]);
@@ -253,10 +331,11 @@ int write_ring(cudaStream_t stream, const GatedLinearArgs& a) {
 
 template <bool F32>
 int run_steps(cudaStream_t stream, const GatedLinearArgs& a) {
-    const int rp = (a.dk + 15) / 16;
-    auto k = rp <= 2 ? gated_step_kernel<F32, 2> : rp <= 4 ? gated_step_kernel<F32, 4> : rp <= 8 ? gated_step_kernel<F32, 8>
-           : rp <= 16 ? gated_step_kernel<F32, 16> : gated_step_kernel<F32, 32>;
-    const size_t smem = ((size_t)3 * round_to(a.dk, 4) + kSCols + round_to(a.rank, 8) + round_to(a.gate_rank, 8)) * 4;
+    const int rp = (a.dk + 31) / 32;
+    auto k = rp <= 1 ? gated_step_kernel<F32, 1> : rp <= 2 ? gated_step_kernel<F32, 2> : rp <= 4 ? gated_step_kernel<F32, 4>
+           : rp <= 8 ? gated_step_kernel<F32, 8> : gated_step_kernel<F32, 16>;
+    const size_t smem = (size_t)step_layout(a.dk, a.rank, a.gate_rank, a.taps).total;
+    if (smem > 220 * 1024) return fail(KMLL_ERR_UNSUPPORTED, "gated linear attention: ranks %d, %d are too large", a.rank, a.gate_rank);
     cudaError_t e = allow_all_dynamic_smem(k);
     if (e == cudaSuccess) e = launch(k, dim3(a.heads, (a.dv + kSCols - 1) / kSCols), dim3(kSThreads), smem, stream, true, a);
     if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "gated linear attention (steps): %s", cudaGetErrorString(e));
@@ -297,120 +376,234 @@ __device__ inline void mma_split(float (&c)[4], const uint32_t (&ah)[4], const u
     mma_bf16(c, ah, bl0, bl1);
 }
 
+// Shared memory of the preparing launch, in bytes: q, k and log decays of the chunk in f32; ahead of them, in the same places, the
+// projected rows they come from.
+struct PrepareLayout {
+    int P, PR;             // pitches: f32 rows, rows of the decay map
+    int off_k, off_g, off_l, off_v, staged_decay, total;
+};
+__host__ __device__ inline PrepareLayout prepare_layout(int DK, int delta, int taps, int rank) {
+    PrepareLayout l;
+    const int rows = kGC + (taps > 0 ? taps - 1 : 0), tile = kGC * (DK + 4) * 4, raw = rows * DK * 2;
+    l.P = DK + 4;
+    l.PR = round_to(rank, 16) + 8;
+    l.off_k = tile;
+    l.off_g = 2 * tile;
+    l.off_l = l.off_g + (2 * raw > tile ? 2 * raw : tile);
+    l.off_v = l.off_l + (delta ? kGC * kAP * 4 : 0);
+    l.total = l.off_v + (delta ? raw : 0);
+    l.staged_decay = (kGC + DK) * l.PR * 2 <= 2 * tile;  // the decay factor and map fit in the places of q and k
+    return l;
+}
+
+// Rows [t0 - taps + 1, t0 + 64) of `cols` consecutive projected channels (from column `col`, ring channel `ch`) -> bf16 tile
+// [..][DK]; zeros where there is no token or channel.
+template <int DK, int NT>
+__device__ inline void stage_rows(const GatedLinearArgs& a, uint16_t* tile, int t0, int n, int col, int ch, int cols, int channels, bool fast) {
+    const uint16_t* in = static_cast<const uint16_t*>(a.in);
+    const int back = a.taps > 0 ? a.taps - 1 : 0, rows = kGC + back;
+    constexpr int RUNS = DK / 8;
+    for (int i = threadIdx.x; i < rows * RUNS; i += NT) {
+        const int r = i / RUNS, c = (i % RUNS) * 8, t = t0 + r - back;
+        uint16_t* dst = tile + r * DK + c;
+        if (t >= 0 && fast) {
+            const bool live = r - back < n && c < cols;
+            cp_async16_zfill_to((uint32_t)__cvta_generic_to_shared(dst), live ? in + (size_t)t * a.ld + col + c : in, live ? 16u : 0u);
+        } else {
+            for (int e = 0; e < 8; ++e) {
+                uint16_t v = 0;
+                if (c + e < cols && r - back < n) {
+                    if (t >= 0) v = in[(size_t)t * a.ld + col + c + e];
+                    else if (a.pos0 + t >= 0) v = f32_to_bf16_bits(a.ring[(size_t)((a.pos0 + t) % a.taps) * channels + ch + c + e]);
+                }
+                dst[e] = v;
+            }
+        }
+    }
+}
+// channels d, d + 1 of token t from a staged tile, through convolution and SiLU; w0, w1: their taps (null: none)
+template <int DK>
+__device__ inline float2 staged_pair(const GatedLinearArgs& a, const uint16_t* tile, int t, int d, const uint16_t* w0, const uint16_t* w1) {
+    if (a.taps == 0) {
+        const uint32_t x = *reinterpret_cast<const uint32_t*>(tile + t * DK + d);
+        return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u));
+    }
+    float2 y = make_float2(0.0f, 0.0f);
+    for (int j = 0; j < a.taps; ++j) {
+        const uint32_t x = *reinterpret_cast<const uint32_t*>(tile + (t + j) * DK + d);
+        y.x = fmaf(bf16_bits_to_f32(w0[j]), __uint_as_float(x << 16), y.x);
+        y.y = fmaf(bf16_bits_to_f32(w1[j]), __uint_as_float(x & 0xffff0000u), y.y);
+    }
+    return make_float2(act_silu(y.x), act_silu(y.y));
+}
+
 template <int DK, bool DELTA>
-__global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const ChunkArgs ca) {
-    constexpr int P = DK + 4;
+__global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(const ChunkArgs ca) {
+    constexpr int NT = DELTA ? 512 : 256, NW = NT / 32, P = DK + 4;
     const GatedLinearArgs& a = ca.a;
-    extern __shared__ __align__(16) float gsm[];
-    float* const Q = gsm;                  // [64][P]
-    float* const K = Q + kGC * P;
-    float* const G = K + kGC * P;          // log2 decays, then their running sums
-    float* const A = G + kGC * P;          // [64][kAP]
-    float* const L = A + kGC * kAP;        // DELTA: L, then its inverse
-    __shared__ float beta[kGC], total[4 * DK];
+    extern __shared__ __align__(16) unsigned char gsm[];
+    const PrepareLayout pl = prepare_layout(DK, DELTA ? 1 : 0, a.taps, a.rank);
+    float* const Q = reinterpret_cast<float*>(gsm);               // [64][P]
+    float* const K = reinterpret_cast<float*>(gsm + pl.off_k);    // [64][P]
+    float* const G = reinterpret_cast<float*>(gsm + pl.off_g);    // [64][P] log2 decays, then their running sums
+    float* const L = reinterpret_cast<float*>(gsm + pl.off_l);    // DELTA: [64][kAP] L, then its inverse
+    const int back = a.taps > 0 ? a.taps - 1 : 0;
+    uint16_t* const raw_q = reinterpret_cast<uint16_t*>(gsm + pl.off_g);
+    uint16_t* const raw_k = raw_q + (kGC + back) * DK;
+    uint16_t* const raw_v = reinterpret_cast<uint16_t*>(gsm + pl.off_v);
+    uint16_t* const sa = reinterpret_cast<uint16_t*>(gsm);        // [64][PR] decay factor
+    uint16_t* const su = sa + kGC * pl.PR;                        // [DK][PR] decay map of this head
+    __shared__ float beta[kGC], total[NT];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
     const int c = blockIdx.x, h = blockIdx.y, t0 = c * kGC, n = min(kGC, a.T - t0);
     const int per = a.heads / a.kv_heads, hq = h / per, nq = a.kv_heads * a.dk, channels = 2 * nq + a.heads * a.dv;
+    const int chq = hq * a.dk, chv = 2 * nq + h * a.dv;
     const uint16_t* in = static_cast<const uint16_t*>(a.in);
+    const bool fast = ((a.ld | a.q_off | a.k_off | a.v_off | a.dk | a.dv) & 7) == 0 && (reinterpret_cast<uintptr_t>(a.in) & 15u) == 0;
     const ChunkLayout lay = chunk_layout(DK, DELTA ? 1 : 0);
     float* const out = ca.planes + ((size_t)c * a.heads + h) * lay.floats;
     uint16_t* const planes = reinterpret_cast<uint16_t*>(out);
-    for (int i = tid; i < kGC * kAP * (DELTA ? 2 : 1); i += kGThreads) A[i] = 0.0f;
+    uint16_t* const Ah = reinterpret_cast<uint16_t*>(out + (DELTA ? 6 : 4) * lay.plane);
+    uint16_t* const Al = Ah + 2 * lay.a_plane;
+    const int rank8 = round_to(a.rank, 8), runs = pl.PR / 8 - 1;
+    if (pl.staged_decay)  // weights never change: ahead of the dependency wait
+        for (int i = tid; i < DK * runs; i += NT) {
+            const int d = i / runs, r = (i - d * runs) * 8;
+            const bool live = d < a.dk && r < rank8;
+            cp_async16_zfill_to((uint32_t)__cvta_generic_to_shared(su + d * pl.PR + r), live ? a.up + (size_t)(h * a.dk + d) * a.ldu + r : a.up, live ? 16u : 0u);
+        }
     const float rate = decay_rate(a, h);
     pdl_wait();
-    // ---- q, k, log decays, write strengths; rows behind the last token change nothing (zeros, decay 1)
-    for (int i = tid; i < kGC * DK; i += kGThreads) {
-        const int t = i / DK, d = i % DK;
-        float q = 0.0f, k = 0.0f;
-        if (t < n && d < a.dk) {
-            const int ch = hq * a.dk + d;
-            q = convolved<false>(a, t0 + t, a.pos0 + t0 + t, a.q_off + ch, ch, channels);
-            k = convolved<false>(a, t0 + t, a.pos0 + t0 + t, a.k_off + ch, nq + ch, channels);
-            if (a.unit_eps <= 0.0f) q *= a.q_scale;
+    if (pl.staged_decay)
+        for (int i = tid; i < kGC * runs; i += NT) {
+            const int t = i / runs, r = (i - t * runs) * 8;
+            const bool live = t < n && r < rank8;
+            cp_async16_zfill_to((uint32_t)__cvta_generic_to_shared(sa + t * pl.PR + r), live ? in + (size_t)(t0 + t) * a.ld + a.a_off + r : in, live ? 16u : 0u);
         }
-        Q[t * P + d] = q;
-        K[t * P + d] = k;
-    }
+    stage_rows<DK, NT>(a, raw_q, t0, n, a.q_off + chq, chq, a.dk, channels, fast);
+    stage_rows<DK, NT>(a, raw_k, t0, n, a.k_off + chq, nq + chq, a.dk, channels, fast);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    if (DELTA) stage_rows<DK, NT>(a, raw_v, t0, n, a.v_off + h * a.dv, chv, a.dv, channels, fast);
+    asm volatile("cp.async.commit_group;" ::: "memory");
     if (tid < kGC) beta[tid] = !DELTA ? 1.0f : tid < n ? act_sigmoid(bf16_bits_to_f32(in[(size_t)(t0 + tid) * a.ld + a.b_off + h])) : 0.0f;
-    {   // z = W_up a: 64 tokens x DK channels, DK / 8 column blocks over the warps
-        constexpr int NB = DK / 64;
-        const int rank8 = round_to(a.rank, 8);
-        float z[NB][4][4];
+    if (DELTA)
+        for (int i = tid; i < kGC * kAP; i += NT) L[i] = 0.0f;
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    // ---- log decays from z = W_up a: 64 tokens x DK channels; a warp holds 16 x MB tokens of 8 x NB channels
+    constexpr int NB = DK == 64 && NW == 16 ? 1 : DK / 64, MB = DK / NB * 4 / 8 / NW;
+    const int cb = warp % (DK / 8 / NB) * NB, mb = warp / (DK / 8 / NB) * MB;
+    float z[NB][MB][4];
 #pragma unroll
-        for (int b = 0; b < NB; ++b)
+    for (int b = 0; b < NB; ++b)
 #pragma unroll
-            for (int m = 0; m < 4; ++m)
+        for (int m = 0; m < MB; ++m)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) z[b][m][e] = 0.0f;
-        for (int k0 = 0; k0 < rank8; k0 += 16) {
-            const int ka = k0 + 2 * tq, kb = ka + 8;
-            uint32_t w[NB][2];
+            for (int e = 0; e < 4; ++e) z[b][m][e] = 0.0f;
+    for (int k0 = 0; k0 < rank8; k0 += 16) {
+        const int ka = k0 + 2 * tq, kb = ka + 8;
+        uint32_t w[NB][2];
 #pragma unroll
-            for (int b = 0; b < NB; ++b) {
-                const int d = (warp * NB + b) * 8 + g;
+        for (int b = 0; b < NB; ++b) {
+            const int d = (cb + b) * 8 + g;
+            if (pl.staged_decay) {
+                w[b][0] = *reinterpret_cast<const uint32_t*>(su + d * pl.PR + ka);
+                w[b][1] = *reinterpret_cast<const uint32_t*>(su + d * pl.PR + kb);
+            } else {
                 const uint16_t* up = a.up + (size_t)(h * a.dk + d) * a.ldu;
                 w[b][0] = d < a.dk && ka < rank8 ? *reinterpret_cast<const uint32_t*>(up + ka) : 0u;
                 w[b][1] = d < a.dk && kb < rank8 ? *reinterpret_cast<const uint32_t*>(up + kb) : 0u;
             }
+        }
 #pragma unroll
-            for (int m = 0; m < 4; ++m) {
-                const int ra = m * 16 + g, rb = ra + 8;
+        for (int m = 0; m < MB; ++m) {
+            const int ra = (mb + m) * 16 + g, rb = ra + 8;
+            uint32_t x[4];
+            if (pl.staged_decay) {
+                x[0] = *reinterpret_cast<const uint32_t*>(sa + ra * pl.PR + ka);
+                x[1] = *reinterpret_cast<const uint32_t*>(sa + rb * pl.PR + ka);
+                x[2] = *reinterpret_cast<const uint32_t*>(sa + ra * pl.PR + kb);
+                x[3] = *reinterpret_cast<const uint32_t*>(sa + rb * pl.PR + kb);
+            } else {
                 const uint16_t* pa = in + (size_t)(t0 + ra) * a.ld + a.a_off;
                 const uint16_t* pb = in + (size_t)(t0 + rb) * a.ld + a.a_off;
-                uint32_t x[4];
                 x[0] = ra < n && ka < rank8 ? *reinterpret_cast<const uint32_t*>(pa + ka) : 0u;
                 x[1] = rb < n && ka < rank8 ? *reinterpret_cast<const uint32_t*>(pb + ka) : 0u;
                 x[2] = ra < n && kb < rank8 ? *reinterpret_cast<const uint32_t*>(pa + kb) : 0u;
                 x[3] = rb < n && kb < rank8 ? *reinterpret_cast<const uint32_t*>(pb + kb) : 0u;
-#pragma unroll
-                for (int b = 0; b < NB; ++b) mma_bf16(z[b][m], x, w[b][0], w[b][1]);
             }
+#pragma unroll
+            for (int b = 0; b < NB; ++b) mma_bf16(z[b][m], x, w[b][0], w[b][1]);
         }
-#pragma unroll
-        for (int b = 0; b < NB; ++b)
-#pragma unroll
-            for (int m = 0; m < 4; ++m)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int t = m * 16 + g + (e >> 1) * 8, d = (warp * NB + b) * 8 + 2 * tq + (e & 1);
-                    float l = 0.0f;
-                    if (t < n && d < a.dk) l = log2_decay(a, z[b][m][e] + (a.bias != nullptr ? bf16_bits_to_f32(a.bias[h * a.dk + d]) : 0.0f), rate);
-                    G[t * P + d] = l;
-                }
     }
-    __syncthreads();
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+#pragma unroll
+        for (int m = 0; m < MB; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {  // tokens behind the last change nothing: decay 1
+                const int t = (mb + m) * 16 + g + (e >> 1) * 8, d = (cb + b) * 8 + 2 * tq + (e & 1);
+                z[b][m][e] = t < n && d < a.dk ? log2_decay(a, z[b][m][e] + (a.bias != nullptr ? bf16_bits_to_f32(a.bias[h * a.dk + d]) : 0.0f), rate) : 0.0f;
+            }
+    __syncthreads();  // the decay factor and map have been read
+    // ---- q and k
+    {
+        constexpr int PAIRS = DK / 2, STEP = NT / PAIRS;
+        const int d = (tid % PAIRS) * 2;
+        const float fq = a.unit_eps > 0.0f ? 1.0f : a.q_scale;
+        const bool live0 = d < a.dk, live1 = d + 1 < a.dk;
+        const uint16_t* wq = a.conv + (size_t)(chq + d) * a.taps;
+        const uint16_t* wk = a.conv + (size_t)(nq + chq + d) * a.taps;
+        for (int t = tid / PAIRS; t < kGC; t += STEP) {
+            float2 q = make_float2(0.0f, 0.0f), k = q;
+            if (live0 && t < n) {
+                q = staged_pair<DK>(a, raw_q, t, d, wq, live1 ? wq + a.taps : wq);
+                k = staged_pair<DK>(a, raw_k, t, d, wk, live1 ? wk + a.taps : wk);
+                if (!live1) q.y = k.y = 0.0f;
+            }
+            *reinterpret_cast<float2*>(Q + t * P + d) = make_float2(q.x * fq, q.y * fq);
+            *reinterpret_cast<float2*>(K + t * P + d) = k;
+        }
+    }
+    __syncthreads();  // the projected rows have been read
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+#pragma unroll
+        for (int m = 0; m < MB; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; e += 2)
+                *reinterpret_cast<float2*>(G + ((mb + m) * 16 + g + (e >> 1) * 8) * P + (cb + b) * 8 + 2 * tq) = make_float2(z[b][m][e], z[b][m][e + 1]);
     // ---- unit vectors; running sums of the log decays
     if (a.unit_eps > 0.0f)
-        for (int r = warp; r < 2 * kGC; r += kGThreads / 32) {
+        for (int r = warp; r < 2 * kGC; r += NW) {
             float* x = (r < kGC ? Q : K) + (r & (kGC - 1)) * P;
-            float s = 0.0f;
+            float v[DK / 32], s = 0.0f;
 #pragma unroll
-            for (int i = 0; i < DK / 32; ++i) s += x[lane + i * 32] * x[lane + i * 32];
+            for (int i = 0; i < DK / 32; ++i) { v[i] = x[lane + i * 32]; s += v[i] * v[i]; }
             const float f = (r < kGC ? a.q_scale : 1.0f) / sqrtf(warp_sum(s) + a.unit_eps);
 #pragma unroll
-            for (int i = 0; i < DK / 32; ++i) x[lane + i * 32] *= f;
+            for (int i = 0; i < DK / 32; ++i) x[lane + i * 32] = v[i] * f;
         }
+    __syncthreads();
     {
-        constexpr int SEG = kGThreads / DK, LEN = kGC / SEG;
+        constexpr int SEG = NT / DK, LEN = kGC / SEG;
         const int d = tid % DK, seg = tid / DK;
-        float run = 0.0f;
+        float run[LEN];
 #pragma unroll
-        for (int i = 0; i < LEN; ++i) {
-            run += G[(seg * LEN + i) * P + d];
-            G[(seg * LEN + i) * P + d] = run;
-        }
-        total[seg * DK + d] = run;
+        for (int i = 0; i < LEN; ++i) run[i] = G[(seg * LEN + i) * P + d];
+#pragma unroll
+        for (int i = 1; i < LEN; ++i) run[i] += run[i - 1];
+        total[seg * DK + d] = run[LEN - 1];
         __syncthreads();
         float before = 0.0f;
         for (int s = 0; s < seg; ++s) before += total[s * DK + d];
-        if (seg > 0)
 #pragma unroll
-            for (int i = 0; i < LEN; ++i) G[(seg * LEN + i) * P + d] += before;
+        for (int i = 0; i < LEN; ++i) G[(seg * LEN + i) * P + d] = run[i] + before;
     }
     __syncthreads();
-    // ---- A and L: six 16 x 16 blocks below the diagonal, then the pairs on the diagonal blocks, 32 at a time
+    // ---- A (to its planes) and L: six 16 x 16 blocks below the diagonal, then the pairs on the diagonal blocks, 32 at a time
     constexpr int kPairs = 136, kUnits = 6 + 4 * kPairs / 32;
-    for (int u = warp; u < kUnits; u += kGThreads / 32) {
+    for (int u = warp; u < kUnits; u += NW) {
         if (u < 6) {
             const int I = u < 1 ? 1 : u < 3 ? 2 : 3, J = u - (I * (I - 1)) / 2, ref = I * 16 - 1;
             const int ia = I * 16 + g, ib = ia + 8;
@@ -453,10 +646,13 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const Ch
 #pragma unroll
             for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int i = (e >> 1) ? ib : ia, j = J * 16 + nb * 8 + 2 * tq + (e & 1);
-                    A[i * kAP + j] = ca_[nb][e];
-                    if (DELTA) L[i * kAP + j] = beta[i] * cl_[nb][e];
+                for (int e = 0; e < 4; e += 2) {
+                    const int i = (e >> 1) ? ib : ia, j = J * 16 + nb * 8 + 2 * tq;
+                    uint32_t hi, lo;
+                    split_bf16x2(ca_[nb][e], ca_[nb][e + 1], hi, lo);
+                    *reinterpret_cast<uint32_t*>(Ah + i * kGC + j) = hi;
+                    *reinterpret_cast<uint32_t*>(Al + i * kGC + j) = lo;
+                    if (DELTA) *reinterpret_cast<float2*>(L + i * kAP + j) = make_float2(beta[i] * cl_[nb][e], beta[i] * cl_[nb][e + 1]);
                 }
         } else {
             const int p = (u - 6) * 32 + lane, B = p / kPairs, r = p - B * kPairs;
@@ -465,28 +661,33 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const Ch
             if ((i + 1) * (i + 2) / 2 <= r) ++i;
             const int j = B * 16 + r - i * (i + 1) / 2;
             i += B * 16;
-            float sa = 0.0f, sl = 0.0f;
-#pragma unroll 2
+            float sq = 0.0f, sl = 0.0f;
+#pragma unroll 4
             for (int d = 0; d < DK; d += 4) {
                 const float4 gi = *reinterpret_cast<const float4*>(G + i * P + d), gj = *reinterpret_cast<const float4*>(G + j * P + d);
                 const float4 kj = *reinterpret_cast<const float4*>(K + j * P + d), qi = *reinterpret_cast<const float4*>(Q + i * P + d);
                 const float w0 = kj.x * ex2_approx(gi.x - gj.x), w1 = kj.y * ex2_approx(gi.y - gj.y), w2 = kj.z * ex2_approx(gi.z - gj.z),
                             w3 = kj.w * ex2_approx(gi.w - gj.w);
-                sa += qi.x * w0 + qi.y * w1 + qi.z * w2 + qi.w * w3;
+                sq += qi.x * w0 + qi.y * w1 + qi.z * w2 + qi.w * w3;
                 if (DELTA) {
                     const float4 ki = *reinterpret_cast<const float4*>(K + i * P + d);
                     sl += ki.x * w0 + ki.y * w1 + ki.z * w2 + ki.w * w3;
                 }
             }
-            A[i * kAP + j] = sa;
-            if (DELTA && j < i) L[i * kAP + j] = beta[i] * sl;
+            const uint16_t hi = f32_to_bf16_bits(sq);
+            Ah[i * kGC + j] = hi;
+            Al[i * kGC + j] = f32_to_bf16_bits(sq - bf16_bits_to_f32(hi));
+            if (j < i) {  // the mirrored place above the diagonal
+                Ah[j * kGC + i] = 0;
+                Al[j * kGC + i] = 0;
+                if (DELTA) L[i * kAP + j] = beta[i] * sl;
+            }
         }
     }
     __syncthreads();
-    // ---- planes of q, k and A; the inverse of I + L by forward substitution, one column per thread of the first two warps
+    // ---- planes of q and k; the inverse of I + L by forward substitution, one column per thread of the first two warps
     if (!DELTA || warp >= 2) {
-        const int first = DELTA ? tid - 64 : tid, step = DELTA ? kGThreads - 64 : kGThreads;
-        const size_t pl = lay.plane * 2;
+        const int first = DELTA ? tid - 64 : tid, step = DELTA ? NT - 64 : NT;
         for (int i = first; i < kGC * DK / 2; i += step) {
             const int t = i / (DK / 2), d = (i % (DK / 2)) * 2;
             const float2 gt = *reinterpret_cast<const float2*>(G + t * P + d), gn = *reinterpret_cast<const float2*>(G + (kGC - 1) * P + d);
@@ -495,18 +696,10 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const Ch
             uint32_t* p = reinterpret_cast<uint32_t*>(planes) + i;
             split_bf16x2(q.x * ex2_approx(gt.x), q.y * ex2_approx(gt.y), hi, lo);
             p[0] = hi;
-            p[pl / 2] = lo;
+            p[lay.plane] = lo;
             split_bf16x2(k.x * ex2_approx(gn.x - gt.x), k.y * ex2_approx(gn.y - gt.y), hi, lo);
-            p[pl] = hi;
-            p[3 * (pl / 2)] = lo;
-        }
-        uint32_t* ap = reinterpret_cast<uint32_t*>(out + (DELTA ? 6 : 4) * lay.plane);
-        for (int i = first; i < kGC * kGC / 2; i += step) {
-            const float2 v = *reinterpret_cast<const float2*>(A + (i / (kGC / 2)) * kAP + (i % (kGC / 2)) * 2);
-            uint32_t hi, lo;
-            split_bf16x2(v.x, v.y, hi, lo);
-            ap[i] = hi;
-            ap[lay.a_plane + i] = lo;
+            p[2 * lay.plane] = hi;
+            p[3 * lay.plane] = lo;
         }
         float* dn = out + (DELTA ? 6 : 4) * lay.plane + 2 * lay.a_plane;
         for (int d = first; d < DK; d += step) dn[d] = ex2_approx(G[(kGC - 1) * P + d]);
@@ -533,29 +726,41 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const Ch
     }
     if (!DELTA) return;
     __syncthreads();
-    // ---- W = X (beta k 2^G), U0 = X (beta v): right-hand sides into Q's place, DK columns at a time
-    for (int i = tid; i < kGC * DK; i += kGThreads) {
+    // ---- W = X (beta k 2^G), U0 = X (beta v): right-hand sides in K's place and, DK columns at a time, in Q's
+    for (int i = tid; i < kGC * DK; i += NT) {
         const int t = i / DK, d = i % DK;
         K[t * P + d] *= beta[t] * ex2_approx(G[t * P + d]);
     }
     const int tiles = (ca.dvp + DK - 1) / DK;
     for (int tile = -1; tile < tiles; ++tile) {
-        const float* R = K;
-        if (tile >= 0) {
+        if (tile > 0) {
             __syncthreads();
-            for (int i = tid; i < kGC * DK; i += kGThreads) {
-                const int t = i / DK, col = tile * DK + i % DK;
-                float v = 0.0f;
-                if (t < n && col < a.dv) v = beta[t] * convolved<false>(a, t0 + t, a.pos0 + t0 + t, a.v_off + h * a.dv + col, 2 * nq + h * a.dv + col, channels);
-                Q[t * P + i % DK] = v;
-            }
-            R = Q;
+            stage_rows<DK, NT>(a, raw_v, t0, n, a.v_off + h * a.dv + tile * DK, chv + tile * DK, a.dv - tile * DK, channels, fast);
+            asm volatile("cp.async.commit_group;" ::: "memory");
         }
+        if (tile >= 0) {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            __syncthreads();
+            constexpr int PAIRS = DK / 2;
+            const int d = (tid % PAIRS) * 2, col = tile * DK + d;
+            const uint16_t* w = a.conv + (size_t)(chv + col) * a.taps;
+            for (int t = tid / PAIRS; t < kGC; t += NT / PAIRS) {
+                float2 v = make_float2(0.0f, 0.0f);
+                if (t < n && col < a.dv) {
+                    v = staged_pair<DK>(a, raw_v, t, d, w, col + 1 < a.dv ? w + a.taps : w);
+                    v.x *= beta[t];
+                    v.y = col + 1 < a.dv ? v.y * beta[t] : 0.0f;
+                }
+                *reinterpret_cast<float2*>(Q + t * P + d) = v;
+            }
+        }
+        const float* R = tile < 0 ? K : Q;
         __syncthreads();
-        constexpr int NB = DK / 64;  // column blocks of 8 per warp
+        constexpr int CB = DK / 8, MG = NW / CB < 1 ? 1 : NW / CB, NBW = CB / (NW / MG);  // warps over column blocks, then over row blocks
+        const int wc = warp % (NW / MG) * NBW, wm = warp / (NW / MG);
 #pragma unroll 1
-        for (int m = 0; m < 4; ++m) {
-            float acc[NB][4] = {};
+        for (int m = wm; m < 4; m += MG) {
+            float acc[NBW][4] = {};
             for (int ks = 0; ks <= m; ++ks) {  // X is lower triangular
                 uint32_t xh[4], xl[4];
 #pragma unroll
@@ -564,8 +769,8 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const Ch
                     for (int y = 0; y < 2; ++y)
                         split_pair(*reinterpret_cast<const float2*>(L + (m * 16 + g + y * 8) * kAP + ks * 16 + x * 8 + 2 * tq), xh[x * 2 + y], xl[x * 2 + y]);
 #pragma unroll
-                for (int b = 0; b < NB; ++b) {
-                    const int d = (warp * NB + b) * 8 + g;
+                for (int b = 0; b < NBW; ++b) {
+                    const int d = (wc + b) * 8 + g;
                     uint32_t bh[2], bl[2];
 #pragma unroll
                     for (int x = 0; x < 2; ++x) {
@@ -576,10 +781,10 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_prepare_kernel(const Ch
                 }
             }
 #pragma unroll
-            for (int b = 0; b < NB; ++b)
+            for (int b = 0; b < NBW; ++b)
 #pragma unroll
                 for (int e = 0; e < 4; e += 2) {
-                    const int t = m * 16 + g + (e >> 1) * 8, d = (warp * NB + b) * 8 + 2 * tq;
+                    const int t = m * 16 + g + (e >> 1) * 8, d = (wc + b) * 8 + 2 * tq;
                     if (tile < 0) {
                         uint32_t hi, lo;
                         split_bf16x2(acc[b][e], acc[b][e + 1], hi, lo);
@@ -807,11 +1012,11 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_scan_kernel(const Chunk
 
 template <int DK, bool DELTA>
 int run_chunked(cudaStream_t stream, const ChunkArgs& ca) {
-    constexpr size_t s1 = ((size_t)3 * kGC * (DK + 4) + (DELTA ? 2 : 1) * kGC * kAP) * 4;
+    const size_t s1 = (size_t)prepare_layout(DK, DELTA ? 1 : 0, ca.a.taps, ca.a.rank).total;
     constexpr size_t s2 = ((size_t)(DELTA ? 6 : 4) * kGC * (DK + 8) + 2 * kGC * (kGC + 8) + 2 * (size_t)DK * 40 + 2 * kGC * 40) * 2 + (size_t)DK * 4;
     cudaError_t e = allow_all_dynamic_smem(gated_chunk_prepare_kernel<DK, DELTA>);
     if (e == cudaSuccess) e = allow_all_dynamic_smem(gated_chunk_scan_kernel<DK, DELTA>);
-    if (e == cudaSuccess) e = launch(gated_chunk_prepare_kernel<DK, DELTA>, dim3(ca.chunks, ca.a.heads), dim3(kGThreads), s1, stream, true, ca);
+    if (e == cudaSuccess) e = launch(gated_chunk_prepare_kernel<DK, DELTA>, dim3(ca.chunks, ca.a.heads), dim3(DELTA ? 512 : 256), s1, stream, true, ca);
     if (e == cudaSuccess) e = launch(gated_chunk_scan_kernel<DK, DELTA>, dim3(ca.a.heads, ca.dvp / 32), dim3(kGThreads), s2, stream, true, ca);
     if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "gated linear attention (chunked): %s", cudaGetErrorString(e));
     return KMLL_OK;
@@ -826,7 +1031,7 @@ int gated_linear_steps(cudaStream_t stream, const GatedLinearArgs& a) {
 }
 
 bool gated_linear_chunked_ok(const GatedLinearArgs& a) {
-    return !a.in_f32 && a.dk <= 128 && a.T >= 4 && a.taps <= kMaxConvTaps && ((a.ld | a.a_off | a.ldu) & 7) == 0;
+    return !a.in_f32 && a.dk <= 128 && a.T >= 4 && a.taps <= kMaxConvTaps && ((a.ld | a.a_off | a.ldu) & 7) == 0 && (reinterpret_cast<uintptr_t>(a.in) & 15u) == 0;
 }
 size_t gated_chunk_scratch_floats(int T, int heads, int dk, int dv, int delta) {
     if (dk > 128) return 4;

@@ -4,7 +4,7 @@
 //
 //   plain form    any size, f32 arithmetic, one block per (token, head): decoders that compute in f32, sizes the others lack
 //   decode form   one token over the bf16 cache: up to 16 query heads of a group are the rows of the MMAs, so the cache is read
-//                 once per group; positions split over blocks, merged by the block that arrives last
+//                 once per group; positions split over the blocks of a cluster, which merge their parts through shared memory
 //   prompt form   tiled attention with online softmax over the cache rows
 // Scores and weights are f32; the weights (and in a decode step the queries) meet the tensor cores split into a bf16 head and
 // remainder.
@@ -87,19 +87,16 @@ __global__ void __launch_bounds__(kPlainWarps * 32) grouped_plain_kernel(const G
 }
 
 // ---- decode form ------------------------------------------------------------------------------------------------------------------
-constexpr int kDT = 128;     // positions per tile
+constexpr int kDT = 160;     // positions per tile
 constexpr int kDRows = 16;   // query heads per block = MMA rows
 constexpr int kDWarps = 8;
-constexpr int kDMaxSplit = 32;
-constexpr int kDMinPart = 64;  // positions per split at least
-struct GroupedPlan { int tiles_per_group, tiles, nsplit, kw, vw; };
+constexpr int kDMaxSplit = 16;
+constexpr int kDMinPart = 32;  // positions per split at least
+struct GroupedPlan { int tiles_per_group, tiles, kw, vw; };
 __host__ __device__ inline GroupedPlan decode_plan(int heads, int kv_heads, int dim, int vdim) {
     GroupedPlan p;
     p.tiles_per_group = (heads / kv_heads + kDRows - 1) / kDRows;
     p.tiles = kv_heads * p.tiles_per_group;
-    p.nsplit = 148 / p.tiles;
-    if (p.nsplit < 1) p.nsplit = 1;
-    if (p.nsplit > kDMaxSplit) p.nsplit = kDMaxSplit;
     p.kw = round_to(dim, 32);
     p.vw = round_to(vdim, 16);
     return p;
@@ -109,6 +106,30 @@ size_t decode_smem(const GroupedPlan& p) {
            ((size_t)kDRows * kDT + kDRows + (size_t)kDRows * kDMaxSplit) * 4;
 }
 
+__device__ inline uint32_t cluster_rank() {
+    uint32_t r;
+    asm("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
+    return r;
+}
+__device__ inline uint32_t cluster_size() {
+    uint32_t r;
+    asm("mov.u32 %0, %%cluster_nctaid.x;" : "=r"(r));
+    return r;
+}
+__device__ inline void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// the float at `p` (this block's shared memory) in block `rank` of the cluster
+__device__ inline float cluster_load(const float* p, uint32_t rank) {
+    uint32_t at;
+    float v;
+    asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"((uint32_t)__cvta_generic_to_shared(p)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(at) : "memory");
+    return v;
+}
+
+// One cluster per (key / value head, 16 query heads); its blocks share the positions.
 __global__ void __launch_bounds__(kDWarps * 32) grouped_decode_kernel(const GroupedArgs a, const GroupedPlan pl) {
     extern __shared__ __align__(16) uint16_t dsm[];
     const int KP = pl.kw + 8, VP = pl.vw + 8;
@@ -121,18 +142,14 @@ __global__ void __launch_bounds__(kDWarps * 32) grouped_decode_kernel(const Grou
     float* const sc = reinterpret_cast<float*>(plo + kDRows * (kDT + 8));  // [16][kDT]
     float* const corr = sc + kDRows * kDT;       // [16]
     float* const f = corr + kDRows;              // [16][kDMaxSplit]
-    __shared__ unsigned int s_last;
+    __shared__ float stat[2 * kDRows];           // maximum and sum of this block's part, per row
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
-    const int split = blockIdx.x, grp = blockIdx.y / pl.tiles_per_group, sub = blockIdx.y % pl.tiles_per_group;
+    const int split = (int)cluster_rank(), nsplit = (int)cluster_size(), grp = blockIdx.y / pl.tiles_per_group, sub = blockIdx.y % pl.tiles_per_group;
     const int per = a.heads / a.kv_heads, h0 = grp * per + sub * kDRows, nh = min(kDRows, per - sub * kDRows);
     // the position was written more than one launch ago, and so was every cache row but the newest
     const int pos = a.at->position, lo = first_seen(pos, a.window, a.chunk), count = pos - lo + 1;
-    const int part_len = max((count + pl.nsplit - 1) / pl.nsplit, kDMinPart), active = (count + part_len - 1) / part_len;
-    const int begin = lo + split * part_len, end = min(begin + part_len, pos + 1);
-    if (split >= active) {
-        pdl_wait();
-        return;
-    }
+    const int part_len = max((count + nsplit - 1) / nsplit, kDMinPart), active = (count + part_len - 1) / part_len;
+    const int begin = lo + split * part_len, end = split < active ? min(begin + part_len, pos + 1) : begin;
     uint16_t* const cache = static_cast<uint16_t*>(a.cache);
     const size_t k0 = (size_t)grp * a.dimp, v0 = (size_t)a.kv_heads * a.dimp + (size_t)grp * a.vdimp;
     auto load_tile = [&](int t0) {  // rows behind the last position are zeros; the newest one comes from the projection
@@ -151,7 +168,7 @@ __global__ void __launch_bounds__(kDWarps * 32) grouped_decode_kernel(const Grou
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    load_tile(begin);
+    if (begin < end) load_tile(begin);
     pdl_wait();
     const float* in = static_cast<const float*>(a.in);
     auto put_newest = [&](int t0) {
@@ -258,60 +275,43 @@ __global__ void __launch_bounds__(kDWarps * 32) grouped_decode_kernel(const Grou
         }
         __syncthreads();
     }
+    // ---- the blocks' parts: (weighted values, maximum, sum) in shared memory, merged slice by slice
+    float* const part = reinterpret_cast<float*>(dsm);  // [16][vw], in the place of the key tile
     if (lane == 0) {
-        corr[warp] = l_run[0];
-        corr[warp + 8] = l_run[1];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            stat[warp + i * 8] = m_run[i];
+            stat[kDRows + warp + i * 8] = l_run[i];
+        }
     }
-    __syncthreads();
-    const size_t hs = a.vdim + 2, ss = (size_t)a.heads * hs;
-    float* const mine = a.work + (size_t)split * ss + (size_t)h0 * hs;
 #pragma unroll
     for (int i = 0; i < NG; ++i)
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = g + (e >> 1) * 8, c = (warp + i * kDWarps) * 16 + j * 8 + 2 * tq + (e & 1);
-                if (r >= nh || c >= a.vdim) continue;
-                if (active == 1) a.out[(size_t)(h0 + r) * a.vdim + c] = o[i][j][e] / corr[r];
-                else mine[r * hs + c] = o[i][j][e];
+            for (int e = 0; e < 4; e += 2) {
+                const int c = (warp + i * kDWarps) * 16 + j * 8 + 2 * tq;
+                if (c < pl.vw) *reinterpret_cast<float2*>(part + (g + (e >> 1) * 8) * pl.vw + c) = make_float2(o[i][j][e], o[i][j][e + 1]);
             }
-    if (active == 1) return;
-    if (lane == 0) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-            if (warp + i * 8 < nh) {
-                mine[(warp + i * 8) * hs + a.vdim] = m_run[i];
-                mine[(warp + i * 8) * hs + a.vdim + 1] = l_run[i];
-            }
-    }
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) s_last = atomicAdd(&a.counters[blockIdx.y], 1u) == (unsigned)active - 1u ? 1u : 0u;
-    __syncthreads();
-    if (s_last == 0u) return;
-    __threadfence();
-    const float* all = a.work + (size_t)h0 * hs;
+    cluster_sync();
     for (int r = warp; r < nh; r += kDWarps) {
         const bool on = lane < active;
-        const float m = on ? __ldcg(all + lane * ss + r * hs + a.vdim) : -INFINITY, l = on ? __ldcg(all + lane * ss + r * hs + a.vdim + 1) : 0.0f;
-        const float mx = warp_max(m), w = on ? expf(m - mx) : 0.0f, total = warp_sum(w * l);
-        f[r * kDMaxSplit + lane] = w / total;
+        const float m = on ? cluster_load(stat + r, lane) : -INFINITY, l = on ? cluster_load(stat + kDRows + r, lane) : 0.0f;
+        const float mx = warp_max(m), w = on ? expf(m - mx) : 0.0f, sum = warp_sum(w * l);
+        if (lane < kDMaxSplit) f[r * kDMaxSplit + lane] = w / sum;
     }
     __syncthreads();
-    for (int i = tid; i < nh * a.vdim; i += kDWarps * 32) {
+    const int outs = nh * a.vdim, slice = (outs + nsplit - 1) / nsplit;
+    for (int i = split * slice + tid; i < min((split + 1) * slice, outs); i += kDWarps * 32) {
         const int r = i / a.vdim, c = i - r * a.vdim;
-        float v = 0.0f;
-        for (int s0 = 0; s0 < active; s0 += 8) {
-            float x[8];
+        float x[kDMaxSplit], v = 0.0f;
 #pragma unroll
-            for (int s = 0; s < 8; ++s) x[s] = s0 + s < active ? __ldcg(all + (s0 + s) * ss + r * hs + c) : 0.0f;
+        for (int s = 0; s < kDMaxSplit; ++s) x[s] = s < active ? cluster_load(part + r * pl.vw + c, s) : 0.0f;
 #pragma unroll
-            for (int s = 0; s < 8; ++s) v = fmaf(f[r * kDMaxSplit + s0 + s], x[s], v);
-        }
+        for (int s = 0; s < kDMaxSplit; ++s) v = fmaf(s < active ? f[r * kDMaxSplit + s] : 0.0f, x[s], v);
         a.out[(size_t)(h0 + r) * a.vdim + c] = v;
     }
-    if (tid == 0) a.counters[blockIdx.y] = 0u;
+    cluster_sync();  // (no block leaves while another reads its part)
 }
 
 // ---- prompt form --------------------------------------------------------------------------------------------------------------------
@@ -501,18 +501,43 @@ int grouped_attention_plain(cudaStream_t stream, const GroupedArgs& a) {
     return KMLL_OK;
 }
 
-size_t grouped_decode_work_floats(int heads, int kv_heads, int vdim) {
-    return (size_t)decode_plan(heads, kv_heads, 1, vdim).nsplit * heads * (vdim + 2);
-}
 bool grouped_decode_ok(const GroupedArgs& a) {
     const GroupedPlan p = decode_plan(a.heads, a.kv_heads, a.dim, a.vdim);
-    return a.T == 1 && !a.cache_f32 && a.in_f32 && a.at != nullptr && a.vdim <= 16 * 2 * kDWarps && p.tiles <= kGroupedMaxTiles && decode_smem(p) <= 220 * 1024;
+    return a.T == 1 && !a.cache_f32 && a.in_f32 && a.at != nullptr && a.vdim <= 16 * 2 * kDWarps && p.tiles <= 65535 && decode_smem(p) <= 220 * 1024;
+}
+// Blocks per cluster: 16 where all clusters are resident at once with it, else the portable 8.
+static int decode_cluster(const GroupedPlan& p, size_t smem, int* out) {
+    *out = 8;
+    if (p.tiles * 16 > 148) return KMLL_OK;
+    cudaError_t e = cudaFuncSetAttribute(grouped_decode_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "grouped attention (decode): %s", cudaGetErrorString(e));
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(16, p.tiles);
+    cfg.blockDim = dim3(kDWarps * 32);
+    cfg.dynamicSmemBytes = smem;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = 16;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    int clusters = 0;
+    if (cudaOccupancyMaxActiveClusters(&clusters, grouped_decode_kernel, &cfg) != cudaSuccess) {
+        cudaGetLastError();  // (a device that has no such clusters)
+        clusters = 0;
+    }
+    if (clusters >= p.tiles) *out = 16;
+    return KMLL_OK;
 }
 int grouped_attention_decode(cudaStream_t stream, const GroupedArgs& a) {
     if (!grouped_decode_ok(a)) return fail(KMLL_ERR_UNSUPPORTED, "grouped attention: no decode form for %d / %d heads of %d, %d", a.heads, a.kv_heads, a.dim, a.vdim);
     const GroupedPlan p = decode_plan(a.heads, a.kv_heads, a.dim, a.vdim);
+    const size_t smem = decode_smem(p);
     cudaError_t e = allow_all_dynamic_smem(grouped_decode_kernel);
-    if (e == cudaSuccess) e = launch(grouped_decode_kernel, dim3(p.nsplit, p.tiles), dim3(kDWarps * 32), decode_smem(p), stream, true, a, p);
+    int cluster = 8;
+    if (e == cudaSuccess) KMLL_TRY_RC(decode_cluster(p, smem, &cluster));
+    if (e == cudaSuccess) e = launch_cluster(grouped_decode_kernel, dim3(cluster, p.tiles), cluster, dim3(kDWarps * 32), smem, stream, true, a, p);
     if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "grouped attention (decode): %s", cudaGetErrorString(e));
     return KMLL_OK;
 }

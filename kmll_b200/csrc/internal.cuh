@@ -360,13 +360,9 @@ struct GroupedArgs {
     int cache_f32, pitch, dimp, vdimp, max_seq;
     float* out;          // [T, ldo] f32
     int ldo;
-    float* work;         // decode: grouped_decode_work_floats()
-    unsigned int* counters;  // decode: kGroupedMaxTiles zeros, left so
 };
-constexpr int kGroupedMaxTiles = 1024;
 int grouped_write_cache(cudaStream_t stream, const GroupedArgs& a);
 int grouped_attention_plain(cudaStream_t stream, const GroupedArgs& a);   // any size, f32 arithmetic, after grouped_write_cache
-size_t grouped_decode_work_floats(int heads, int kv_heads, int vdim);
 bool grouped_decode_ok(const GroupedArgs& a);
 int grouped_attention_decode(cudaStream_t stream, const GroupedArgs& a);  // T = 1, bf16 cache; writes the cache row itself
 bool grouped_prefill_ok(const GroupedArgs& a);

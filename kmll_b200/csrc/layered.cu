@@ -72,7 +72,6 @@ struct Layered {
     int saved_at = -1;
     // one-token scratch
     float *proj1 = nullptr, *o1 = nullptr, *z1 = nullptr, *work = nullptr, *gate1 = nullptr;
-    unsigned int* split_counters = nullptr;
     // prompt scratch for `rows` tokens
     int rows = 0;
     std::vector<void*> row_allocs;
@@ -216,7 +215,6 @@ int create_mixer(Decoder* d, LMixer* m, size_t* work) {
         *work = std::max(*work, latent_decode_work_floats(s.heads, s.kv_rank, s.rot_dim, span));
     } else if (s.mixer == KMLL_MIXER_ATTENTION) {
         KMLL_TRY(cache(m->kv_heads() * (up8(s.dim) + up8(s.vdim))));
-        *work = std::max(*work, grouped_decode_work_floats(s.heads, m->kv_heads(), s.vdim));
     } else {
         if (s.out_norm == KMLL_OUT_NORM_JOINT) KMLL_TRY(alloc_vec(d, &m->mix_norm, s.heads * s.vdim));
         if (s.out_norm == KMLL_OUT_NORM_HEAD_WEIGHTED) KMLL_TRY(alloc_vec(d, &m->mix_norm, s.vdim));
@@ -307,8 +305,6 @@ int create(Decoder* d, const kmll_layered_config& c, const kmll_layer_spec* spec
     KMLL_TRY(dalloc(d, &L->saved_logits, (size_t)c.vocab_size));
     KMLL_TRY(dalloc(d, &L->counter, (size_t)4));
     KMLL_CUDA(cudaMemset(L->counter, 0, 16));
-    KMLL_TRY(dalloc(d, &L->split_counters, (size_t)kGroupedMaxTiles));
-    KMLL_CUDA(cudaMemset(L->split_counters, 0, kGroupedMaxTiles * 4));
     KMLL_TRY(dalloc(d, &L->token_log, (size_t)c.max_seq_len));
     KMLL_CUDA(cudaMemset(L->token_log, 0, (size_t)c.max_seq_len * 4));
     KMLL_TRY(dalloc(d, &L->proj1, (size_t)L->ldp));
@@ -376,8 +372,6 @@ GroupedArgs grouped_args(const Layered* L, const LMixer& m) {
     a.heads = m.sp.heads; a.kv_heads = m.kv_heads(); a.dim = m.sp.dim; a.vdim = m.sp.vdim; a.window = m.sp.window; a.chunk = m.sp.chunk;
     a.scale = m.sp.score_scale;
     a.cache = m.cache; a.cache_f32 = L->cfg.compute_f32; a.pitch = m.pitch; a.dimp = up8(m.sp.dim); a.vdimp = up8(m.sp.vdim); a.max_seq = L->cfg.max_seq_len;
-    a.work = L->work;
-    a.counters = L->split_counters;
     return a;
 }
 GatedLinearArgs gated_args(const Layered* L, const LMixer& m) {

@@ -183,13 +183,8 @@ int kmll_mixer_output_linear_bf16(kmll_stream_t s, const kmll_mixer_spec* mixers
     return bf16_matvec(as_stream(s), v);
 }
 
-size_t kmll_grouped_attention_workspace_bytes(const kmll_mixer_spec* m) {
-    if (m == nullptr || m->heads <= 0 || m->vdim <= 0) return 0;
-    return kGroupedMaxTiles * 4 + grouped_decode_work_floats(m->heads, m->kv_heads > 0 ? m->kv_heads : m->heads, m->vdim) * 4;
-}
-
 int kmll_grouped_attention(kmll_stream_t s, const kmll_mixer_spec* m, const void* in, int in_f32, int ld, int q_off, int k_off, int v_off, int tokens, int position,
-                           const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, void* workspace, float* out, int ldo) {
+                           const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, float* out, int ldo) {
     KMLL_REQUIRE_PTR(m); KMLL_REQUIRE_PTR(in); KMLL_REQUIRE_PTR(cache); KMLL_REQUIRE_PTR(out);
     const int g = m->kv_heads > 0 ? m->kv_heads : m->heads;
     KMLL_REQUIRE(m->heads > 0 && m->heads % g == 0 && m->dim > 0 && m->vdim > 0 && m->window >= 0 && m->chunk >= 0 && tokens > 0 && position >= 0 &&
@@ -203,11 +198,7 @@ int kmll_grouped_attention(kmll_stream_t s, const kmll_mixer_spec* m, const void
     a.pos0 = position;
     a.cache = cache; a.cache_f32 = cache_f32; a.pitch = pitch; a.dimp = up8(m->dim); a.vdimp = up8(m->vdim); a.max_seq = max_seq;
     a.out = out; a.ldo = ldo;
-    if (workspace != nullptr) {
-        a.counters = static_cast<unsigned int*>(workspace);
-        a.work = static_cast<float*>(workspace) + kGroupedMaxTiles;
-        if (grouped_decode_ok(a)) return grouped_attention_decode(as_stream(s), a);
-    }
+    if (grouped_decode_ok(a)) return grouped_attention_decode(as_stream(s), a);
     KMLL_TRY_RC(grouped_write_cache(as_stream(s), a));
     return position_device == nullptr && grouped_prefill_ok(a) ? grouped_attention_prefill(as_stream(s), a) : grouped_attention_plain(as_stream(s), a);
 }

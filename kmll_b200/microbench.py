@@ -519,8 +519,8 @@ def suite_somopel(reps, cpu=None, only="", context=2048):
 
         if want("mixer decode"):
             caches = [bf(n + 64, kv, std=0.5) for _ in range(48)]
-            x, out, ws = torch.randn((1, (H + 2 * G) * D), device="cuda"), torch.empty((1, H * D), device="cuda"), ops.grouped_attention_workspace(att)
-            us = time_graph([lambda c=c: ops.grouped_attention(att, x, aoff, pos, c, ws, out) for c in caches], reps)
+            x, out = torch.randn((1, (H + 2 * G) * D), device="cuda"), torch.empty((1, H * D), device="cuda")
+            us = time_graph([lambda c=c: ops.grouped_attention(att, x, aoff, pos, c, out) for c in caches], reps)
             report(f"mixer decode attention {H}/{G} heads x {D}, bf16 cache, context {n}", us, n * kv * 2)
             del caches
             caches = [(torch.randn((n + 64) * G * D, device="cuda"), torch.randn((n + 64) * G * D, device="cuda")) for _ in range(24)]
@@ -561,7 +561,7 @@ def suite_somopel(reps, cpu=None, only="", context=2048):
             for chunk in (SOMOPEL_CHUNK, 512):
                 att.chunk = chunk
                 seen = min(chunk, T)
-                us = time_graph([lambda i=i: ops.grouped_attention(att, xs[i], aoff, 0, caches[i], None, out) for i in range(4)], reps)
+                us = time_graph([lambda i=i: ops.grouped_attention(att, xs[i], aoff, 0, caches[i], out) for i in range(4)], reps)
                 report(f"mixer prompt attention (2 launches) {T} tokens, {H}/{G} heads x {D}, chunk {chunk}", us, T * (H + 2 * G) * D * 2 + T * kv * 2 + T * H * D * 4,
                        flops=2.0 * H * T * seen * D)
             att.chunk = SOMOPEL_CHUNK

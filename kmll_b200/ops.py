@@ -683,11 +683,7 @@ def mixer_output_linear_bf16(mixers, x, norm_weights, gates, w, eps: float, resi
     return out
 
 
-def grouped_attention_workspace(mixer, device="cuda") -> torch.Tensor:
-    return torch.zeros(load().kmll_grouped_attention_workspace_bytes(C.byref(mixer._mixer())) // 4, dtype=torch.float32, device=device)
-
-
-def grouped_attention(mixer, qkv, offsets, position, cache, workspace=None, out=None):
+def grouped_attention(mixer, qkv, offsets, position, cache, out=None):
     """qkv [tokens, ld] f32 or bf16 with q, k, v at `offsets`; position: an int, or an int32 tensor on the device; cache
     [max_seq, pitch] f32 or bf16 (the tokens' rows are written)."""
     tokens, ld = qkv.shape
@@ -695,7 +691,7 @@ def grouped_attention(mixer, qkv, offsets, position, cache, workspace=None, out=
     dev = isinstance(position, torch.Tensor)
     check(load().kmll_grouped_attention(_stream(), C.byref(mixer._mixer()), _p(qkv), 1 if qkv.dtype == torch.float32 else 0, ld, *offsets, tokens,
                                         0 if dev else position, _p(position) if dev else None, _p(cache), 1 if cache.dtype == torch.float32 else 0, cache.shape[1],
-                                        cache.shape[0], _p(workspace), _p(out), out.shape[1]))
+                                        cache.shape[0], _p(out), out.shape[1]))
     return out
 
 

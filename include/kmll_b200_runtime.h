@@ -306,7 +306,7 @@ int kmll_mixer_output_linear_bf16(kmll_stream_t stream, const kmll_mixer_spec* m
 int kmll_grouped_attention(kmll_stream_t stream, const kmll_mixer_spec* mixer, const void* in, int in_f32, int ld, int q_off, int k_off, int v_off, int tokens,
                            int position, const int* position_device, void* cache, int cache_f32, int pitch, int max_seq, float* out, int ldo);
 /* Gated linear attention.  in [tokens, ld]: q, k, v, the decay factor (decay_rank), the logits of beta (heads) and the gate factor
- * (gate_rank) at offsets[0 .. 5].  conv [q | k | v channels][taps]; ring [taps][channels] f32 holds the inputs of earlier
+ * (gate_rank) at offsets[0 .. 5]; the maps' columns are padded with zeros to their pitch (a multiple of 8).  conv [q | k | v channels][taps]; ring [taps][channels] f32 holds the inputs of earlier
  * positions.  state [heads, dim, vdim] f32 and ring are updated.  scratch == null: token after token in f32, the low-rank gate goes
  * to gate [tokens, heads*vdim]; else (bf16 input, dim up to 128, 4 or more tokens) chunks of 64 tokens on the tensor cores,
  * _scratch_floats() floats, no gate. */

@@ -52,19 +52,18 @@ __device__ inline float convolved(const GatedLinearArgs& a, int t, int pos, int 
     for (int j = 0; j < a.taps; ++j) y = fmaf(bf16_bits_to_f32(w[j]), earlier<F32>(a, t, pos, a.taps - 1 - j, col, ch, channels), y);
     return act_silu(y);
 }
-// dot product of a bf16 row of n (a multiple of 8, 16-byte aligned) with f32 values
-__device__ inline float dot_row(const uint16_t* w, const float* x, int n) {
-    float s = 0.0f;
-    for (int r = 0; r < n; r += 8) {
-        const uint4 t = *reinterpret_cast<const uint4*>(w + r);
-        const uint32_t ww[4] = {t.x, t.y, t.z, t.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            s = fmaf(__uint_as_float(ww[e] << 16), x[r + 2 * e], s);
-            s = fmaf(__uint_as_float(ww[e] & 0xffff0000u), x[r + 2 * e + 1], s);
-        }
-    }
-    return s;
+// dot product of eight bf16 weights with eight values (both 16-byte aligned)
+__device__ inline float dot8(const uint16_t* w, const float* x) {
+    const uint4 t = *reinterpret_cast<const uint4*>(w);
+    const float4 u = *reinterpret_cast<const float4*>(x), v = *reinterpret_cast<const float4*>(x + 4);
+    float s = __uint_as_float(t.x << 16) * u.x, r = __uint_as_float(t.z << 16) * v.x;
+    s = fmaf(__uint_as_float(t.x & 0xffff0000u), u.y, s);
+    r = fmaf(__uint_as_float(t.z & 0xffff0000u), v.y, r);
+    s = fmaf(__uint_as_float(t.y << 16), u.z, s);
+    r = fmaf(__uint_as_float(t.w << 16), v.z, r);
+    s = fmaf(__uint_as_float(t.y & 0xffff0000u), u.w, s);
+    r = fmaf(__uint_as_float(t.w & 0xffff0000u), v.w, r);
+    return s + r;
 }
 
 // ---- step form ------------------------------------------------------------------------------------------------------------------
@@ -74,7 +73,7 @@ __device__ inline float dot_row(const uint16_t* w, const float* x, int n) {
 constexpr int kSThreads = 256, kSCols = 32;
 struct StepLayout {
     int dkr, rank8, gate8, chans;  // padded sizes; channels a block convolves
-    int off_part, off_maps;        // in floats / bytes: partial convolutions, then the staged maps
+    int off_part, off_maps;        // in floats: partial convolutions; in bytes: the staged maps
     bool staged;
     int total;
 };
@@ -94,7 +93,7 @@ __host__ __device__ inline StepLayout step_layout(int dk, int rank, int gate_ran
 
 template <bool F32, int RP>
 __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinearArgs a) {
-    extern __shared__ __align__(16) float ssm[];  // q | k | decay, [dk] each | v [32] | a [rank] | g [gate_rank], padded | ..
+    extern __shared__ __align__(16) float ssm[];  // q | k | decay, [dk] each | v [32] | decay factor | gate factor | ..
     const StepLayout sl = step_layout(a.dk, a.rank, a.gate_rank, a.taps);
     const int rank8 = sl.rank8, gate8 = sl.gate8;
     float* const sq = ssm;
@@ -105,7 +104,6 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
     float* const sgr = sa + rank8;
     float* const early = ssm + sl.off_part;       // one token: sum over the earlier taps, then the last tap, per channel
     uint16_t* const maps = reinterpret_cast<uint16_t*>(reinterpret_cast<unsigned char*>(ssm) + sl.off_maps);
-    __shared__ float dots[4];  // q.q, k.k, q.k, beta
     const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int col0 = blockIdx.y * kSCols, lc = warp * 4, c0 = col0 + lc;
     const int per = a.heads / a.kv_heads, hq = h / per, nq = a.kv_heads * a.dk, channels = 2 * nq + a.heads * a.dv;
@@ -165,14 +163,23 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
         return col0 + c < a.dv;
     };
     if (single && a.taps > 0)
+#pragma unroll 2
         for (int i = tid; i < sl.chans; i += kSThreads) {
             int col, ch;
             float y = 0.0f, last = 0.0f;
             if (place(i, col, ch)) {
                 const uint16_t* w = a.conv + (size_t)ch * a.taps;
-                for (int j = 0; j + 1 < a.taps; ++j) {
-                    const int p = pos0 - (a.taps - 1 - j);
-                    if (p >= 0) y = fmaf(bf16_bits_to_f32(w[j]), a.ring[(size_t)(p % a.taps) * channels + ch], y);
+                for (int j0 = 0; j0 + 1 < a.taps; j0 += 4) {  // four loads in flight
+                    float x[4], f[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const int p = pos0 - (a.taps - 1 - j0 - j);
+                        const bool live = j0 + j + 1 < a.taps && p >= 0;
+                        x[j] = live ? a.ring[(size_t)(p % a.taps) * channels + ch] : 0.0f;
+                        f[j] = live ? bf16_bits_to_f32(w[j0 + j]) : 0.0f;
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) y = fmaf(f[j], x[j], y);
                 }
                 last = bf16_bits_to_f32(w[a.taps - 1]);
             }
@@ -184,46 +191,51 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
     for (int t = 0; t < a.T; ++t) {
         const int pos = pos0 + t;
         const size_t row = (size_t)t * a.ld;
-        // ---- q, k, v, and the inputs of the low-rank maps
-        for (int i = tid; i < sl.chans + rank8 + gate8; i += kSThreads) {
-            if (i < sl.chans) {
-                int col, ch;
-                float y = 0.0f;
-                if (place(i, col, ch)) {
-                    if (single && a.taps > 0) {
-                        const float x = in_at<F32>(a.in, col);
-                        y = act_silu(fmaf(early[sl.chans + i], x, early[i]));
-                        if (i >= 2 * a.dk || (blockIdx.y == 0 && h == hq * per)) a.ring[(size_t)(pos % a.taps) * channels + ch] = x;
+        // ---- q, k, v; decays (two lanes per channel); gate (eight lanes per column)
+        const int entries = sl.chans + rank8 + gate8;
+        for (int i0 = tid; i0 < entries; i0 += 4 * kSThreads) {
+            float x[4];
+            int ch[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {  // four loads in flight
+                const int i = i0 + j * kSThreads, r = i - sl.chans;
+                int col = -1;
+                ch[j] = -1;
+                if (i < sl.chans) {
+                    if (!place(i, col, ch[j])) col = ch[j] = -1;
+                } else if (i < entries) {
+                    if (r < rank8) col = r < a.rank ? a.a_off + r : -1;
+                    else col = r - rank8 < a.gate_rank ? a.g_off + r - rank8 : -1;
+                }
+                x[j] = col >= 0 ? in_at<F32>(a.in, row + col) : 0.0f;
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int i = i0 + j * kSThreads;
+                if (i >= entries) break;
+                float y = x[j];
+                if (ch[j] >= 0 && a.taps > 0) {
+                    if (single) {
+                        y = act_silu(fmaf(early[sl.chans + i], x[j], early[i]));
+                        if (i >= 2 * a.dk || (blockIdx.y == 0 && h == hq * per)) a.ring[(size_t)(pos % a.taps) * channels + ch[j]] = x[j];
                     } else {
-                        y = convolved<F32>(a, t, pos, col, ch, channels);
+                        int col, unused;
+                        place(i, col, unused);
+                        y = convolved<F32>(a, t, pos, col, ch[j], channels);
                     }
                 }
-                (i < a.dk ? sq : i < 2 * a.dk ? sk - a.dk : sv - 2 * a.dk)[i] = y;
-            } else if (i < sl.chans + rank8) {
-                const int r = i - sl.chans;
-                sa[r] = r < a.rank ? in_at<F32>(a.in, row + a.a_off + r) : 0.0f;
-            } else {
-                const int r = i - sl.chans - rank8;
-                sgr[r] = r < a.gate_rank ? in_at<F32>(a.in, row + a.g_off + r) : 0.0f;
+                (i < a.dk ? sq : i < 2 * a.dk ? sk - a.dk : sv - 2 * a.dk)[i] = y;  // (the factors follow v)
             }
         }
-        if (warp == 3 && lane == 0) dots[3] = a.delta ? act_sigmoid(in_at<F32>(a.in, row + a.b_off + h)) : 1.0f;
+        const float beta = a.delta ? act_sigmoid(in_at<F32>(a.in, row + a.b_off + h)) : 1.0f;
         if (t == 0 && sl.staged) asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        // ---- decays (two lanes per channel), norms of q and k, gate (eight lanes per column)
-        if (warp < 3) {
-            const float* x = warp == 1 ? sk : sq;
-            const float* y = warp == 0 ? sq : sk;
-            float d = 0.0f;
-            for (int i = lane; i < a.dk; i += 32) d = fmaf(x[i], y[i], d);
-            d = warp_sum(d);
-            if (lane == 0) dots[warp] = d;
-        }
         for (int i0 = 0; i0 < 2 * a.dk; i0 += kSThreads) {
             const int d = (i0 + tid) >> 1;
             float z = 0.0f;
             if (d < a.dk)
-                for (int r = (tid & 1) * 8; r < rank8; r += 16) z += dot_row(up + (size_t)d * up_pitch + r, sa + r, 8);
+#pragma unroll 4
+                for (int r = (tid & 1) * 8; r < rank8; r += 16) z += dot8(up + (size_t)d * up_pitch + r, sa + r);
             z += __shfl_xor_sync(0xffffffffu, z, 1);
             if (d < a.dk && (tid & 1) == 0) {
                 if (a.bias != nullptr) z += bf16_bits_to_f32(a.bias[h * a.dk + d]);
@@ -234,7 +246,7 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
             const int c = tid >> 3, part = tid & 7;
             float g = 0.0f;
             if (col0 + c < a.dv)
-                for (int r = part * 8; r < gate8; r += 64) g += dot_row(gate_up + (size_t)c * gate_pitch + r, sgr + r, 8);
+                for (int r = part * 8; r < gate8; r += 64) g += dot8(gate_up + (size_t)c * gate_pitch + r, sgr + r);
             g += __shfl_xor_sync(0xffffffffu, g, 1);
             g += __shfl_xor_sync(0xffffffffu, g, 2);
             g += __shfl_xor_sync(0xffffffffu, g, 4);
@@ -242,49 +254,50 @@ __global__ void __launch_bounds__(kSThreads) gated_step_kernel(const GatedLinear
         }
         __syncthreads();
         // ---- the recurrence
-        float fq = a.q_scale, fk = 1.0f;
-        if (a.unit_eps > 0.0f) {
-            fq *= 1.0f / sqrtf(dots[0] + a.unit_eps);
-            fk = 1.0f / sqrtf(dots[1] + a.unit_eps);
-        }
-        const float qk = dots[2] * fq * fk, beta = dots[3];
-        float sums[8] = {};  // of the decayed state: S^T k, S^T q
+        float sums[16] = {};  // of the decayed state: S^T k, S^T q; then q.q, k.k, q.k
 #pragma unroll
         for (int r = 0; r < RP; ++r) {
             const int i = lane + r * 32;
             if (i < a.dk) {
-                const float g = sg[i], k = sk[i] * fk, q = sq[i] * fq;
+                const float g = sg[i], k = sk[i], q = sq[i];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     s[r][e] *= g;
                     sums[e] = fmaf(k, s[r][e], sums[e]);
                     sums[4 + e] = fmaf(q, s[r][e], sums[4 + e]);
                 }
+                sums[8] = fmaf(q, q, sums[8]);
+                sums[9] = fmaf(k, k, sums[9]);
+                sums[10] = fmaf(q, k, sums[10]);
             }
         }
-        // fold eight sums over 32 lanes: lanes keep one half of them in each step; lanes 4 j .. 4 j + 3 end up with sum j
+        // fold the sums over 32 lanes: lanes keep one half of them in each step; lanes 2 j and 2 j + 1 end up with sum j
 #pragma unroll
-        for (int n = 4, off = 16; n >= 1; n >>= 1, off >>= 1) {
+        for (int n = 8, off = 16; n >= 1; n >>= 1, off >>= 1) {
             const bool high = (lane & off) != 0;
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+            for (int i = 0; i < 8; ++i)
                 if (i < n) {
                     const float keep = high ? sums[i + n] : sums[i], give = high ? sums[i] : sums[i + n];
                     sums[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
                 }
         }
-        float all = sums[0];
-        all += __shfl_xor_sync(0xffffffffu, all, 2);
-        all += __shfl_xor_sync(0xffffffffu, all, 1);
+        const float all = sums[0] + __shfl_xor_sync(0xffffffffu, sums[0], 1);
+        float fq = a.q_scale, fk = 1.0f;
+        if (a.unit_eps > 0.0f) {
+            fq *= 1.0f / sqrtf(__shfl_sync(0xffffffffu, all, 16) + a.unit_eps);
+            fk = 1.0f / sqrtf(__shfl_sync(0xffffffffu, all, 18) + a.unit_eps);
+        }
+        const float qk = __shfl_sync(0xffffffffu, all, 20) * fq * fk;
         float u[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const float kv = __shfl_sync(0xffffffffu, all, e * 4);
-            u[e] = a.delta ? beta * (sv[lc + e] - kv) : sv[lc + e];
+            const float kv = __shfl_sync(0xffffffffu, all, e * 2);
+            u[e] = a.delta ? beta * (sv[lc + e] - fk * kv) : sv[lc + e];
         }
-        const float qs = __shfl_sync(0xffffffffu, all, 16 + (lane & 3) * 4);
+        const float qs = __shfl_sync(0xffffffffu, all, 8 + (lane & 3) * 2);
         if (lane < 4 && c0 + lane < a.dv)  // S^T q with the token's own write
-            a.out[(size_t)t * a.ldo + (size_t)h * a.dv + c0 + lane] = qs + qk * (lane == 0 ? u[0] : lane == 1 ? u[1] : lane == 2 ? u[2] : u[3]);
+            a.out[(size_t)t * a.ldo + (size_t)h * a.dv + c0 + lane] = fq * qs + qk * (lane == 0 ? u[0] : lane == 1 ? u[1] : lane == 2 ? u[2] : u[3]);
 #pragma unroll
         for (int r = 0; r < RP; ++r) {
             const int i = lane + r * 32;
@@ -1027,6 +1040,7 @@ int run_chunked(cudaStream_t stream, const ChunkArgs& ca) {
 int gated_linear_steps(cudaStream_t stream, const GatedLinearArgs& a) {
     if (a.dk > 512) return fail(KMLL_ERR_UNSUPPORTED, "gated linear attention: key size %d above 512", a.dk);
     if (a.taps > kMaxConvTaps) return fail(KMLL_ERR_UNSUPPORTED, "gated linear attention: %d taps", a.taps);
+    if ((a.ldu & 7) != 0 || (a.gate_rank > 0 && (a.ldg & 7) != 0)) return fail(KMLL_ERR_SHAPE, "gated linear attention: pitches %d, %d are no multiples of 8", a.ldu, a.ldg);
     return a.in_f32 ? run_steps<true>(stream, a) : run_steps<false>(stream, a);
 }
 

@@ -19,7 +19,6 @@ template <bool F32>
 __device__ inline float val(const void* p, size_t i) {
     return F32 ? static_cast<const float*>(p)[i] : bf16_bits_to_f32(static_cast<const uint16_t*>(p)[i]);
 }
-__host__ __device__ inline int round_to(int v, int m) { return (v + m - 1) / m * m; }
 // first position that position `pos` sees
 __device__ inline int first_seen(int pos, int window, int chunk) {
     int lo = 0;
@@ -87,33 +86,22 @@ __global__ void __launch_bounds__(kPlainWarps * 32) grouped_plain_kernel(const G
 }
 
 // ---- decode form ------------------------------------------------------------------------------------------------------------------
-constexpr int kDT = 160;     // positions per tile
-constexpr int kDRows = 16;   // query heads per block = MMA rows
-constexpr int kDWarps = 8;
-constexpr int kDMaxSplit = 16;
-constexpr int kDMinPart = 32;  // positions per split at least
-struct GroupedPlan { int tiles_per_group, tiles, kw, vw; };
-__host__ __device__ inline GroupedPlan decode_plan(int heads, int kv_heads, int dim, int vdim) {
-    GroupedPlan p;
-    p.tiles_per_group = (heads / kv_heads + kDRows - 1) / kDRows;
-    p.tiles = kv_heads * p.tiles_per_group;
-    p.kw = round_to(dim, 32);
-    p.vw = round_to(vdim, 16);
-    return p;
-}
-size_t decode_smem(const GroupedPlan& p) {
-    return ((size_t)(kDT + 2 * kDRows) * (p.kw + 8) + (size_t)kDT * (p.vw + 8) + 2 * (size_t)kDRows * (kDT + 8)) * 2 +
-           ((size_t)kDRows * kDT + kDRows + (size_t)kDRows * kDMaxSplit) * 4;
+// One cluster of eight blocks per (key / value head, 16 query heads).  The positions are cut into steps of 16, dealt out to the
+// warps of all blocks; a warp keeps its own running softmax and weighted values, so nothing but the query is shared until the
+// warps, and then the blocks, merge their parts.
+constexpr int kDRows = 16;     // query heads per block = MMA rows
+constexpr int kDStep = 16;     // positions per step of a warp
+constexpr int kDCluster = 8;
+inline int decode_tiles(const GroupedArgs& a) { return a.kv_heads * ((a.heads / a.kv_heads + kDRows - 1) / kDRows); }
+__host__ __device__ constexpr int decode_warps(int KW, int VW) { return KW + VW > 256 ? 8 : 16; }
+__host__ __device__ constexpr size_t decode_smem(int KW, int VW) {
+    const int NW = decode_warps(KW, VW), steps = NW * kDStep * (KW + VW + 16) * 2, parts = NW * kDRows * VW * 4;
+    return (size_t)2 * kDRows * (KW + 8) * 2 + (steps > parts ? steps : parts) + (size_t)kDRows * VW * 4;
 }
 
 __device__ inline uint32_t cluster_rank() {
     uint32_t r;
     asm("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-    return r;
-}
-__device__ inline uint32_t cluster_size() {
-    uint32_t r;
-    asm("mov.u32 %0, %%cluster_nctaid.x;" : "=r"(r));
     return r;
 }
 __device__ inline void cluster_sync() {
@@ -129,189 +117,205 @@ __device__ inline float cluster_load(const float* p, uint32_t rank) {
     return v;
 }
 
-// One cluster per (key / value head, 16 query heads); its blocks share the positions.
-__global__ void __launch_bounds__(kDWarps * 32) grouped_decode_kernel(const GroupedArgs a, const GroupedPlan pl) {
+template <int KW, int VW>
+__global__ void __launch_bounds__(decode_warps(KW, VW) * 32) grouped_decode_kernel(const GroupedArgs a) {
+    constexpr int NW = decode_warps(KW, VW), KP = KW + 8, VP = VW + 8;
     extern __shared__ __align__(16) uint16_t dsm[];
-    const int KP = pl.kw + 8, VP = pl.vw + 8;
-    uint16_t* const kt = dsm;                    // [kDT][KP]
-    uint16_t* const vt = kt + kDT * KP;          // [kDT][VP]
-    uint16_t* const qh = vt + kDT * VP;          // [16][KP]
+    uint16_t* const qh = dsm;                    // [16][KP]
     uint16_t* const ql = qh + kDRows * KP;
-    uint16_t* const ph = ql + kDRows * KP;       // [16][kDT + 8]
-    uint16_t* const plo = ph + kDRows * (kDT + 8);
-    float* const sc = reinterpret_cast<float*>(plo + kDRows * (kDT + 8));  // [16][kDT]
-    float* const corr = sc + kDRows * kDT;       // [16]
-    float* const f = corr + kDRows;              // [16][kDMaxSplit]
-    __shared__ float stat[2 * kDRows];           // maximum and sum of this block's part, per row
+    uint16_t* const steps = ql + kDRows * KP;    // per warp: keys [16][KP], values [16][VP]; later the warps' parts [NW][16][VW] f32
+    float* const res = reinterpret_cast<float*>(reinterpret_cast<unsigned char*>(dsm) + decode_smem(KW, VW)) - kDRows * VW;  // [16][VW]
+    __shared__ float warp_max_[NW][kDRows], warp_sum_[NW][kDRows], stat[2 * kDRows], f[kDRows * kDCluster];
+    __shared__ uint16_t newest[KW + VW];  // key and value of the newest position
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
-    const int split = (int)cluster_rank(), nsplit = (int)cluster_size(), grp = blockIdx.y / pl.tiles_per_group, sub = blockIdx.y % pl.tiles_per_group;
-    const int per = a.heads / a.kv_heads, h0 = grp * per + sub * kDRows, nh = min(kDRows, per - sub * kDRows);
+    const int per = a.heads / a.kv_heads, tiles = (per + kDRows - 1) / kDRows;
+    const int split = (int)cluster_rank(), grp = blockIdx.y / tiles, sub = blockIdx.y % tiles;
+    const int h0 = grp * per + sub * kDRows, nh = min(kDRows, per - sub * kDRows);
     // the position was written more than one launch ago, and so was every cache row but the newest
-    const int pos = a.at->position, lo = first_seen(pos, a.window, a.chunk), count = pos - lo + 1;
-    const int part_len = max((count + nsplit - 1) / nsplit, kDMinPart), active = (count + part_len - 1) / part_len;
-    const int begin = lo + split * part_len, end = split < active ? min(begin + part_len, pos + 1) : begin;
+    const int pos = a.at->position, lo = first_seen(pos, a.window, a.chunk), n_steps = (pos - lo + kDStep) / kDStep;
     uint16_t* const cache = static_cast<uint16_t*>(a.cache);
     const size_t k0 = (size_t)grp * a.dimp, v0 = (size_t)a.kv_heads * a.dimp + (size_t)grp * a.vdimp;
-    auto load_tile = [&](int t0) {  // rows behind the last position are zeros; the newest one comes from the projection
-        const int rows = min(kDT, round_to(end - t0, 16)), rk = pl.kw / 8, runs = rk + pl.vw / 8;
-        for (int r = warp; r < rows; r += kDWarps) {
-            const int p = t0 + r;
+    uint16_t* const kt = steps + warp * kDStep * (KP + VP);
+    uint16_t* const vt = kt + kDStep * KP;
+    auto load_step = [&](int st) {  // rows behind the last position are zeros; the newest one comes from the projection
+        constexpr int RK = KW / 8, RUNS = RK + VW / 8;
+        const int p0 = lo + st * kDStep;
+#pragma unroll
+        for (int i0 = 0; i0 < kDStep * RUNS; i0 += 32) {
+            const int i = i0 + lane, r = i / RUNS, c = i % RUNS, p = p0 + r;
+            const bool is_k = c < RK;
+            const int col = (is_k ? c : c - RK) * 8;
             if (p == pos) continue;
-            const uint16_t* src = cache + (size_t)min(p, pos) * a.pitch;
-            for (int c = lane; c < runs; c += 32) {
-                const bool is_k = c < rk;
-                const int col = (is_k ? c : c - rk) * 8;
-                const bool live = p < end && col < (is_k ? a.dimp : a.vdimp);
-                const uint32_t dst = (uint32_t)__cvta_generic_to_shared(is_k ? kt + r * KP + col : vt + r * VP + col);
-                cp_async16_zfill_to(dst, live ? src + (is_k ? k0 : v0) + col : cache, live ? 16u : 0u);
-            }
+            const bool live = p < pos && col < (is_k ? a.dimp : a.vdimp);
+            const uint32_t dst = (uint32_t)__cvta_generic_to_shared(is_k ? kt + r * KP + col : vt + r * VP + col);
+            cp_async16_zfill_to(dst, live ? cache + (size_t)p * a.pitch + (is_k ? k0 : v0) + col : cache, live ? 16u : 0u);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    if (begin < end) load_tile(begin);
+    int st = split + warp * kDCluster;
+    if (st < n_steps) load_step(st);
     pdl_wait();
     const float* in = static_cast<const float*>(a.in);
-    auto put_newest = [&](int t0) {
-        if (pos < t0 || pos >= min(t0 + kDT, end)) return;
-        const int r = pos - t0;
-        for (int i = tid; i < pl.kw + pl.vw; i += kDWarps * 32) {
-            const bool is_k = i < pl.kw;
-            const int c = is_k ? i : i - pl.kw;
-            const bool live = c < (is_k ? a.dim : a.vdim);
-            const uint16_t v = live ? f32_to_bf16_bits(in[is_k ? a.k_off + grp * a.dim + c : a.v_off + grp * a.vdim + c]) : (uint16_t)0;
-            if (is_k) kt[r * KP + c] = v;
-            else vt[r * VP + c] = v;
-            if (live && sub == 0 && pos < a.max_seq) cache[(size_t)pos * a.pitch + (is_k ? k0 : v0) + c] = v;
-        }
-    };
-    for (int i = tid; i < kDRows * pl.kw; i += kDWarps * 32) {  // queries (times the score factor), head and remainder
-        const int r = i / pl.kw, c = i - r * pl.kw;
+    for (int i = tid; i < kDRows * KW; i += NW * 32) {  // queries (times the score factor), head and remainder
+        const int r = i / KW, c = i % KW;
         const float v = r < nh && c < a.dim ? in[a.q_off + (size_t)(h0 + r) * a.dim + c] * a.scale : 0.0f;
         const uint16_t hi = f32_to_bf16_bits(v);
         qh[r * KP + c] = hi;
         ql[r * KP + c] = f32_to_bf16_bits(v - bf16_bits_to_f32(hi));
     }
-    constexpr int NG = 2;  // groups of 16 value columns per warp (vdim <= 256)
-    float o[NG][2][4];
-#pragma unroll
-    for (int i = 0; i < NG; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) o[i][j][e] = 0.0f;
-    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};  // of rows `warp` and `warp + 8`
-    for (int t0 = begin; t0 < end; t0 += kDT) {
-        if (t0 > begin) load_tile(t0);
-        put_newest(t0);
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();
-        const int live = min(kDT, end - t0);
-        for (int pb = warp * 8; pb < live; pb += kDWarps * 8) {  // scores: eight positions per warp and round
-            float s4[4][4] = {};
-#pragma unroll 2
-            for (int k = 0; k < pl.kw; k += 32) {
-                uint32_t b[4], ah[4], al[4];
-                ldmatrix_x4(b, kt + (size_t)(pb + (lane & 7)) * KP + k + (lane >> 3) * 8);
-#pragma unroll
-                for (int kk = 0; kk < 2; ++kk) {
-                    const size_t ao = (size_t)(lane & 15) * KP + k + kk * 16 + (lane >> 4) * 8;
-                    ldmatrix_x4(ah, qh + ao);
-                    ldmatrix_x4(al, ql + ao);
-                    mma_bf16(s4[2 * kk], ah, b[2 * kk], b[2 * kk + 1]);
-                    mma_bf16(s4[2 * kk + 1], al, b[2 * kk], b[2 * kk + 1]);
-                }
-            }
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-                sc[(g + (e >> 1) * 8) * kDT + pb + 2 * tq + (e & 1)] = (s4[0][e] + s4[1][e]) + (s4[2][e] + s4[3][e]);
+    if ((n_steps - 1) % kDCluster == split)  // (the block that reads the newest position)
+        for (int i = tid; i < KW + VW; i += NW * 32) {
+            const bool is_k = i < KW;
+            const int c = is_k ? i : i - KW;
+            const bool live = c < (is_k ? a.dim : a.vdim);
+            const uint16_t v = live ? f32_to_bf16_bits(in[is_k ? a.k_off + grp * a.dim + c : a.v_off + grp * a.vdim + c]) : (uint16_t)0;
+            newest[i] = v;
+            if (live && sub == 0 && pos < a.max_seq) cache[(size_t)pos * a.pitch + (is_k ? k0 : v0) + c] = v;
         }
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {  // softmax: warp w, rows w and w + 8
-            const int r = warp + i * 8;
-            float v[kDT / 32], mx = m_run[i], sum = 0.0f;
-#pragma unroll
-            for (int j = 0; j < kDT / 32; ++j) {
-                v[j] = lane + 32 * j < live ? sc[r * kDT + lane + 32 * j] : -INFINITY;
-                mx = fmaxf(mx, v[j]);
-            }
-            mx = warp_max(mx);  // (position t0 is always live, so it is finite)
-            const float cf = expf(m_run[i] - mx);
-#pragma unroll
-            for (int j = 0; j < kDT / 32; ++j) {
-                const float w = expf(v[j] - mx);
-                sum += w;
-                const uint16_t hi = f32_to_bf16_bits(w);
-                ph[r * (kDT + 8) + lane + 32 * j] = hi;
-                plo[r * (kDT + 8) + lane + 32 * j] = f32_to_bf16_bits(w - bf16_bits_to_f32(hi));
-            }
-            m_run[i] = mx;
-            l_run[i] = l_run[i] * cf + warp_sum(sum);
-            if (lane == 0) corr[r] = cf;
-        }
-        __syncthreads();
-        const float ca = corr[g], cb = corr[g + 8];
-#pragma unroll
-        for (int i = 0; i < NG; ++i)
-#pragma unroll
-            for (int j = 0; j < 2; ++j) { o[i][j][0] *= ca; o[i][j][1] *= ca; o[i][j][2] *= cb; o[i][j][3] *= cb; }
-#pragma unroll
-        for (int j = 0; j < kDT / 16; ++j) {
-            if (j * 16 >= live) break;
-            uint32_t ah[4], al[4], b[4];
-            const int ao = (lane & 15) * (kDT + 8) + j * 16 + (lane >> 4) * 8;
-            ldmatrix_x4(ah, ph + ao);
-            ldmatrix_x4(al, plo + ao);
-#pragma unroll
-            for (int i = 0; i < NG; ++i) {
-                const int c = (warp + i * kDWarps) * 16;
-                if (c >= pl.vw) break;
-                ldmatrix_x4_trans(b, vt + (size_t)(j * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * VP + c + (lane >> 4) * 8);
-                mma_bf16(o[i][0], ah, b[0], b[1]);
-                mma_bf16(o[i][1], ah, b[2], b[3]);
-                mma_bf16(o[i][0], al, b[0], b[1]);
-                mma_bf16(o[i][1], al, b[2], b[3]);
-            }
-        }
-        __syncthreads();
-    }
-    // ---- the blocks' parts: (weighted values, maximum, sum) in shared memory, merged slice by slice
-    float* const part = reinterpret_cast<float*>(dsm);  // [16][vw], in the place of the key tile
-    if (lane == 0) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            stat[warp + i * 8] = m_run[i];
-            stat[kDRows + warp + i * 8] = l_run[i];
-        }
-    }
-#pragma unroll
-    for (int i = 0; i < NG; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; e += 2) {
-                const int c = (warp + i * kDWarps) * 16 + j * 8 + 2 * tq;
-                if (c < pl.vw) *reinterpret_cast<float2*>(part + (g + (e >> 1) * 8) * pl.vw + c) = make_float2(o[i][j][e], o[i][j][e + 1]);
-            }
-    cluster_sync();
-    for (int r = warp; r < nh; r += kDWarps) {
-        const bool on = lane < active;
-        const float m = on ? cluster_load(stat + r, lane) : -INFINITY, l = on ? cluster_load(stat + kDRows + r, lane) : 0.0f;
-        const float mx = warp_max(m), w = on ? expf(m - mx) : 0.0f, sum = warp_sum(w * l);
-        if (lane < kDMaxSplit) f[r * kDMaxSplit + lane] = w / sum;
-    }
     __syncthreads();
-    const int outs = nh * a.vdim, slice = (outs + nsplit - 1) / nsplit;
-    for (int i = split * slice + tid; i < min((split + 1) * slice, outs); i += kDWarps * 32) {
+    float o[VW / 8][4];
+#pragma unroll
+    for (int i = 0; i < VW / 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};  // of rows g and g + 8
+    for (; st < n_steps; st += kDCluster * NW) {
+        const int p0 = lo + st * kDStep;
+        if (pos < p0 + kDStep)  // the newest position is the last of the last step
+            for (int i = lane; i < KW + VW; i += 32) (i < KW ? kt + (pos - p0) * KP : vt + (pos - p0) * VP - KW)[i] = newest[i];
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncwarp();
+        float s[2][4] = {}, s2[2][4] = {};  // scores: heads, remainders of the query
+#pragma unroll
+        for (int k = 0; k < KW / 16; ++k) {
+            uint32_t b[4], ah[4], al[4];
+            ldmatrix_x4(b, kt + ((lane >> 4) * 8 + (lane & 7)) * KP + k * 16 + ((lane >> 3) & 1) * 8);
+            ldmatrix_x4(ah, qh + (lane & 15) * KP + k * 16 + (lane >> 4) * 8);
+            ldmatrix_x4(al, ql + (lane & 15) * KP + k * 16 + (lane >> 4) * 8);
+            mma_bf16(s[0], ah, b[0], b[1]);
+            mma_bf16(s[1], ah, b[2], b[3]);
+            mma_bf16(s2[0], al, b[0], b[1]);
+            mma_bf16(s2[1], al, b[2], b[3]);
+        }
+        float mx[2] = {m_run[0], m_run[1]};
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                s[i][e] = p0 + i * 8 + 2 * tq + (e & 1) <= pos ? s[i][e] + s2[i][e] : -INFINITY;
+                mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
+            }
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+            mx[y] = fmaxf(mx[y], __shfl_xor_sync(0xffffffffu, mx[y], 1));
+            mx[y] = fmaxf(mx[y], __shfl_xor_sync(0xffffffffu, mx[y], 2));  // (the step's first position is always seen, so it is finite)
+        }
+        const float ca = expf(m_run[0] - mx[0]), cb = expf(m_run[1] - mx[1]);
+        float sum[2] = {0.0f, 0.0f};
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                s[i][e] = expf(s[i][e] - mx[e >> 1]);
+                sum[e >> 1] += s[i][e];
+            }
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+            sum[y] += __shfl_xor_sync(0xffffffffu, sum[y], 1);
+            sum[y] += __shfl_xor_sync(0xffffffffu, sum[y], 2);
+            m_run[y] = mx[y];
+        }
+        l_run[0] = l_run[0] * ca + sum[0];
+        l_run[1] = l_run[1] * cb + sum[1];
+        uint32_t ph[4], pl[4];
+        split_bf16x2(s[0][0], s[0][1], ph[0], pl[0]);
+        split_bf16x2(s[0][2], s[0][3], ph[1], pl[1]);
+        split_bf16x2(s[1][0], s[1][1], ph[2], pl[2]);
+        split_bf16x2(s[1][2], s[1][3], ph[3], pl[3]);
+#pragma unroll
+        for (int d2 = 0; d2 < VW / 16; ++d2) {
+            uint32_t b[4];
+            ldmatrix_x4_trans(b, vt + (((lane >> 3) & 1) * 8 + (lane & 7)) * VP + d2 * 16 + (lane >> 4) * 8);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                float (&c)[4] = o[2 * d2 + i];
+                c[0] *= ca; c[1] *= ca; c[2] *= cb; c[3] *= cb;
+                mma_bf16(c, ph, b[2 * i], b[2 * i + 1]);
+                mma_bf16(c, pl, b[2 * i], b[2 * i + 1]);
+            }
+        }
+        __syncwarp();
+        if (st + kDCluster * NW < n_steps) load_step(st + kDCluster * NW);
+    }
+    // ---- the warps' parts -> this block's (weighted values, maximum, sum)
+    if (tq == 0) {
+        warp_max_[warp][g] = m_run[0];
+        warp_max_[warp][g + 8] = m_run[1];
+        warp_sum_[warp][g] = l_run[0];
+        warp_sum_[warp][g + 8] = l_run[1];
+    }
+    __syncthreads();  // every step has been read
+    float* const parts = reinterpret_cast<float*>(steps);
+#pragma unroll
+    for (int i = 0; i < VW / 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+            const int r = g + (e >> 1) * 8;
+            if (r < nh) *reinterpret_cast<float2*>(parts + (warp * kDRows + r) * VW + i * 8 + 2 * tq) = make_float2(o[i][e], o[i][e + 1]);
+        }
+    if (warp < kDRows && lane < NW)
+        for (int r = warp; r < nh; r += NW) {  // lane w: warp w's factor of row r
+            const float m = warp_max_[lane][r];
+            float mx = m;
+#pragma unroll
+            for (int off = NW / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync((1u << (NW - 1)) * 2u - 1u, mx, off));
+            const float w = m == -INFINITY ? 0.0f : expf(m - mx);
+            float l = w * warp_sum_[lane][r];
+#pragma unroll
+            for (int off = NW / 2; off > 0; off >>= 1) l += __shfl_xor_sync((1u << (NW - 1)) * 2u - 1u, l, off);
+            warp_sum_[lane][r] = w;  // (read above by this lane only)
+            if (lane == 0) { stat[r] = mx; stat[kDRows + r] = l; }
+        }
+    __syncthreads();
+    for (int i = tid; i < nh * VW; i += NW * 32) {
+        const int r = i / VW, c = i % VW;
+        float v = 0.0f;
+#pragma unroll
+        for (int w = 0; w < NW; ++w) v = fmaf(warp_sum_[w][r], parts[(w * kDRows + r) * VW + c], v);
+        res[i] = v;
+    }
+    cluster_sync();
+    // ---- the blocks' parts, a slice of the outputs each
+    for (int i = tid; i < nh * kDCluster; i += NW * 32) f[i] = cluster_load(stat + i / kDCluster, i % kDCluster);
+    const int outs = nh * a.vdim, slice = (outs + kDCluster - 1) / kDCluster;
+    __syncthreads();
+    for (int i = split * slice + tid; i < min((split + 1) * slice, outs); i += NW * 32) {
         const int r = i / a.vdim, c = i - r * a.vdim;
-        float x[kDMaxSplit], v = 0.0f;
+        float x[kDCluster], l[kDCluster], mx = -INFINITY, v = 0.0f, total = 0.0f;
 #pragma unroll
-        for (int s = 0; s < kDMaxSplit; ++s) x[s] = s < active ? cluster_load(part + r * pl.vw + c, s) : 0.0f;
+        for (int s = 0; s < kDCluster; ++s) {
+            x[s] = cluster_load(res + r * VW + c, s);
+            l[s] = cluster_load(stat + kDRows + r, s);
+            mx = fmaxf(mx, f[r * kDCluster + s]);
+        }
 #pragma unroll
-        for (int s = 0; s < kDMaxSplit; ++s) v = fmaf(s < active ? f[r * kDMaxSplit + s] : 0.0f, x[s], v);
-        a.out[(size_t)(h0 + r) * a.vdim + c] = v;
+        for (int s = 0; s < kDCluster; ++s) {
+            const float m = f[r * kDCluster + s], w = m == -INFINITY ? 0.0f : expf(m - mx);
+            v = fmaf(w, x[s], v);
+            total = fmaf(w, l[s], total);
+        }
+        a.out[(size_t)(h0 + r) * a.vdim + c] = v / total;
     }
     cluster_sync();  // (no block leaves while another reads its part)
+}
+
+template <int KW, int VW>
+int run_decode(cudaStream_t stream, const GroupedArgs& a) {
+    cudaError_t e = allow_all_dynamic_smem(grouped_decode_kernel<KW, VW>);
+    if (e == cudaSuccess)
+        e = launch_cluster(grouped_decode_kernel<KW, VW>, dim3(kDCluster, decode_tiles(a)), kDCluster, dim3(decode_warps(KW, VW) * 32), decode_smem(KW, VW), stream, true, a);
+    if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "grouped attention (decode): %s", cudaGetErrorString(e));
+    return KMLL_OK;
 }
 
 // ---- prompt form --------------------------------------------------------------------------------------------------------------------
@@ -502,44 +506,13 @@ int grouped_attention_plain(cudaStream_t stream, const GroupedArgs& a) {
 }
 
 bool grouped_decode_ok(const GroupedArgs& a) {
-    const GroupedPlan p = decode_plan(a.heads, a.kv_heads, a.dim, a.vdim);
-    return a.T == 1 && !a.cache_f32 && a.in_f32 && a.at != nullptr && a.vdim <= 16 * 2 * kDWarps && p.tiles <= 65535 && decode_smem(p) <= 220 * 1024;
-}
-// Blocks per cluster: 16 where all clusters are resident at once with it, else the portable 8.
-static int decode_cluster(const GroupedPlan& p, size_t smem, int* out) {
-    *out = 8;
-    if (p.tiles * 16 > 148) return KMLL_OK;
-    cudaError_t e = cudaFuncSetAttribute(grouped_decode_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-    if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "grouped attention (decode): %s", cudaGetErrorString(e));
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(16, p.tiles);
-    cfg.blockDim = dim3(kDWarps * 32);
-    cfg.dynamicSmemBytes = smem;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeClusterDimension;
-    attr[0].val.clusterDim.x = 16;
-    attr[0].val.clusterDim.y = 1;
-    attr[0].val.clusterDim.z = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = 1;
-    int clusters = 0;
-    if (cudaOccupancyMaxActiveClusters(&clusters, grouped_decode_kernel, &cfg) != cudaSuccess) {
-        cudaGetLastError();  // (a device that has no such clusters)
-        clusters = 0;
-    }
-    if (clusters >= p.tiles) *out = 16;
-    return KMLL_OK;
+    return a.T == 1 && !a.cache_f32 && a.in_f32 && a.at != nullptr && a.dim <= 256 && a.vdim <= 256 && decode_tiles(a) <= 65535;
 }
 int grouped_attention_decode(cudaStream_t stream, const GroupedArgs& a) {
     if (!grouped_decode_ok(a)) return fail(KMLL_ERR_UNSUPPORTED, "grouped attention: no decode form for %d / %d heads of %d, %d", a.heads, a.kv_heads, a.dim, a.vdim);
-    const GroupedPlan p = decode_plan(a.heads, a.kv_heads, a.dim, a.vdim);
-    const size_t smem = decode_smem(p);
-    cudaError_t e = allow_all_dynamic_smem(grouped_decode_kernel);
-    int cluster = 8;
-    if (e == cudaSuccess) KMLL_TRY_RC(decode_cluster(p, smem, &cluster));
-    if (e == cudaSuccess) e = launch_cluster(grouped_decode_kernel, dim3(cluster, p.tiles), cluster, dim3(kDWarps * 32), smem, stream, true, a, p);
-    if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "grouped attention (decode): %s", cudaGetErrorString(e));
-    return KMLL_OK;
+    if (a.dim <= 64) return a.vdim <= 64 ? run_decode<64, 64>(stream, a) : a.vdim <= 128 ? run_decode<64, 128>(stream, a) : run_decode<64, 256>(stream, a);
+    if (a.dim <= 128) return a.vdim <= 64 ? run_decode<128, 64>(stream, a) : a.vdim <= 128 ? run_decode<128, 128>(stream, a) : run_decode<128, 256>(stream, a);
+    return a.vdim <= 64 ? run_decode<256, 64>(stream, a) : a.vdim <= 128 ? run_decode<256, 128>(stream, a) : run_decode<256, 256>(stream, a);
 }
 
 bool grouped_prefill_ok(const GroupedArgs& a) { return !a.in_f32 && !a.cache_f32 && a.dim <= 256 && a.vdim <= 128; }

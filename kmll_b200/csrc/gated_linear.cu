@@ -356,7 +356,7 @@ int run_steps(cudaStream_t stream, const GatedLinearArgs& a) {
 }
 
 // ---- chunked form -----------------------------------------------------------------------------------------------------------------
-constexpr int kGC = 64, kGThreads = 256, kAP = kGC + 4;  // tokens per chunk; pitch of the token-by-token matrices in f32
+constexpr int kGC = 64, kGThreads = 256, kAP = kGC + 8;  // tokens per chunk; pitch of token-by-token matrices
 
 // What the preparing launch leaves per (chunk, head): bf16 head / remainder planes [64][DK] of q 2^G, k 2^(G_n - G) and (delta) W,
 // [64][64] of A, then 2^G_n [DK] in f32.
@@ -380,8 +380,16 @@ struct ChunkArgs {
 };
 inline int padded_keys(int dk) { return dk <= 64 ? 64 : 128; }
 
-// f32 pairs in shared memory -> operand registers (head, remainder)
-__device__ inline void split_pair(const float2 v, uint32_t& hi, uint32_t& lo) { split_bf16x2(v.x, v.y, hi, lo); }
+// SiLU and log2 of the decay from the hardware's 2^x and log2 (a few ulp)
+__device__ inline float fast_silu(float z) { return __fdividef(z, 1.0f + ex2_approx(-z * kLog2e)); }
+__device__ inline float fast_softplus(float z) {
+    const float t = ex2_approx(-fabsf(z) * kLog2e);
+    return fmaxf(z, 0.0f) + (t < 0.015625f ? t * (1.0f - t * (0.5f - t * (1.0f / 3.0f))) : __logf(1.0f + t));
+}
+__device__ inline float fast_log2_decay(const GatedLinearArgs& a, float z, float rate) {
+    const float l = a.decay == KMLL_DECAY_LOGISTIC ? -fast_softplus(-z) * a.inv_tau : -rate * fast_softplus(z);
+    return fmaxf(l * kLog2e, -150.0f);
+}
 // c += (ah + al) (bh + bl) without the product of the remainders
 __device__ inline void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
     mma_bf16(c, ah, bh0, bh1);
@@ -434,20 +442,49 @@ __device__ inline void stage_rows(const GatedLinearArgs& a, uint16_t* tile, int 
         }
     }
 }
-// channels d, d + 1 of token t from a staged tile, through convolution and SiLU; w0, w1: their taps (null: none)
-template <int DK>
-__device__ inline float2 staged_pair(const GatedLinearArgs& a, const uint16_t* tile, int t, int d, const uint16_t* w0, const uint16_t* w1) {
+__device__ inline float2 unpack2(uint32_t x) { return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u)); }
+// channels d, d + 1 of tokens t .. t + ROWS - 1 from a staged tile, through convolution and SiLU; ch: ring channel of d; odd:
+// channel d + 1 does not exist
+template <int DK, int ROWS>
+__device__ inline void staged_rows(const GatedLinearArgs& a, const uint16_t* tile, int t, int d, int ch, bool odd, float2 (&y)[ROWS]) {
+    auto at = [&](int r) { return unpack2(*reinterpret_cast<const uint32_t*>(tile + r * DK + d)); };
     if (a.taps == 0) {
-        const uint32_t x = *reinterpret_cast<const uint32_t*>(tile + t * DK + d);
-        return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u));
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) y[i] = at(t + i);
+        return;
     }
-    float2 y = make_float2(0.0f, 0.0f);
-    for (int j = 0; j < a.taps; ++j) {
-        const uint32_t x = *reinterpret_cast<const uint32_t*>(tile + (t + j) * DK + d);
-        y.x = fmaf(bf16_bits_to_f32(w0[j]), __uint_as_float(x << 16), y.x);
-        y.y = fmaf(bf16_bits_to_f32(w1[j]), __uint_as_float(x & 0xffff0000u), y.y);
+    const uint16_t* w0 = a.conv + (size_t)ch * a.taps;
+    const uint16_t* w1 = odd ? w0 : w0 + a.taps;
+    if (a.taps <= 4) {
+        const int lead = 4 - a.taps;  // missing taps
+        float2 w[4], x[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            w[j] = j >= lead ? make_float2(bf16_bits_to_f32(w0[j - lead]), bf16_bits_to_f32(w1[j - lead])) : make_float2(0.0f, 0.0f);
+            x[j] = j >= lead && j < 3 ? at(t + j - lead) : make_float2(0.0f, 0.0f);
+        }
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) {
+            x[3] = at(t + i + 3 - lead);
+            float2 s = __ffma2_rn(w[0], x[0], make_float2(0.0f, 0.0f));
+            s = __ffma2_rn(w[1], x[1], s);
+            s = __ffma2_rn(w[2], x[2], s);
+            y[i] = __ffma2_rn(w[3], x[3], s);
+            x[0] = x[1];
+            x[1] = x[2];
+            x[2] = x[3];
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) y[i] = make_float2(0.0f, 0.0f);
+        for (int j = 0; j < a.taps; ++j) {
+            const float2 w = make_float2(bf16_bits_to_f32(w0[j]), bf16_bits_to_f32(w1[j]));
+#pragma unroll
+            for (int i = 0; i < ROWS; ++i) y[i] = __ffma2_rn(w, at(t + i + j), y[i]);
+        }
     }
-    return make_float2(act_silu(y.x), act_silu(y.y));
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) y[i] = make_float2(fast_silu(y[i].x), fast_silu(y[i].y));
 }
 
 template <int DK, bool DELTA>
@@ -556,26 +593,27 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
 #pragma unroll
             for (int e = 0; e < 4; ++e) {  // tokens behind the last change nothing: decay 1
                 const int t = (mb + m) * 16 + g + (e >> 1) * 8, d = (cb + b) * 8 + 2 * tq + (e & 1);
-                z[b][m][e] = t < n && d < a.dk ? log2_decay(a, z[b][m][e] + (a.bias != nullptr ? bf16_bits_to_f32(a.bias[h * a.dk + d]) : 0.0f), rate) : 0.0f;
+                z[b][m][e] = t < n && d < a.dk ? fast_log2_decay(a, z[b][m][e] + (a.bias != nullptr ? bf16_bits_to_f32(a.bias[h * a.dk + d]) : 0.0f), rate) : 0.0f;
             }
     __syncthreads();  // the decay factor and map have been read
+    constexpr int PAIRS = DK / 2, ROWS = kGC * PAIRS / NT;  // a thread: two channels of ROWS tokens
+    const int pd = (tid % PAIRS) * 2, pt = tid / PAIRS * ROWS;
     // ---- q and k
     {
-        constexpr int PAIRS = DK / 2, STEP = NT / PAIRS;
-        const int d = (tid % PAIRS) * 2;
         const float fq = a.unit_eps > 0.0f ? 1.0f : a.q_scale;
-        const bool live0 = d < a.dk, live1 = d + 1 < a.dk;
-        const uint16_t* wq = a.conv + (size_t)(chq + d) * a.taps;
-        const uint16_t* wk = a.conv + (size_t)(nq + chq + d) * a.taps;
-        for (int t = tid / PAIRS; t < kGC; t += STEP) {
-            float2 q = make_float2(0.0f, 0.0f), k = q;
-            if (live0 && t < n) {
-                q = staged_pair<DK>(a, raw_q, t, d, wq, live1 ? wq + a.taps : wq);
-                k = staged_pair<DK>(a, raw_k, t, d, wk, live1 ? wk + a.taps : wk);
-                if (!live1) q.y = k.y = 0.0f;
-            }
-            *reinterpret_cast<float2*>(Q + t * P + d) = make_float2(q.x * fq, q.y * fq);
-            *reinterpret_cast<float2*>(K + t * P + d) = k;
+        const bool live = pd < a.dk, odd = pd + 1 >= a.dk;
+        float2 q[ROWS], k[ROWS];
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) q[i] = k[i] = make_float2(0.0f, 0.0f);
+        if (live) {
+            staged_rows<DK, ROWS>(a, raw_q, pt, pd, chq + pd, odd, q);
+            staged_rows<DK, ROWS>(a, raw_k, pt, pd, nq + chq + pd, odd, k);
+        }
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) {
+            const bool on = live && pt + i < n;
+            *reinterpret_cast<float2*>(Q + (pt + i) * P + pd) = make_float2(on ? q[i].x * fq : 0.0f, on && !odd ? q[i].y * fq : 0.0f);
+            *reinterpret_cast<float2*>(K + (pt + i) * P + pd) = make_float2(on ? k[i].x : 0.0f, on && !odd ? k[i].y : 0.0f);
         }
     }
     __syncthreads();  // the projected rows have been read
@@ -589,13 +627,19 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
     // ---- unit vectors; running sums of the log decays
     if (a.unit_eps > 0.0f)
         for (int r = warp; r < 2 * kGC; r += NW) {
-            float* x = (r < kGC ? Q : K) + (r & (kGC - 1)) * P;
-            float v[DK / 32], s = 0.0f;
+            constexpr int V = DK / 32;
+            float* x = (r < kGC ? Q : K) + (r & (kGC - 1)) * P + lane * V;
+            float v[V], sq = 0.0f;
 #pragma unroll
-            for (int i = 0; i < DK / 32; ++i) { v[i] = x[lane + i * 32]; s += v[i] * v[i]; }
-            const float f = (r < kGC ? a.q_scale : 1.0f) / sqrtf(warp_sum(s) + a.unit_eps);
+            for (int i = 0; i < V; i += 2) {
+                const float2 t = *reinterpret_cast<const float2*>(x + i);
+                v[i] = t.x;
+                v[i + 1] = t.y;
+                sq += t.x * t.x + t.y * t.y;
+            }
+            const float f = (r < kGC ? a.q_scale : 1.0f) * rsqrtf(warp_sum(sq) + a.unit_eps);
 #pragma unroll
-            for (int i = 0; i < DK / 32; ++i) x[lane + i * 32] = v[i] * f;
+            for (int i = 0; i < V; i += 2) *reinterpret_cast<float2*>(x + i) = make_float2(v[i] * f, v[i + 1] * f);
         }
     __syncthreads();
     {
@@ -674,19 +718,24 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
             if ((i + 1) * (i + 2) / 2 <= r) ++i;
             const int j = B * 16 + r - i * (i + 1) / 2;
             i += B * 16;
-            float sq = 0.0f, sl = 0.0f;
+            float2 sq2 = make_float2(0.0f, 0.0f), sl2 = sq2;
+            const float2 minus = make_float2(-1.0f, -1.0f);
 #pragma unroll 4
             for (int d = 0; d < DK; d += 4) {
                 const float4 gi = *reinterpret_cast<const float4*>(G + i * P + d), gj = *reinterpret_cast<const float4*>(G + j * P + d);
                 const float4 kj = *reinterpret_cast<const float4*>(K + j * P + d), qi = *reinterpret_cast<const float4*>(Q + i * P + d);
-                const float w0 = kj.x * ex2_approx(gi.x - gj.x), w1 = kj.y * ex2_approx(gi.y - gj.y), w2 = kj.z * ex2_approx(gi.z - gj.z),
-                            w3 = kj.w * ex2_approx(gi.w - gj.w);
-                sq += qi.x * w0 + qi.y * w1 + qi.z * w2 + qi.w * w3;
+                float2 e0 = __ffma2_rn(make_float2(gj.x, gj.y), minus, make_float2(gi.x, gi.y)), e1 = __ffma2_rn(make_float2(gj.z, gj.w), minus, make_float2(gi.z, gi.w));
+                e0 = __fmul2_rn(make_float2(kj.x, kj.y), make_float2(ex2_approx(e0.x), ex2_approx(e0.y)));
+                e1 = __fmul2_rn(make_float2(kj.z, kj.w), make_float2(ex2_approx(e1.x), ex2_approx(e1.y)));
+                sq2 = __ffma2_rn(make_float2(qi.x, qi.y), e0, sq2);
+                sq2 = __ffma2_rn(make_float2(qi.z, qi.w), e1, sq2);
                 if (DELTA) {
                     const float4 ki = *reinterpret_cast<const float4*>(K + i * P + d);
-                    sl += ki.x * w0 + ki.y * w1 + ki.z * w2 + ki.w * w3;
+                    sl2 = __ffma2_rn(make_float2(ki.x, ki.y), e0, sl2);
+                    sl2 = __ffma2_rn(make_float2(ki.z, ki.w), e1, sl2);
                 }
             }
+            const float sq = sq2.x + sq2.y, sl = sl2.x + sl2.y;
             const uint16_t hi = f32_to_bf16_bits(sq);
             Ah[i * kGC + j] = hi;
             Al[i * kGC + j] = f32_to_bf16_bits(sq - bf16_bits_to_f32(hi));
@@ -734,81 +783,102 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
             x[i] = (s0 + s1) + (s2 + s3);
         }
         asm volatile("bar.sync 1, 64;" ::: "memory");  // both warps have read L
+        uint16_t* const X = reinterpret_cast<uint16_t*>(L);  // [2][64][kAP]: heads, remainders
 #pragma unroll
-        for (int i = 0; i < kGC; ++i) L[i * kAP + tid] = x[i];
+        for (int i = 0; i < kGC; ++i) {
+            const uint16_t hi = f32_to_bf16_bits(x[i]);
+            X[i * kAP + tid] = hi;
+            X[(kGC + i) * kAP + tid] = f32_to_bf16_bits(x[i] - bf16_bits_to_f32(hi));
+        }
     }
     if (!DELTA) return;
-    __syncthreads();
-    // ---- W = X (beta k 2^G), U0 = X (beta v): right-hand sides in K's place and, DK columns at a time, in Q's
-    for (int i = tid; i < kGC * DK; i += NT) {
-        const int t = i / DK, d = i % DK;
-        K[t * P + d] *= beta[t] * ex2_approx(G[t * P + d]);
+    // ---- W = X (beta k 2^G), U0 = X (beta v): right-hand sides as head / remainder planes [2][64][PB] in the places of q, k and the
+    // decays, DK value columns at a time; a warp takes 16 columns
+    constexpr int PB = DK + 8;
+    uint16_t* const X = reinterpret_cast<uint16_t*>(L);
+    uint16_t* const Rk = reinterpret_cast<uint16_t*>(gsm);
+    uint16_t* const Rv = Rk + 2 * kGC * PB;
+    auto put = [&](uint16_t* R, int t, float x, float y) {
+        uint32_t hi, lo;
+        split_bf16x2(x, y, hi, lo);
+        *reinterpret_cast<uint32_t*>(R + t * PB + pd) = hi;
+        *reinterpret_cast<uint32_t*>(R + (kGC + t) * PB + pd) = lo;
+    };
+    {
+        __syncthreads();
+        float2 k[ROWS];
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) {
+            const int t = pt + i;
+            const float2 kk = *reinterpret_cast<const float2*>(K + t * P + pd), gg = *reinterpret_cast<const float2*>(G + t * P + pd);
+            k[i] = make_float2(beta[t] * kk.x * ex2_approx(gg.x), beta[t] * kk.y * ex2_approx(gg.y));
+        }
+        __syncthreads();  // k and the decays have been read
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) put(Rk, pt + i, k[i].x, k[i].y);
     }
-    const int tiles = (ca.dvp + DK - 1) / DK;
-    for (int tile = -1; tile < tiles; ++tile) {
-        if (tile > 0) {
+    for (int v0 = 0; v0 < ca.dvp; v0 += DK) {
+        if (v0 > 0) {
             __syncthreads();
-            stage_rows<DK, NT>(a, raw_v, t0, n, a.v_off + h * a.dv + tile * DK, chv + tile * DK, a.dv - tile * DK, channels, fast);
+            stage_rows<DK, NT>(a, raw_v, t0, n, a.v_off + h * a.dv + v0, chv + v0, a.dv - v0, channels, fast);
             asm volatile("cp.async.commit_group;" ::: "memory");
         }
-        if (tile >= 0) {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-            __syncthreads();
-            constexpr int PAIRS = DK / 2;
-            const int d = (tid % PAIRS) * 2, col = tile * DK + d;
-            const uint16_t* w = a.conv + (size_t)(chv + col) * a.taps;
-            for (int t = tid / PAIRS; t < kGC; t += NT / PAIRS) {
-                float2 v = make_float2(0.0f, 0.0f);
-                if (t < n && col < a.dv) {
-                    v = staged_pair<DK>(a, raw_v, t, d, w, col + 1 < a.dv ? w + a.taps : w);
-                    v.x *= beta[t];
-                    v.y = col + 1 < a.dv ? v.y * beta[t] : 0.0f;
-                }
-                *reinterpret_cast<float2*>(Q + t * P + d) = v;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        {
+            const int col = v0 + pd;
+            const bool live = col < a.dv, odd = col + 1 >= a.dv;
+            float2 v[ROWS];
+            if (live) staged_rows<DK, ROWS>(a, raw_v, pt, pd, chv + col, odd, v);
+#pragma unroll
+            for (int i = 0; i < ROWS; ++i) {
+                const bool on = live && pt + i < n;
+                put(Rv, pt + i, on ? beta[pt + i] * v[i].x : 0.0f, on && !odd ? beta[pt + i] * v[i].y : 0.0f);
             }
         }
-        const float* R = tile < 0 ? K : Q;
         __syncthreads();
-        constexpr int CB = DK / 8, MG = NW / CB < 1 ? 1 : NW / CB, NBW = CB / (NW / MG);  // warps over column blocks, then over row blocks
-        const int wc = warp % (NW / MG) * NBW, wm = warp / (NW / MG);
-#pragma unroll 1
-        for (int m = wm; m < 4; m += MG) {
-            float acc[NBW][4] = {};
-            for (int ks = 0; ks <= m; ++ks) {  // X is lower triangular
-                uint32_t xh[4], xl[4];
+        constexpr int CG = DK / 16;  // column groups of one right-hand side
+        for (int cg = warp + (v0 > 0 ? CG : 0); cg < 2 * CG; cg += NW) {
+            const bool is_v = cg >= CG;
+            const uint16_t* R = is_v ? Rv : Rk;
+            const int c0 = (is_v ? cg - CG : cg) * 16;
+            if (is_v && v0 + c0 >= ca.dvp) break;
+            uint32_t bh[4][4], bl[4][4];
 #pragma unroll
-                for (int x = 0; x < 2; ++x)
-#pragma unroll
-                    for (int y = 0; y < 2; ++y)
-                        split_pair(*reinterpret_cast<const float2*>(L + (m * 16 + g + y * 8) * kAP + ks * 16 + x * 8 + 2 * tq), xh[x * 2 + y], xl[x * 2 + y]);
-#pragma unroll
-                for (int b = 0; b < NBW; ++b) {
-                    const int d = (wc + b) * 8 + g;
-                    uint32_t bh[2], bl[2];
-#pragma unroll
-                    for (int x = 0; x < 2; ++x) {
-                        const int r = ks * 16 + x * 8 + 2 * tq;
-                        split_bf16x2(R[r * P + d], R[(r + 1) * P + d], bh[x], bl[x]);
-                    }
-                    mma_split(acc[b], xh, xl, bh[0], bh[1], bl[0], bl[1]);
-                }
+            for (int ks = 0; ks < 4; ++ks) {
+                const int bo = (ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * PB + c0 + (lane >> 4) * 8;
+                ldmatrix_x4_trans(bh[ks], R + bo);
+                ldmatrix_x4_trans(bl[ks], R + kGC * PB + bo);
             }
 #pragma unroll
-            for (int b = 0; b < NBW; ++b)
+            for (int m = 0; m < 4; ++m) {
+                float acc[2][4] = {};
 #pragma unroll
-                for (int e = 0; e < 4; e += 2) {
-                    const int t = m * 16 + g + (e >> 1) * 8, d = (wc + b) * 8 + 2 * tq;
-                    if (tile < 0) {
-                        uint32_t hi, lo;
-                        split_bf16x2(acc[b][e], acc[b][e + 1], hi, lo);
-                        uint32_t* p = reinterpret_cast<uint32_t*>(out + 4 * lay.plane) + (t * DK + d) / 2;
-                        p[0] = hi;
-                        p[lay.plane] = lo;
-                    } else if (tile * DK + d < ca.dvp) {
-                        float* p = ca.u0 + (((size_t)c * a.heads + h) * kGC + t) * ca.dvp + tile * DK + d;
-                        *reinterpret_cast<float2*>(p) = make_float2(acc[b][e], acc[b][e + 1]);
-                    }
+                for (int ks = 0; ks <= m; ++ks) {  // X is lower triangular
+                    uint32_t xh[4], xl[4];
+                    const int ao = (m * 16 + (lane & 15)) * kAP + ks * 16 + (lane >> 4) * 8;
+                    ldmatrix_x4(xh, X + ao);
+                    ldmatrix_x4(xl, X + kGC * kAP + ao);
+                    mma_split(acc[0], xh, xl, bh[ks][0], bh[ks][1], bl[ks][0], bl[ks][1]);
+                    mma_split(acc[1], xh, xl, bh[ks][2], bh[ks][3], bl[ks][2], bl[ks][3]);
                 }
+#pragma unroll
+                for (int b = 0; b < 2; ++b)
+#pragma unroll
+                    for (int e = 0; e < 4; e += 2) {
+                        const int t = m * 16 + g + (e >> 1) * 8, d = c0 + b * 8 + 2 * tq;
+                        if (!is_v) {
+                            uint32_t hi, lo;
+                            split_bf16x2(acc[b][e], acc[b][e + 1], hi, lo);
+                            uint32_t* p = reinterpret_cast<uint32_t*>(out + 4 * lay.plane) + (t * DK + d) / 2;
+                            p[0] = hi;
+                            p[lay.plane] = lo;
+                        } else if (v0 + d < ca.dvp) {
+                            float* p = ca.u0 + (((size_t)c * a.heads + h) * kGC + t) * ca.dvp + v0 + d;
+                            *reinterpret_cast<float2*>(p) = make_float2(acc[b][e], acc[b][e + 1]);
+                        }
+                    }
+            }
         }
     }
 }

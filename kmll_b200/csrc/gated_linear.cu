@@ -11,9 +11,13 @@
 //   o_i = (q_i 2^G_i) S_in + sum_{j <= i} A_ij u_j           A_ij = sum_d q_id k_jd 2^(G_id - G_jd)
 //   S_out = diag(2^G_n) S_in + sum_j (k_j 2^(G_n - G_j)) u_j^T
 // and for the delta rule (I + L) U = beta (V - (K 2^G) S_in) with L_ij = beta_i sum_d k_id k_jd 2^(G_id - G_jd), j < i; so with
-// X = (I + L)^-1 each chunk's U = X beta V - W S_in, W = X beta (K 2^G).  Every exponent that is evaluated is a sum of log decays
-// over consecutive tokens, hence not positive: blocks of 16 x 16 tokens below the diagonal factor through the row ahead of the
-// block, blocks on the diagonal are summed directly.
+// X = (I + L)^-1 each chunk's U = X beta V - W S_in, W = X beta (K 2^G).  A and L are made in blocks of 16 x 16 tokens whose
+// factors refer to one row's G.  Below the diagonal that is the row ahead of the block, so that both exponents are sums of log
+// decays and not positive.  On the diagonal it is the block's first row, and the keys' exponents are positive; a block in which
+// some channel decays to less than 2^-90 is summed pair by pair instead.
+
+#include <type_traits>
+
 #include "activations.cuh"
 #include "mma_bf16.cuh"
 
@@ -401,7 +405,7 @@ __device__ inline void mma_split(float (&c)[4], const uint32_t (&ah)[4], const u
 // projected rows they come from.
 struct PrepareLayout {
     int P, PR;             // pitches: f32 rows, rows of the decay map
-    int off_k, off_g, off_l, off_v, staged_decay, total;
+    int off_k, off_g, off_l, off_x, off_v, staged_decay, total;
 };
 __host__ __device__ inline PrepareLayout prepare_layout(int DK, int delta, int taps, int rank) {
     PrepareLayout l;
@@ -411,7 +415,8 @@ __host__ __device__ inline PrepareLayout prepare_layout(int DK, int delta, int t
     l.off_k = tile;
     l.off_g = 2 * tile;
     l.off_l = l.off_g + (2 * raw > tile ? 2 * raw : tile);
-    l.off_v = l.off_l + (delta ? kGC * kAP * 4 : 0);
+    l.off_x = l.off_l + (delta ? kGC * kAP * 4 : 0);
+    l.off_v = l.off_x + (delta ? 2 * kGC * kAP * 2 : 0);
     l.total = l.off_v + (delta ? raw : 0);
     l.staged_decay = (kGC + DK) * l.PR * 2 <= 2 * tile;  // the decay factor and map fit in the places of q and k
     return l;
@@ -443,38 +448,47 @@ __device__ inline void stage_rows(const GatedLinearArgs& a, uint16_t* tile, int 
     }
 }
 __device__ inline float2 unpack2(uint32_t x) { return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u)); }
-// channels d, d + 1 of tokens t .. t + ROWS - 1 from a staged tile, through convolution and SiLU; ch: ring channel of d; odd:
-// channel d + 1 does not exist
+// taps of channels ch, ch + 1 (odd: of ch alone), up to four of them, the last at index 3
+struct PairTaps { float2 w[4]; };
+__device__ inline PairTaps load_taps(const GatedLinearArgs& a, int ch, bool live, bool odd) {
+    PairTaps p;
+    const int lead = 4 - a.taps;
+    const uint16_t* w = a.conv + (size_t)ch * a.taps;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const bool on = live && a.taps > 0 && a.taps <= 4 && j >= lead;
+        p.w[j] = make_float2(on ? bf16_bits_to_f32(w[j - lead]) : 0.0f, on && !odd ? bf16_bits_to_f32(w[a.taps + j - lead]) : 0.0f);
+    }
+    return p;
+}
+// channels d, d + 1 of tokens t .. t + ROWS - 1 from a staged tile, through convolution and SiLU
 template <int DK, int ROWS>
-__device__ inline void staged_rows(const GatedLinearArgs& a, const uint16_t* tile, int t, int d, int ch, bool odd, float2 (&y)[ROWS]) {
+__device__ inline void staged_rows(const GatedLinearArgs& a, const uint16_t* tile, int t, int d, const PairTaps& taps, int ch, bool odd, float2 (&y)[ROWS]) {
     auto at = [&](int r) { return unpack2(*reinterpret_cast<const uint32_t*>(tile + r * DK + d)); };
     if (a.taps == 0) {
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) y[i] = at(t + i);
         return;
     }
-    const uint16_t* w0 = a.conv + (size_t)ch * a.taps;
-    const uint16_t* w1 = odd ? w0 : w0 + a.taps;
     if (a.taps <= 4) {
         const int lead = 4 - a.taps;  // missing taps
-        float2 w[4], x[4];
+        float2 x[4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            w[j] = j >= lead ? make_float2(bf16_bits_to_f32(w0[j - lead]), bf16_bits_to_f32(w1[j - lead])) : make_float2(0.0f, 0.0f);
-            x[j] = j >= lead && j < 3 ? at(t + j - lead) : make_float2(0.0f, 0.0f);
-        }
+        for (int j = 0; j < 3; ++j) x[j] = j >= lead ? at(t + j - lead) : make_float2(0.0f, 0.0f);
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) {
             x[3] = at(t + i + 3 - lead);
-            float2 s = __ffma2_rn(w[0], x[0], make_float2(0.0f, 0.0f));
-            s = __ffma2_rn(w[1], x[1], s);
-            s = __ffma2_rn(w[2], x[2], s);
-            y[i] = __ffma2_rn(w[3], x[3], s);
+            float2 s = __fmul2_rn(taps.w[0], x[0]);
+            s = __ffma2_rn(taps.w[1], x[1], s);
+            s = __ffma2_rn(taps.w[2], x[2], s);
+            y[i] = __ffma2_rn(taps.w[3], x[3], s);
             x[0] = x[1];
             x[1] = x[2];
             x[2] = x[3];
         }
     } else {
+        const uint16_t* w0 = a.conv + (size_t)ch * a.taps;
+        const uint16_t* w1 = odd ? w0 : w0 + a.taps;
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) y[i] = make_float2(0.0f, 0.0f);
         for (int j = 0; j < a.taps; ++j) {
@@ -496,7 +510,8 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
     float* const Q = reinterpret_cast<float*>(gsm);               // [64][P]
     float* const K = reinterpret_cast<float*>(gsm + pl.off_k);    // [64][P]
     float* const G = reinterpret_cast<float*>(gsm + pl.off_g);    // [64][P] log2 decays, then their running sums
-    float* const L = reinterpret_cast<float*>(gsm + pl.off_l);    // DELTA: [64][kAP] L, then its inverse
+    float* const L = reinterpret_cast<float*>(gsm + pl.off_l);    // DELTA: [64][kAP]
+    uint16_t* const X = reinterpret_cast<uint16_t*>(gsm + pl.off_x);  // DELTA: (I + L)^-1, [2][64][kAP] heads, remainders
     const int back = a.taps > 0 ? a.taps - 1 : 0;
     uint16_t* const raw_q = reinterpret_cast<uint16_t*>(gsm + pl.off_g);
     uint16_t* const raw_k = raw_q + (kGC + back) * DK;
@@ -523,6 +538,22 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
             cp_async16_zfill_to((uint32_t)__cvta_generic_to_shared(su + d * pl.PR + r), live ? a.up + (size_t)(h * a.dk + d) * a.ldu + r : a.up, live ? 16u : 0u);
         }
     const float rate = decay_rate(a, h);
+    constexpr int PAIRS = DK / 2, ROWS = kGC * PAIRS / NT;  // a thread convolves two channels of ROWS tokens
+    const int pd = (tid % PAIRS) * 2, pt = tid / PAIRS * ROWS;
+    const bool p_live = pd < a.dk, p_odd = pd + 1 >= a.dk;
+    const PairTaps wq = load_taps(a, chq + pd, p_live, p_odd), wk = load_taps(a, nq + chq + pd, p_live, p_odd);
+    PairTaps wv = load_taps(a, chv + pd, DELTA && pd < a.dv, pd + 1 >= a.dv);
+    // log decays: a warp holds 16 x MB tokens of 8 x NB channels
+    constexpr int NB = DK == 64 && NW == 16 ? 1 : DK / 64, MB = DK / NB * 4 / 8 / NW;
+    const int cb = warp % (DK / 8 / NB) * NB, mb = warp / (DK / 8 / NB) * MB;
+    float bias[NB][2];
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int d = (cb + b) * 8 + 2 * tq + e;
+            bias[b][e] = a.bias != nullptr && d < a.dk ? bf16_bits_to_f32(a.bias[h * a.dk + d]) : 0.0f;
+        }
     pdl_wait();
     if (pl.staged_decay)
         for (int i = tid; i < kGC * runs; i += NT) {
@@ -536,13 +567,9 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
     if (DELTA) stage_rows<DK, NT>(a, raw_v, t0, n, a.v_off + h * a.dv, chv, a.dv, channels, fast);
     asm volatile("cp.async.commit_group;" ::: "memory");
     if (tid < kGC) beta[tid] = !DELTA ? 1.0f : tid < n ? act_sigmoid(bf16_bits_to_f32(in[(size_t)(t0 + tid) * a.ld + a.b_off + h])) : 0.0f;
-    if (DELTA)
-        for (int i = tid; i < kGC * kAP; i += NT) L[i] = 0.0f;
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
-    // ---- log decays from z = W_up a: 64 tokens x DK channels; a warp holds 16 x MB tokens of 8 x NB channels
-    constexpr int NB = DK == 64 && NW == 16 ? 1 : DK / 64, MB = DK / NB * 4 / 8 / NW;
-    const int cb = warp % (DK / 8 / NB) * NB, mb = warp / (DK / 8 / NB) * MB;
+    // ---- log decays from z = W_up a
     float z[NB][MB][4];
 #pragma unroll
     for (int b = 0; b < NB; ++b)
@@ -593,27 +620,24 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
 #pragma unroll
             for (int e = 0; e < 4; ++e) {  // tokens behind the last change nothing: decay 1
                 const int t = (mb + m) * 16 + g + (e >> 1) * 8, d = (cb + b) * 8 + 2 * tq + (e & 1);
-                z[b][m][e] = t < n && d < a.dk ? fast_log2_decay(a, z[b][m][e] + (a.bias != nullptr ? bf16_bits_to_f32(a.bias[h * a.dk + d]) : 0.0f), rate) : 0.0f;
+                z[b][m][e] = t < n && d < a.dk ? fast_log2_decay(a, z[b][m][e] + bias[b][e & 1], rate) : 0.0f;
             }
     __syncthreads();  // the decay factor and map have been read
-    constexpr int PAIRS = DK / 2, ROWS = kGC * PAIRS / NT;  // a thread: two channels of ROWS tokens
-    const int pd = (tid % PAIRS) * 2, pt = tid / PAIRS * ROWS;
     // ---- q and k
     {
         const float fq = a.unit_eps > 0.0f ? 1.0f : a.q_scale;
-        const bool live = pd < a.dk, odd = pd + 1 >= a.dk;
         float2 q[ROWS], k[ROWS];
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) q[i] = k[i] = make_float2(0.0f, 0.0f);
-        if (live) {
-            staged_rows<DK, ROWS>(a, raw_q, pt, pd, chq + pd, odd, q);
-            staged_rows<DK, ROWS>(a, raw_k, pt, pd, nq + chq + pd, odd, k);
+        if (p_live) {
+            staged_rows<DK, ROWS>(a, raw_q, pt, pd, wq, chq + pd, p_odd, q);
+            staged_rows<DK, ROWS>(a, raw_k, pt, pd, wk, nq + chq + pd, p_odd, k);
         }
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) {
-            const bool on = live && pt + i < n;
-            *reinterpret_cast<float2*>(Q + (pt + i) * P + pd) = make_float2(on ? q[i].x * fq : 0.0f, on && !odd ? q[i].y * fq : 0.0f);
-            *reinterpret_cast<float2*>(K + (pt + i) * P + pd) = make_float2(on ? k[i].x : 0.0f, on && !odd ? k[i].y : 0.0f);
+            const bool on = p_live && pt + i < n;
+            *reinterpret_cast<float2*>(Q + (pt + i) * P + pd) = make_float2(on ? q[i].x * fq : 0.0f, on && !p_odd ? q[i].y * fq : 0.0f);
+            *reinterpret_cast<float2*>(K + (pt + i) * P + pd) = make_float2(on ? k[i].x : 0.0f, on && !p_odd ? k[i].y : 0.0f);
         }
     }
     __syncthreads();  // the projected rows have been read
@@ -625,22 +649,36 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
             for (int e = 0; e < 4; e += 2)
                 *reinterpret_cast<float2*>(G + ((mb + m) * 16 + g + (e >> 1) * 8) * P + (cb + b) * 8 + 2 * tq) = make_float2(z[b][m][e], z[b][m][e + 1]);
     // ---- unit vectors; running sums of the log decays
-    if (a.unit_eps > 0.0f)
-        for (int r = warp; r < 2 * kGC; r += NW) {
-            constexpr int V = DK / 32;
-            float* x = (r < kGC ? Q : K) + (r & (kGC - 1)) * P + lane * V;
-            float v[V], sq = 0.0f;
+    if (a.unit_eps > 0.0f) {
+        constexpr int RN = 2 * kGC / NW, V = DK / 32;  // rows per warp, four at a time; entries per lane
 #pragma unroll
-            for (int i = 0; i < V; i += 2) {
-                const float2 t = *reinterpret_cast<const float2*>(x + i);
-                v[i] = t.x;
-                v[i + 1] = t.y;
-                sq += t.x * t.x + t.y * t.y;
+        for (int r0 = 0; r0 < RN; r0 += 4) {
+            float v[4][V], sum[4];
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                const int r = warp * RN + r0 + x;
+                const float* p = (r < kGC ? Q : K - kGC * P) + r * P + lane * V;
+                sum[x] = 0.0f;
+#pragma unroll
+                for (int i = 0; i < V; ++i) {
+                    v[x][i] = p[i];
+                    sum[x] += v[x][i] * v[x][i];
+                }
             }
-            const float f = (r < kGC ? a.q_scale : 1.0f) * rsqrtf(warp_sum(sq) + a.unit_eps);
 #pragma unroll
-            for (int i = 0; i < V; i += 2) *reinterpret_cast<float2*>(x + i) = make_float2(v[i] * f, v[i + 1] * f);
+            for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) sum[x] += __shfl_xor_sync(0xffffffffu, sum[x], off);
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                const int r = warp * RN + r0 + x;
+                float* p = (r < kGC ? Q : K - kGC * P) + r * P + lane * V;
+                const float f = (r < kGC ? a.q_scale : 1.0f) * rsqrtf(sum[x] + a.unit_eps);
+#pragma unroll
+                for (int i = 0; i < V; ++i) p[i] = v[x][i] * f;
+            }
         }
+    }
     __syncthreads();
     {
         constexpr int SEG = NT / DK, LEN = kGC / SEG;
@@ -658,99 +696,136 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
         for (int i = 0; i < LEN; ++i) G[(seg * LEN + i) * P + d] = run[i] + before;
     }
     __syncthreads();
-    // ---- A (to its planes) and L: six 16 x 16 blocks below the diagonal, then the pairs on the diagonal blocks, 32 at a time
-    constexpr int kPairs = 136, kUnits = 6 + 4 * kPairs / 32;
-    for (int u = warp; u < kUnits; u += NW) {
-        if (u < 6) {
-            const int I = u < 1 ? 1 : u < 3 ? 2 : 3, J = u - (I * (I - 1)) / 2, ref = I * 16 - 1;
-            const int ia = I * 16 + g, ib = ia + 8;
-            float ca_[2][4] = {}, cl_[2][4] = {};
-#pragma unroll 2
-            for (int k0 = 0; k0 < DK; k0 += 16) {
-                uint32_t qh[4], ql[4], kh[4], kl[4];
+    // ---- A (to its planes) and L: ten 16 x 16 blocks; steep ones on the diagonal in tiles of 2 x 2 tokens, two lanes each
+    unsigned steep = 0;  // bit b: block b on the diagonal
 #pragma unroll
-                for (int x = 0; x < 2; ++x) {  // channels d, d + 1 of both rows
-                    const int d = k0 + x * 8 + 2 * tq;
-                    const float2 gr = *reinterpret_cast<const float2*>(G + ref * P + d);
+    for (int b = 0; b < 4; ++b) {
+        bool far = false;
+#pragma unroll
+        for (int d = 0; d < DK; d += 32) far |= G[b * 16 * P + d + lane] - G[(b * 16 + 15) * P + d + lane] > 90.0f;
+        steep |= __any_sync(0xffffffffu, far) ? 1u << b : 0u;
+    }
+    for (int u = warp; u < (steep != 0u ? 19 : 10); u += NW) {
+        if (u >= 10) {
+            const int p = (u - 10) * 32 + lane, half = p & 1, B = (p >> 1) / 36;
+            if ((__ballot_sync(0xffffffffu, (steep >> B & 1u) != 0u)) == 0u) continue;
+            const bool mine = (steep >> B & 1u) != 0u;
+            int ti = 0, tj = (p >> 1) - B * 36;
+            while (tj > ti) tj -= ++ti;
+            const int i = B * 16 + ti * 2, j = B * 16 + tj * 2;
+            const float2 minus = make_float2(-1.0f, -1.0f);
+            float2 sq[2][2] = {}, sl[2][2] = {};
+#pragma unroll 2
+            for (int d = half * 4; d < DK; d += 8) {
+                float4 gi[2], gj[2], qi[2], ki[2], kj[2];
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    gi[x] = *reinterpret_cast<const float4*>(G + (i + x) * P + d);
+                    gj[x] = *reinterpret_cast<const float4*>(G + (j + x) * P + d);
+                    qi[x] = *reinterpret_cast<const float4*>(Q + (i + x) * P + d);
+                    kj[x] = *reinterpret_cast<const float4*>(K + (j + x) * P + d);
+                    if (DELTA) ki[x] = *reinterpret_cast<const float4*>(K + (i + x) * P + d);
+                }
+#pragma unroll
+                for (int x = 0; x < 2; ++x)
 #pragma unroll
                     for (int y = 0; y < 2; ++y) {
-                        const int i = y == 0 ? ia : ib;
-                        const float2 gi = *reinterpret_cast<const float2*>(G + i * P + d);
-                        const float e0 = ex2_approx(gi.x - gr.x), e1 = ex2_approx(gi.y - gr.y);
-                        const float2 q = *reinterpret_cast<const float2*>(Q + i * P + d);
-                        split_bf16x2(q.x * e0, q.y * e1, qh[x * 2 + y], ql[x * 2 + y]);
+                        float2 e0 = __ffma2_rn(make_float2(gj[y].x, gj[y].y), minus, make_float2(gi[x].x, gi[x].y));
+                        float2 e1 = __ffma2_rn(make_float2(gj[y].z, gj[y].w), minus, make_float2(gi[x].z, gi[x].w));
+                        e0 = __fmul2_rn(make_float2(kj[y].x, kj[y].y), make_float2(ex2_approx(e0.x), ex2_approx(e0.y)));
+                        e1 = __fmul2_rn(make_float2(kj[y].z, kj[y].w), make_float2(ex2_approx(e1.x), ex2_approx(e1.y)));
+                        sq[x][y] = __ffma2_rn(make_float2(qi[x].x, qi[x].y), e0, sq[x][y]);
+                        sq[x][y] = __ffma2_rn(make_float2(qi[x].z, qi[x].w), e1, sq[x][y]);
                         if (DELTA) {
-                            const float2 k = *reinterpret_cast<const float2*>(K + i * P + d);
-                            split_bf16x2(k.x * e0, k.y * e1, kh[x * 2 + y], kl[x * 2 + y]);
+                            sl[x][y] = __ffma2_rn(make_float2(ki[x].x, ki[x].y), e0, sl[x][y]);
+                            sl[x][y] = __ffma2_rn(make_float2(ki[x].z, ki[x].w), e1, sl[x][y]);
                         }
                     }
-                }
+            }
+            float vq[2][2], vl[2][2];
 #pragma unroll
-                for (int nb = 0; nb < 2; ++nb) {
-                    const int j = J * 16 + nb * 8 + g;
-                    uint32_t bh[2], bl[2];
+            for (int x = 0; x < 2; ++x)
 #pragma unroll
-                    for (int x = 0; x < 2; ++x) {
-                        const int d = k0 + x * 8 + 2 * tq;
-                        const float2 gr = *reinterpret_cast<const float2*>(G + ref * P + d), gj = *reinterpret_cast<const float2*>(G + j * P + d);
-                        const float2 k = *reinterpret_cast<const float2*>(K + j * P + d);
-                        split_bf16x2(k.x * ex2_approx(gr.x - gj.x), k.y * ex2_approx(gr.y - gj.y), bh[x], bl[x]);
+                for (int y = 0; y < 2; ++y) {
+                    vq[x][y] = sq[x][y].x + sq[x][y].y;
+                    vq[x][y] += __shfl_xor_sync(0xffffffffu, vq[x][y], 1);
+                    if (DELTA) {
+                        vl[x][y] = sl[x][y].x + sl[x][y].y;
+                        vl[x][y] += __shfl_xor_sync(0xffffffffu, vl[x][y], 1);
                     }
-                    mma_split(ca_[nb], qh, ql, bh[0], bh[1], bl[0], bl[1]);
-                    if (DELTA) mma_split(cl_[nb], kh, kl, bh[0], bh[1], bl[0], bl[1]);
                 }
+            if (!mine) continue;
+            // this lane's row i + half, columns j and j + 1; tokens behind it are not seen (their sums may be anything)
+            const int r = i + half;
+            uint32_t hi, lo;
+            split_bf16x2(half ? vq[1][0] : vq[0][0], j + 1 <= r ? (half ? vq[1][1] : vq[0][1]) : 0.0f, hi, lo);
+            *reinterpret_cast<uint32_t*>(Ah + r * kGC + j) = hi;
+            *reinterpret_cast<uint32_t*>(Al + r * kGC + j) = lo;
+            if (DELTA) *reinterpret_cast<float2*>(L + r * kAP + j) =
+                make_float2(j < r ? beta[r] * (half ? vl[1][0] : vl[0][0]) : 0.0f, j + 1 < r ? beta[r] * (half ? vl[1][1] : vl[0][1]) : 0.0f);
+            if (tj < ti) {  // the mirrored tile above the diagonal
+                *reinterpret_cast<uint32_t*>(Ah + (j + half) * kGC + i) = 0u;
+                *reinterpret_cast<uint32_t*>(Al + (j + half) * kGC + i) = 0u;
             }
-#pragma unroll
-            for (int nb = 0; nb < 2; ++nb)
-#pragma unroll
-                for (int e = 0; e < 4; e += 2) {
-                    const int i = (e >> 1) ? ib : ia, j = J * 16 + nb * 8 + 2 * tq;
-                    uint32_t hi, lo;
-                    split_bf16x2(ca_[nb][e], ca_[nb][e + 1], hi, lo);
-                    *reinterpret_cast<uint32_t*>(Ah + i * kGC + j) = hi;
-                    *reinterpret_cast<uint32_t*>(Al + i * kGC + j) = lo;
-                    if (DELTA) *reinterpret_cast<float2*>(L + i * kAP + j) = make_float2(beta[i] * cl_[nb][e], beta[i] * cl_[nb][e + 1]);
-                }
-        } else {
-            const int p = (u - 6) * 32 + lane, B = p / kPairs, r = p - B * kPairs;
-            int i = (int)((sqrtf(8.0f * (float)r + 1.0f) - 1.0f) * 0.5f);
-            if (i * (i + 1) / 2 > r) --i;
-            if ((i + 1) * (i + 2) / 2 <= r) ++i;
-            const int j = B * 16 + r - i * (i + 1) / 2;
-            i += B * 16;
-            float2 sq2 = make_float2(0.0f, 0.0f), sl2 = sq2;
-            const float2 minus = make_float2(-1.0f, -1.0f);
+            continue;
+        }
+        const int I = u < 1 ? 0 : u < 3 ? 1 : u < 6 ? 2 : 3, J = u - I * (I + 1) / 2, ref = J < I ? I * 16 - 1 : I * 16;
+        if (J == I && (steep >> I & 1u) != 0u) continue;
+        const int ia = I * 16 + g, ib = ia + 8;
+        float ca_[2][4] = {}, cl_[2][4] = {};
 #pragma unroll 4
-            for (int d = 0; d < DK; d += 4) {
-                const float4 gi = *reinterpret_cast<const float4*>(G + i * P + d), gj = *reinterpret_cast<const float4*>(G + j * P + d);
-                const float4 kj = *reinterpret_cast<const float4*>(K + j * P + d), qi = *reinterpret_cast<const float4*>(Q + i * P + d);
-                float2 e0 = __ffma2_rn(make_float2(gj.x, gj.y), minus, make_float2(gi.x, gi.y)), e1 = __ffma2_rn(make_float2(gj.z, gj.w), minus, make_float2(gi.z, gi.w));
-                e0 = __fmul2_rn(make_float2(kj.x, kj.y), make_float2(ex2_approx(e0.x), ex2_approx(e0.y)));
-                e1 = __fmul2_rn(make_float2(kj.z, kj.w), make_float2(ex2_approx(e1.x), ex2_approx(e1.y)));
-                sq2 = __ffma2_rn(make_float2(qi.x, qi.y), e0, sq2);
-                sq2 = __ffma2_rn(make_float2(qi.z, qi.w), e1, sq2);
-                if (DELTA) {
-                    const float4 ki = *reinterpret_cast<const float4*>(K + i * P + d);
-                    sl2 = __ffma2_rn(make_float2(ki.x, ki.y), e0, sl2);
-                    sl2 = __ffma2_rn(make_float2(ki.z, ki.w), e1, sl2);
+        for (int k0 = 0; k0 < DK; k0 += 16) {
+            uint32_t qh[4], ql[4], kh[4], kl[4];
+            float2 gr[2];
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {  // channels d, d + 1 of both rows
+                const int d = k0 + x * 8 + 2 * tq;
+                gr[x] = *reinterpret_cast<const float2*>(G + ref * P + d);
+#pragma unroll
+                for (int y = 0; y < 2; ++y) {
+                    const int i = y == 0 ? ia : ib;
+                    const float2 gi = *reinterpret_cast<const float2*>(G + i * P + d);
+                    const float2 e = make_float2(ex2_approx(gi.x - gr[x].x), ex2_approx(gi.y - gr[x].y));
+                    const float2 q = __fmul2_rn(*reinterpret_cast<const float2*>(Q + i * P + d), e);
+                    split_bf16x2(q.x, q.y, qh[x * 2 + y], ql[x * 2 + y]);
+                    if (DELTA) {
+                        const float2 k = __fmul2_rn(*reinterpret_cast<const float2*>(K + i * P + d), e);
+                        split_bf16x2(k.x, k.y, kh[x * 2 + y], kl[x * 2 + y]);
+                    }
                 }
             }
-            const float sq = sq2.x + sq2.y, sl = sl2.x + sl2.y;
-            const uint16_t hi = f32_to_bf16_bits(sq);
-            Ah[i * kGC + j] = hi;
-            Al[i * kGC + j] = f32_to_bf16_bits(sq - bf16_bits_to_f32(hi));
-            if (j < i) {  // the mirrored place above the diagonal
-                Ah[j * kGC + i] = 0;
-                Al[j * kGC + i] = 0;
-                if (DELTA) L[i * kAP + j] = beta[i] * sl;
+#pragma unroll
+            for (int nb = 0; nb < 2; ++nb) {
+                const int j = J * 16 + nb * 8 + g;
+                uint32_t bh[2], bl[2];
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const int d = k0 + x * 8 + 2 * tq;
+                    const float2 gj = *reinterpret_cast<const float2*>(G + j * P + d);
+                    const float2 k = __fmul2_rn(*reinterpret_cast<const float2*>(K + j * P + d), make_float2(ex2_approx(gr[x].x - gj.x), ex2_approx(gr[x].y - gj.y)));
+                    split_bf16x2(k.x, k.y, bh[x], bl[x]);
+                }
+                mma_split(ca_[nb], qh, ql, bh[0], bh[1], bl[0], bl[1]);
+                if (DELTA) mma_split(cl_[nb], kh, kl, bh[0], bh[1], bl[0], bl[1]);
             }
         }
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+                const int i = (e >> 1) ? ib : ia, j = J * 16 + nb * 8 + 2 * tq;
+                uint32_t hi, lo;
+                split_bf16x2(j <= i ? ca_[nb][e] : 0.0f, j + 1 <= i ? ca_[nb][e + 1] : 0.0f, hi, lo);
+                *reinterpret_cast<uint32_t*>(Ah + i * kGC + j) = hi;
+                *reinterpret_cast<uint32_t*>(Al + i * kGC + j) = lo;
+                if (DELTA) *reinterpret_cast<float2*>(L + i * kAP + j) = make_float2(j < i ? beta[i] * cl_[nb][e] : 0.0f, j + 1 < i ? beta[i] * cl_[nb][e + 1] : 0.0f);
+            }
     }
     __syncthreads();
-    // ---- planes of q and k; the inverse of I + L by forward substitution, one column per thread of the first two warps
-    if (!DELTA || warp >= 2) {
-        const int first = DELTA ? tid - 64 : tid, step = DELTA ? NT - 64 : NT;
-        for (int i = first; i < kGC * DK / 2; i += step) {
+    // ---- planes of q and k; meanwhile the first four warps invert I + L
+    constexpr int IW = DELTA ? 128 : 0;  // threads that invert
+    if (!DELTA || warp >= 4) {
+        for (int i = tid - IW; i < kGC * DK / 2; i += NT - IW) {
             const int t = i / (DK / 2), d = (i % (DK / 2)) * 2;
             const float2 gt = *reinterpret_cast<const float2*>(G + t * P + d), gn = *reinterpret_cast<const float2*>(G + (kGC - 1) * P + d);
             const float2 q = *reinterpret_cast<const float2*>(Q + t * P + d), k = *reinterpret_cast<const float2*>(K + t * P + d);
@@ -764,38 +839,76 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
             p[3 * lay.plane] = lo;
         }
         float* dn = out + (DELTA ? 6 : 4) * lay.plane + 2 * lay.a_plane;
-        for (int d = first; d < DK; d += step) dn[d] = ex2_approx(G[(kGC - 1) * P + d]);
+        for (int d = tid - IW; d < DK; d += NT - IW) dn[d] = ex2_approx(G[(kGC - 1) * P + d]);
     } else if (DELTA) {
-        float x[kGC];
+        if (warp < 2) {  // the four blocks on the diagonal by forward substitution, a column per thread
+            const int r0 = (tid >> 4) * 16, col = tid & 15;
+            float x[16];
 #pragma unroll
-        for (int i = 0; i < kGC; ++i) {
-            float s0 = i == tid ? 1.0f : 0.0f, s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
+            for (int i = 0; i < 16; ++i) {
+                float s0 = i == col ? 1.0f : 0.0f, s1 = 0.0f;
 #pragma unroll
-            for (int m = 0; m + 3 < i; m += 4) {
-                const float4 l = *reinterpret_cast<const float4*>(L + i * kAP + m);
-                s0 = fmaf(-l.x, x[m], s0);
-                s1 = fmaf(-l.y, x[m + 1], s1);
-                s2 = fmaf(-l.z, x[m + 2], s2);
-                s3 = fmaf(-l.w, x[m + 3], s3);
+                for (int m = 0; m < i; ++m) {
+                    const float l = L[(r0 + i) * kAP + r0 + m];
+                    if (m & 1) s1 = fmaf(-l, x[m], s1);
+                    else s0 = fmaf(-l, x[m], s0);
+                }
+                x[i] = s0 + s1;
             }
 #pragma unroll
-            for (int m = i / 4 * 4; m < i; ++m) s0 = fmaf(-L[i * kAP + m], x[m], s0);
-            x[i] = (s0 + s1) + (s2 + s3);
+            for (int i = 0; i < 16; ++i) {
+                const uint16_t hi = f32_to_bf16_bits(x[i]);
+                X[(r0 + i) * kAP + r0 + col] = hi;
+                X[(kGC + r0 + i) * kAP + r0 + col] = f32_to_bf16_bits(x[i] - bf16_bits_to_f32(hi));
+            }
         }
-        asm volatile("bar.sync 1, 64;" ::: "memory");  // both warps have read L
-        uint16_t* const X = reinterpret_cast<uint16_t*>(L);  // [2][64][kAP]: heads, remainders
+        for (int dist = 1; dist < 4; ++dist) {  // X_IJ = -X_II sum_{J <= M < I} L_IM X_MJ, blocks `dist` below the diagonal
+            asm volatile("bar.sync 1, 128;" ::: "memory");
+            if (warp >= 4 - dist) continue;
+            const int J = warp, I = J + dist;
+            float pt_[2][4] = {};  // the sum, transposed: [column of X_MJ][row of L_IM]
+            for (int M = J; M < I; ++M) {
+                uint32_t xh[4], xl[4];
+                const int ao = (M * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * kAP + J * 16 + ((lane >> 3) & 1) * 8;
+                ldmatrix_x4_trans(xh, X + ao);
+                ldmatrix_x4_trans(xl, X + kGC * kAP + ao);
 #pragma unroll
-        for (int i = 0; i < kGC; ++i) {
-            const uint16_t hi = f32_to_bf16_bits(x[i]);
-            X[i * kAP + tid] = hi;
-            X[(kGC + i) * kAP + tid] = f32_to_bf16_bits(x[i] - bf16_bits_to_f32(hi));
+                for (int nb = 0; nb < 2; ++nb) {
+                    uint32_t bh[2], bl[2];
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        const float2 l = *reinterpret_cast<const float2*>(L + (I * 16 + nb * 8 + g) * kAP + M * 16 + x * 8 + 2 * tq);
+                        split_bf16x2(l.x, l.y, bh[x], bl[x]);
+                    }
+                    mma_split(pt_[nb], xh, xl, bh[0], bh[1], bl[0], bl[1]);
+                }
+            }
+            uint32_t dh[4], dl[4];
+            const int ao = (I * 16 + (lane & 15)) * kAP + I * 16 + (lane >> 4) * 8;
+            ldmatrix_x4(dh, X + ao);
+            ldmatrix_x4(dl, X + kGC * kAP + ao);
+#pragma unroll
+            for (int nb = 0; nb < 2; ++nb) {
+                float r[4] = {};
+                uint32_t bh[2], bl[2];
+                split_bf16x2(-pt_[0][2 * nb], -pt_[0][2 * nb + 1], bh[0], bl[0]);
+                split_bf16x2(-pt_[1][2 * nb], -pt_[1][2 * nb + 1], bh[1], bl[1]);
+                mma_split(r, dh, dl, bh[0], bh[1], bl[0], bl[1]);
+#pragma unroll
+                for (int e = 0; e < 4; e += 2) {
+                    uint32_t hi, lo;
+                    split_bf16x2(r[e], r[e + 1], hi, lo);
+                    const int o = (I * 16 + g + (e >> 1) * 8) * kAP + J * 16 + nb * 8 + 2 * tq;
+                    *reinterpret_cast<uint32_t*>(X + o) = hi;
+                    *reinterpret_cast<uint32_t*>(X + kGC * kAP + o) = lo;
+                }
+            }
         }
     }
     if (!DELTA) return;
     // ---- W = X (beta k 2^G), U0 = X (beta v): right-hand sides as head / remainder planes [2][64][PB] in the places of q, k and the
     // decays, DK value columns at a time; a warp takes 16 columns
     constexpr int PB = DK + 8;
-    uint16_t* const X = reinterpret_cast<uint16_t*>(L);
     uint16_t* const Rk = reinterpret_cast<uint16_t*>(gsm);
     uint16_t* const Rv = Rk + 2 * kGC * PB;
     auto put = [&](uint16_t* R, int t, float x, float y) {
@@ -828,8 +941,9 @@ __global__ void __launch_bounds__(DELTA ? 512 : 256) gated_chunk_prepare_kernel(
         {
             const int col = v0 + pd;
             const bool live = col < a.dv, odd = col + 1 >= a.dv;
+            if (v0 > 0) wv = load_taps(a, chv + col, live, odd);
             float2 v[ROWS];
-            if (live) staged_rows<DK, ROWS>(a, raw_v, pt, pd, chv + col, odd, v);
+            if (live) staged_rows<DK, ROWS>(a, raw_v, pt, pd, wv, chv + col, odd, v);
 #pragma unroll
             for (int i = 0; i < ROWS; ++i) {
                 const bool on = live && pt + i < n;
@@ -912,28 +1026,30 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_scan_kernel(const Chunk
             s[i][e] = d < a.dk && col < a.dv ? S[(size_t)d * a.dv + col] : 0.0f;
         }
     pdl_wait();
-    auto copy = [&](uint16_t* tile, const uint16_t* src, int rows, int cols, int pitch) {
-        const int runs = cols / 8;
-        for (int i = tid; i < rows * runs; i += kGThreads) {
-            const int r = i / runs, cc = (i - r * runs) * 8;
-            cp_async16_to((uint32_t)__cvta_generic_to_shared(tile + r * pitch + cc), src + (size_t)r * cols + cc);
-        }
+    auto copy = [&](uint16_t* tile, const uint16_t* src, auto columns) {  // head and remainder planes [2][64][columns]
+        constexpr int COLS = decltype(columns)::value, RUNS = COLS / 8;
+        const uint32_t dst = (uint32_t)__cvta_generic_to_shared(tile) + (uint32_t)((tid / RUNS) * (COLS + 8) + (tid % RUNS) * 8) * 2;
+#pragma unroll
+        for (int i = 0; i < 2 * kGC * RUNS / kGThreads; ++i)
+            cp_async16_to(dst + (uint32_t)(i * (kGThreads / RUNS) * (COLS + 8)) * 2, src + (size_t)(i * kGThreads + tid) * 8);
     };
+    using Keys = std::integral_constant<int, DK>;
+    using Tokens = std::integral_constant<int, kGC>;
     auto source = [&](int c) { return ca.planes + ((size_t)c * a.heads + h) * lay.floats; };
     auto load_first = [&](int c) {  // q 2^G, W
         if (c < ca.chunks) {
             const float* p = source(c);
-            copy(Qt, reinterpret_cast<const uint16_t*>(p), 2 * kGC, DK, P);
-            if (DELTA) copy(Wt, reinterpret_cast<const uint16_t*>(p + 4 * lay.plane), 2 * kGC, DK, P);
+            copy(Qt, reinterpret_cast<const uint16_t*>(p), Keys{});
+            if (DELTA) copy(Wt, reinterpret_cast<const uint16_t*>(p + 4 * lay.plane), Keys{});
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     auto load_second = [&](int c) {  // k 2^(G_n - G), A, 2^G_n
         if (c < ca.chunks) {
             const float* p = source(c);
-            copy(Kt, reinterpret_cast<const uint16_t*>(p + 2 * lay.plane), 2 * kGC, DK, P);
+            copy(Kt, reinterpret_cast<const uint16_t*>(p + 2 * lay.plane), Keys{});
             const float* ap = p + (DELTA ? 6 : 4) * lay.plane;
-            copy(At, reinterpret_cast<const uint16_t*>(ap), 2 * kGC, kGC, PA);
+            copy(At, reinterpret_cast<const uint16_t*>(ap), Tokens{});
             if (tid < DK / 4) cp_async16_to((uint32_t)__cvta_generic_to_shared(Dn + tid * 4), ap + 2 * lay.a_plane + tid * 4);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -942,9 +1058,30 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_scan_kernel(const Chunk
     load_second(0);
     const int wr = (warp & 3) * 16;  // rows of this warp in the products with 64 rows
     const uint16_t* in = static_cast<const uint16_t*>(a.in);
+    const bool pairs = ((a.ld | a.v_off | a.dv) & 1) == 0;
+    float2 u[4][2];      // DELTA: U0 of the next chunk, first four warps
+    uint32_t uv[4][2];   // else v, as pairs of bf16
+    auto load_u = [&](int c) {
+        if (warp >= 4 || c >= ca.chunks) return;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int y = 0; y < 2; ++y) {
+                const int t = wr + g + y * 8, col = v0 + i * 8 + 2 * tq;
+                if (DELTA) {
+                    u[i][y] = *reinterpret_cast<const float2*>(ca.u0 + (((size_t)c * a.heads + h) * kGC + t) * ca.dvp + col);
+                } else {
+                    const bool row = c * kGC + t < a.T;
+                    const uint16_t* v = in + (size_t)(c * kGC + t) * a.ld + a.v_off + (size_t)h * a.dv + col;
+                    if (pairs) uv[i][y] = row && col < a.dv ? *reinterpret_cast<const uint32_t*>(v) : 0u;
+                    else uv[i][y] = (row && col < a.dv ? (uint32_t)v[0] : 0u) | (row && col + 1 < a.dv ? (uint32_t)v[1] << 16 : 0u);
+                }
+            }
+    };
+    load_u(0);
     for (int c = 0; c < ca.chunks; ++c) {
         const int t0 = c * kGC, n = min(kGC, a.T - t0);
-        // ---- the state as head / remainder planes; U0 (or v) on its way
+        // ---- the state as head / remainder planes
 #pragma unroll
         for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -955,22 +1092,6 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_scan_kernel(const Chunk
                 *reinterpret_cast<uint32_t*>(Ss + o) = hi;
                 *reinterpret_cast<uint32_t*>(Ss + DK * PU + o) = lo;
             }
-        float2 u[4][2];
-        if (warp < 4) {
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int y = 0; y < 2; ++y) {
-                    const int t = wr + g + y * 8, col = v0 + i * 8 + 2 * tq;
-                    if (DELTA) {
-                        u[i][y] = *reinterpret_cast<const float2*>(ca.u0 + (((size_t)c * a.heads + h) * kGC + t) * ca.dvp + col);
-                    } else {
-                        const uint16_t* v = in + (size_t)(t0 + t) * a.ld + a.v_off + (size_t)h * a.dv + col;
-                        u[i][y].x = t < n && col < a.dv ? bf16_bits_to_f32(v[0]) : 0.0f;
-                        u[i][y].y = t < n && col + 1 < a.dv ? bf16_bits_to_f32(v[1]) : 0.0f;
-                    }
-                }
-        }
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
         // ---- first half of the block: U = U0 - W S; second half: q 2^G S
@@ -1002,8 +1123,8 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_scan_kernel(const Chunk
             for (int i = 0; i < 4; ++i)
 #pragma unroll
                 for (int y = 0; y < 2; ++y) {
-                    uint32_t hi, lo;
-                    split_bf16x2(u[i][y].x - o[i][2 * y], u[i][y].y - o[i][2 * y + 1], hi, lo);
+                    uint32_t hi = uv[i][y], lo = 0u;
+                    if (DELTA) split_bf16x2(u[i][y].x - o[i][2 * y], u[i][y].y - o[i][2 * y + 1], hi, lo);
                     const int at_ = (wr + g + y * 8) * PU + i * 8 + 2 * tq;
                     *reinterpret_cast<uint32_t*>(Us + at_) = hi;
                     if (DELTA) *reinterpret_cast<uint32_t*>(Us + kGC * PU + at_) = lo;
@@ -1012,6 +1133,7 @@ __global__ void __launch_bounds__(kGThreads) gated_chunk_scan_kernel(const Chunk
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         load_first(c + 1);
+        load_u(c + 1);
         // ---- outputs: + A U
         if (warp >= 4) {
             for (int k = 0; k <= (warp & 3); ++k) {

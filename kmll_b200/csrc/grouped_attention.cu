@@ -44,6 +44,17 @@ __global__ void __launch_bounds__(128) grouped_write_kernel(const GroupedArgs a)
     }
 }
 
+// bf16 rows whose heads are multiples of 8 entries: 16 bytes per thread
+__global__ void __launch_bounds__(256) grouped_copy_kernel(const GroupedArgs a) {
+    pdl_wait();
+    const int nk = a.kv_heads * a.dim / 8, runs = nk + a.kv_heads * a.vdim / 8;
+    const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+    const int t = (int)(i / runs), j = (int)(i - (long long)t * runs);
+    if (t >= a.T || a.pos0 + t >= a.max_seq) return;
+    const uint16_t* src = static_cast<const uint16_t*>(a.in) + (size_t)t * a.ld + (j < nk ? a.k_off + j * 8 : a.v_off + (j - nk) * 8);
+    *reinterpret_cast<uint4*>(static_cast<uint16_t*>(a.cache) + (size_t)(a.pos0 + t) * a.pitch + j * 8) = *reinterpret_cast<const uint4*>(src);
+}
+
 // ---- plain form -----------------------------------------------------------------------------------------------------------------
 constexpr int kPlainWarps = 4;
 template <bool IN32, bool C32>
@@ -487,6 +498,12 @@ int run_prefill(cudaStream_t stream, const GroupedArgs& a) {
 }  // namespace
 
 int grouped_write_cache(cudaStream_t stream, const GroupedArgs& a) {
+    if (!a.in_f32 && !a.cache_f32 && a.at == nullptr && ((a.dim | a.vdim | a.ld | a.k_off | a.v_off) & 7) == 0 && (reinterpret_cast<uintptr_t>(a.in) & 15u) == 0) {
+        const long long items = (long long)a.T * a.kv_heads * (a.dim + a.vdim) / 8;
+        cudaError_t e = launch(grouped_copy_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, stream, true, a);
+        if (e != cudaSuccess) return fail(KMLL_ERR_CUDA, "grouped cache write: %s", cudaGetErrorString(e));
+        return KMLL_OK;
+    }
     auto k = a.in_f32 ? (a.cache_f32 ? grouped_write_kernel<true, true> : grouped_write_kernel<true, false>)
                       : (a.cache_f32 ? grouped_write_kernel<false, true> : grouped_write_kernel<false, false>);
     cudaError_t e = launch(k, dim3(a.T), dim3(128), 0, stream, true, a);

@@ -140,7 +140,7 @@ def forward(config, tensors, tokens, per_layer=None):
 # ---- small random models ----------------------------------------------------------------------------------------------
 def tensor_shapes(config, ranks=None):
     """name -> shape of every tensor; `ranks`: inner sizes of the low-rank pairs (config.json does not name them)."""
-    r = {"a1": 6, "g1": 10, **(ranks or {})}
+    r = {"a1": 6, "g1": 10, "right.a1": 5, **(ranks or {})}
     w, out = config["width"], {}
 
     def norm(name):
@@ -158,7 +158,7 @@ def tensor_shapes(config, ranks=None):
                         p + "left.o": (w, H * a["vdim"])})
             K, V = b["heads"] * b["dim"], b["heads"] * b["vdim"]
             out.update({p + "right.q": (K, w), p + "right.k": (K, w), p + "right.v": (V, w), p + "right.g": (V, w), p + "right.o": (w, V),
-                        p + "right.norm": (b["vdim"],), p + "right.a1": (r["a1"], w), p + "right.a2": (K, r["a1"]), p + "right.a2.b": (K,)})
+                        p + "right.norm": (b["vdim"],), p + "right.a1": (r["right.a1"], w), p + "right.a2": (K, r["right.a1"]), p + "right.a2.b": (K,)})
         else:
             H, G, taps = m["heads"], m["kv_heads"], m["conv"]
             K, V = H * m["dim"], H * m["vdim"]
